@@ -1,10 +1,10 @@
 """The cache manager: paged keys and values with a block table per request, and state slots.
 
-Layers with the same needs (``kv_heads``, ``head_dim``, ``window``) form a *group*;
+Layers with the same needs (``kv_heads``, ``head_dim``, ``window``, ``chunk``) form a *group*;
 each group has its own pool of pages, its own key/value storage and its own block
 tables, so a model whose layers differ (all keys here, a window of them there) gives
 every kind of layer pages of the right shape and gives a window's pages back as soon
-as the window has passed them.  The reference has one geometry for all layers
+as the window has passed them (a chunk's when the next chunk has begun).  The reference has one geometry for all layers
 (src/kv_cache/paged.cpp:100-104, src/model/cuda_llama.cpp:147-154); groups are this
 engine's own.
 
@@ -49,6 +49,31 @@ class KvNeed:
     head_dim: int
     window: Optional[int] = None     # None: every earlier key stays live
     keep_first: int = 0              # with a window: the first keys stay live behind it
+    chunk: Optional[int] = None      # keys of earlier chunks of this many positions are not seen
+
+    def __post_init__(self) -> None:
+        if self.chunk is not None and self.keep_first:
+            raise ValueError("kept first keys belong to a window, not to chunks")
+
+    @property
+    def reach(self) -> Optional[int]:
+        """The most keys one position sees, kept first ones aside (None: no bound)."""
+        bounds = [bound for bound in (self.window, self.chunk) if bound is not None]
+        return min(bounds) if bounds else None
+
+    @property
+    def bounded(self) -> bool:
+        """Whether pages are given back while their request lives."""
+        return self.window is not None or self.chunk is not None
+
+    def first_seen(self, position: int) -> int:
+        """The first position (kept first keys aside) that a query at ``position`` sees."""
+        first = 0
+        if self.window is not None:
+            first = max(0, position - self.window + 1)
+        if self.chunk is not None:
+            first = max(first, position // self.chunk * self.chunk)
+        return first
 
 
 @dataclasses.dataclass(frozen=True)
@@ -147,15 +172,14 @@ class CacheManager:
         for entry in sorted(kv_needs):
             by_need.setdefault(kv_needs[entry], []).append(entry)
         # ``num_pages`` is every group's pool unless ``window_pages`` gives the groups of a
-        # window (by its length) a pool of their own size: a request never holds more of such
-        # a group than its window, the page being filled and the portion it is fed.
+        # window or of chunks (by its length) a pool of their own size: a request never holds
+        # more of such a group than that, the page being filled and the portion it is fed.
         window_pages = dict(window_pages or {})
-        unknown = set(window_pages) - {need.window for need in by_need}
+        unknown = set(window_pages) - {need.reach for need in by_need}
         if unknown:
             raise ValueError(f"window_pages names windows no layer has: {sorted(unknown)}")
         for need, entries in by_need.items():
-            pages = window_pages.get(need.window, num_pages) if need.window is not None \
-                else num_pages
+            pages = window_pages.get(need.reach, num_pages) if need.bounded else num_pages
             if pages <= 0:
                 raise ValueError("a pool needs at least one page")
             group = CacheGroup(len(self.groups), need, entries, pages, self.page_size,
@@ -232,9 +256,9 @@ class CacheManager:
         window passes them and never holds more than the window and the page being filled."""
         needed = []
         for group in self.groups:
-            window = group.need.window
-            live = rows if window is None else \
-                min(rows, window + (1 + self.window_slack_pages) * self.page_size
+            reach = group.need.reach
+            live = rows if reach is None else \
+                min(rows, reach + (1 + self.window_slack_pages) * self.page_size
                     + self.kept_pages(group) * self.page_size)
             needed.append(self.pages_for(live))
         return needed
@@ -247,12 +271,9 @@ class CacheManager:
         return self.pages_for(group.need.keep_first)
 
     def first_page_seen(self, group: CacheGroup, length: int) -> int:
-        """Index of the first page that the window of the query at position ``length`` still
-        reaches in ``group``: 0 without a window.  (Kept first pages lie before it.)"""
-        window = group.need.window
-        if window is None:
-            return 0
-        return max(0, length - window + 1) // self.page_size
+        """Index of the first page that the query at position ``length`` still reaches in
+        ``group``: 0 without a window or chunks.  (Kept first pages lie before it.)"""
+        return group.need.first_seen(length) // self.page_size
 
     def pages_to_extend(self, request: Hashable, new_length: int) -> List[int]:
         """Pages each group must add so that positions ``[0, new_length)`` have a place."""
@@ -333,11 +354,12 @@ class CacheManager:
                              f"reserved {record.reserved}")
         record.length = new_length
         for index, group in enumerate(self.groups):
-            window = group.need.window
-            if window is None:
+            if not group.need.bounded:
                 continue
-            # the next query sits at position new_length and reads keys >= new_length-window+1
-            dead_pages = max(0, self.first_page_seen(group, new_length) - self.window_slack_pages)
+            # the next query sits at position new_length; with slack, what a query that many
+            # pages earlier reads stays too
+            slack = self.window_slack_pages * self.page_size
+            dead_pages = self.first_page_seen(group, max(0, new_length - slack))
             table = record.tables[index]
             # pages in front of `first_live` are gone but for the kept first ones
             first = max(record.first_live[index], self.kept_pages(group))
@@ -424,7 +446,8 @@ class CacheManager:
             if parent.first_live[index] > first:
                 raise ValueError(
                     f"group {group.index}: the source has given back pages that a request at "
-                    f"{tokens} tokens still reads (window {group.need.window})")
+                    f"{tokens} tokens still reads (window {group.need.window}, chunk "
+                    f"{group.need.chunk})")
             kept = min(self.kept_pages(group), first, count)
             shared.append(list(parent.tables[index][:kept]) + [-1] * (first - kept)
                           + list(parent.tables[index][first:count]))
@@ -487,7 +510,7 @@ class CacheManager:
         """With a windowed group an anchor holds the pages its window reaches from the END of
         the prefix, and with per-request state the state at its end, so a request can adopt
         all of the prefix or none of it; otherwise any number of its leading pages."""
-        return bool(self.states) or any(group.need.window is not None for group in self.groups)
+        return bool(self.states) or any(group.need.bounded for group in self.groups)
 
     # Per-request state is not in pages: what a later request needs of a prefix is the state
     # as it stood at the prefix's end.  The engine copies it there (in stream order behind the
@@ -610,6 +633,7 @@ class CacheManager:
             "parked_pages": self.parked_pages,
             "groups": [{
                 "window": group.need.window,
+                "chunk": group.need.chunk,
                 "layers": len(group.entries),
                 "pages": group.pool.num_pages,
                 "free_pages": group.pool.free_pages,

@@ -80,7 +80,7 @@ class PrefixIndex:
         self.maximum_entries = int(maximum_entries)
         # an entry's pages are counted as its prefix's length in pages, which is what it holds
         # of every group that keeps all keys (a windowed group holds a few pages per entry)
-        pools = [group.pool.num_pages for group in cache.groups if group.need.window is None] \
+        pools = [group.pool.num_pages for group in cache.groups if not group.need.bounded] \
             or [group.pool.num_pages for group in cache.groups]
         smallest_pool = min(pools)
         self.maximum_page_references = int(maximum_page_references

@@ -26,6 +26,7 @@ SOURCES = (
     "hx_short_conv.cu",
     "hx_streams.cu",
     "hx_recurrent.cu",
+    "hx_gated_recurrence.cu",
     "hx_rotary_norm.cu",
     "hx_gated_connection.cu",
     "hx_normed_residual.cu",

@@ -1,7 +1,8 @@
 // Paged causal attention over block tables for decode tokens and short prompt portions.
 //
 // Every query token of the flattened batch attends to the keys of its own request at
-// absolute positions [lo, position], lo = 0 or position - window + 1; this step's
+// absolute positions [lo, position], lo = 0, position - window + 1 or the start of the chunk
+// of positions the token lies in; this step's
 // own keys are already in the pages (the rotary/append kernel ran first), so prompt
 // portions and single decode tokens are the same case.  The reference computes the
 // same thing in three stages through a materialised score tensor
@@ -85,6 +86,8 @@ struct AttentionArgs {
   // position i is lowered by slopes[h] * (i - j).
   const float* sinks = nullptr;
   const float* slopes = nullptr;
+  int chunk = 0;          // > 0: positions see each other only inside chunks of this many
+  float softcap = 0.0f;   // > 0: the scaled score s becomes softcap * tanh(s / softcap)
 };
 
 // A finished row with maximum m, weight l and unnormalised sum o, and a sink s: the result is
@@ -107,7 +110,7 @@ __device__ __forceinline__ bool skipped(const AttentionArgs& a, int token) {
 __device__ __forceinline__ void key_range(const AttentionArgs& a, int token, int& lo, int& hi) {
   const int position = a.positions[token];
   hi = position + 1;
-  lo = a.window > 0 ? max(0, hi - a.window) : 0;
+  lo = hx_first_seen(position, a.window, a.chunk);
 }
 
 // With kept first keys a row sees [0, kept) and [lo, hi), kept = min(keep_first, lo).  The
@@ -295,6 +298,7 @@ __global__ __launch_bounds__(WARPS_PER_BLOCK * 32) void paged_attention_kernel(A
         dot = fmaf(qs[d + 1], hx_to_float<T>(k[1]), dot);
       }
       score = dot * a.scale;
+      if (a.softcap > 0.0f) score = a.softcap * tanhf(score / a.softcap);
       if (a.slopes != nullptr)
         score -= a.slopes[item.head] * static_cast<float>(a.positions[item.token] - key);
     }
@@ -394,8 +398,8 @@ __device__ __forceinline__ int row_keys(const AttentionArgs& a, int token) {
   return a.positions[token] + 1;
 }
 
-// With a window a row of `keys` keys (its own position + 1) sees the keys from
-// lo = keys - window on, and the first keep_first keys behind that.  Its chunks are the blocks
+// With a window or chunks a row of `keys` keys (its own position + 1) sees the keys from
+// lo = hx_first_seen() on, and the first keep_first keys behind that.  Its chunks are the blocks
 // of KEYS keys that hold kept keys (as far as they end before the block of `lo`) followed by
 // the blocks from the one that holds `lo`: chunk c of the row is block c below `kept`, block
 // c + skip from there on.
@@ -405,8 +409,8 @@ __device__ __forceinline__ void row_chunks(const AttentionArgs& a, int keys, int
   kept = 0;
   skip = 0;
   n = (keys + KEYS - 1) / KEYS;
-  if (a.window > 0 && keys > a.window) {
-    const int first_block = (keys - a.window) / KEYS;
+  if (keys > 0 && (a.window > 0 || a.chunk > 0)) {
+    const int first_block = hx_first_seen(keys - 1, a.window, a.chunk) / KEYS;
     kept = min((a.keep_first + KEYS - 1) / KEYS, first_block);
     skip = first_block - kept;
     n -= skip;
@@ -661,9 +665,9 @@ void paged_attention_stream_kernel(
   // lane 0 issues
   auto request_chunk = [&](int slot) {
     const int first = ahead.block() * pages_per_chunk;
-    // keys below this one are outside the row's window; their pages, unless they hold kept
-    // keys, may have been given back and are not read
-    const int first_seen = a.window > 0 ? max(0, ahead.keys - a.window) : 0;
+    // keys below this one are outside the row's window or chunk; their pages, unless they hold
+    // kept keys, may have been given back and are not read
+    const int first_seen = hx_first_seen(ahead.keys - 1, a.window, a.chunk);
     if (ahead.token != window_token || first < window_base || first >= window_base + 32) {
       window_token = ahead.token;
       window_base = first & ~31;
@@ -793,8 +797,8 @@ void paged_attention_stream_kernel(
     const uint32_t v_half = k_half + Config::kChunkBytes;
     const int block_key0 = at.block() * KEYS;            // position of the chunk's first key
     const int keys_here = min(KEYS, at.keys - block_key0);
-    // a chunk that reaches below the window's first key holds keys the row does not see
-    const int window_from = a.window > 0 ? at.keys - a.window - block_key0 : -1;
+    // a block that reaches below the row's first key holds keys the row does not see
+    const int window_from = hx_first_seen(at.keys - 1, a.window, a.chunk) - block_key0;
     const unsigned bad_pages = (unreadable >> (4 * slot)) & 0xfu;
 
     // Whatever lies behind the last key of the request in its last page, and pages that
@@ -837,9 +841,15 @@ void paged_attention_stream_kernel(
       score[2 * tile + 1] = s[tile][2];
     }
     float chunk_max = -INFINITY;
+    if (a.softcap > 0.0f) {
+      hx_level_off_fast(score, a.scale / a.softcap, a.softcap);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 2 * kTiles; ++j) score[j] *= a.scale;
+    }
     if (a.slopes != nullptr) {
       // the distance from the row's own position (at.keys - 1) to key group + 8 j of the chunk
-      const float slope = a.slopes[at.head] / a.scale;
+      const float slope = a.slopes[at.head];
       const int distance0 = at.keys - 1 - block_key0 - group;
 #pragma unroll
       for (int j = 0; j < 2 * kTiles; ++j)
@@ -847,17 +857,14 @@ void paged_attention_stream_kernel(
     }
     if (keys_here == KEYS && bad_pages == 0u && window_from <= 0) {
 #pragma unroll
-      for (int j = 0; j < 2 * kTiles; ++j) {
-        score[j] *= a.scale;
-        chunk_max = fmaxf(chunk_max, score[j]);
-      }
+      for (int j = 0; j < 2 * kTiles; ++j) chunk_max = fmaxf(chunk_max, score[j]);
     } else {
 #pragma unroll
       for (int j = 0; j < 2 * kTiles; ++j) {
         const int key = group + 8 * j;
         const bool visible = key < keys_here && !((bad_pages >> (key / page_size)) & 1u) &&
                              (key >= window_from || block_key0 + key < a.keep_first);
-        score[j] = visible ? score[j] * a.scale : -INFINITY;
+        score[j] = visible ? score[j] : -INFINITY;
         chunk_max = fmaxf(chunk_max, score[j]);
       }
     }
@@ -1091,7 +1098,8 @@ HX_API long long hx_paged_attention_scratch_floats_for(int dtype, int tokens, in
 
 // hx_paged_attention with kept first keys: a row at position p sees key j <= p when
 // p - j < window or j < keep_first (window 0: every earlier key, keep_first is then unused).
-// ... and with the optional per-head sinks and distance slopes (see AttentionArgs; null: none).
+// ... and with the optional per-head sinks and distance slopes (null: none), chunks (0: none)
+// and a level the scores run into (0: none); see AttentionArgs.
 HX_API int hx_paged_attention_biased(const void* q, int ldq, const void* k_cache,
                                      const void* v_cache, int dtype, const int* positions,
                                      const int* token_request, const int* request_table_row,
@@ -1101,7 +1109,8 @@ HX_API int hx_paged_attention_biased(const void* q, int ldq, const void* k_cache
                                      int kv_heads, int head_dim, int page_size, int num_pages,
                                      int window, int keep_first, float scale, int split_keys,
                                      int max_splits, const float* sinks, const float* slopes,
-                                     int* status, cudaStream_t stream) {
+                                     int chunk, float softcap, int* status, cudaStream_t stream) {
+  HX_REQUIRE(chunk >= 0 && softcap >= 0.0f, "hx_paged_attention: bad chunk or softcap");
   HX_REQUIRE(keep_first >= 0, "hx_paged_attention: keep_first must not be negative");
   if (window == 0) keep_first = 0;
   HX_REQUIRE(tokens >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0,
@@ -1121,8 +1130,8 @@ HX_API int hx_paged_attention_biased(const void* q, int ldq, const void* k_cache
   AttentionArgs a{q, ldq, k_cache, v_cache, positions, token_request, request_table_row,
                   block_tables, table_stride, request_start, skip_query_len, out, ldo, partial,
                   arrivals, tokens, heads, kv_heads, head_dim, page_size, num_pages, window,
-                  keep_first, scale, split_keys, max_splits, status, sinks, slopes};
-  HX_REQUIRE(slopes == nullptr || scale != 0.0f, "hx_paged_attention: slopes need a scale");
+                  keep_first, scale, split_keys, max_splits, status, sinks, slopes, chunk,
+                  softcap};
   const long long items = static_cast<long long>(tokens) * heads * max_splits;
   HX_REQUIRE(items / STREAM_WARPS < (1ll << 31) - 1, "hx_paged_attention: grid too large");
   int rc;
@@ -1151,7 +1160,8 @@ HX_API int hx_paged_attention_kept(const void* q, int ldq, const void* k_cache, 
                                    request_table_row, block_tables, table_stride, request_start,
                                    skip_query_len, out, ldo, partial, arrivals, tokens, heads,
                                    kv_heads, head_dim, page_size, num_pages, window, keep_first,
-                                   scale, split_keys, max_splits, nullptr, nullptr, status, stream);
+                                   scale, split_keys, max_splits, nullptr, nullptr, 0, 0.0f, status,
+                                   stream);
 }
 
 HX_API int hx_paged_attention(const void* q, int ldq, const void* k_cache, const void* v_cache,

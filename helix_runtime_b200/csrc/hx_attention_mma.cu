@@ -62,6 +62,8 @@ struct PrefillArgs {
   // position i is lowered by slopes[h] * (i - j).
   const float* sinks = nullptr;
   const float* slopes = nullptr;
+  int chunk = 0;          // > 0: positions see each other only inside chunks of this many
+  float softcap = 0.0f;   // > 0: the scaled score s becomes softcap * tanh(s / softcap)
 };
 
 constexpr int RING = 2;                         // key/value tiles in flight per CTA
@@ -131,11 +133,11 @@ __global__ __launch_bounds__(THREADS, D <= 128 ? 3 : 1) void prefill_attention_k
   const int tokens_here = min(tile_tokens, q_len - row0);
   const int rows_here = tokens_here * pack;
   const int last_key = context + row0 + tokens_here - 1;      // last key any row here sees
-  // With a window the CTA walks the tiles that hold kept first keys, then the tiles from the
-  // one that holds the first key its FIRST row sees through the window; `n_tiles` counts
+  // With a window or chunks the CTA walks the tiles that hold kept first keys, then the tiles
+  // from the one that holds the first key its FIRST row sees; `n_tiles` counts
   // both runs and tile_at(i) is the i-th of them.  Keys from keep_first up to first_needed
   // are seen by no row of the CTA: their pages may have been given back and are not read.
-  const int first_needed = a.window > 0 ? max(0, context + row0 - a.window + 1) : 0;
+  const int first_needed = hx_first_seen(context + row0, a.window, a.chunk);
   const int window_tile0 = first_needed / BLOCK_N;
   const int kept_tiles = a.window > 0 ? min((a.keep_first + BLOCK_N - 1) / BLOCK_N, window_tile0) : 0;
   const int n_tiles = kept_tiles + last_key / BLOCK_N + 1 - window_tile0;
@@ -247,6 +249,10 @@ __global__ __launch_bounds__(THREADS, D <= 128 ? 3 : 1) void prefill_attention_k
   // heads of this lane's two rows (a packed tile's rows are a token's heads side by side)
   const int row_head[2] = {head0 + (warp_row + (lane >> 2)) % pack,
                            head0 + (warp_row + (lane >> 2) + 8) % pack};
+  // the first key each of this lane's two rows sees, and the warp's last row does
+  const int row_first[2] = {hx_first_seen(q_pos0, a.window, a.chunk),
+                            hx_first_seen(q_pos1, a.window, a.chunk)};
+  const int warp_first_last = hx_first_seen(warp_pos_last, a.window, a.chunk);
   float row_slope[2] = {0.0f, 0.0f};
   if (a.slopes != nullptr) {
     row_slope[0] = a.slopes[min(row_head[0], a.heads - 1)];
@@ -274,7 +280,7 @@ __global__ __launch_bounds__(THREADS, D <= 128 ? 3 : 1) void prefill_attention_k
     const int first_stale = tile_state[stage] ? 0 : last_key + 1 - tile * BLOCK_N;
     const int unseen_from = max(a.keep_first, 0) - tile * BLOCK_N;     // tile-relative, may be < 0
     const int unseen_to = first_needed - tile * BLOCK_N;               // exclusive
-    const bool has_unseen = a.window > 0 && unseen_to > 0 && unseen_from < BLOCK_N &&
+    const bool has_unseen = unseen_to > 0 && unseen_from < BLOCK_N &&
                             unseen_from < unseen_to;
     if (first_stale < BLOCK_N || has_unseen) {
       for (int index = tid; index < BLOCK_N * (D / 8); index += THREADS) {
@@ -310,25 +316,33 @@ __global__ __launch_bounds__(THREADS, D <= 128 ? 3 : 1) void prefill_attention_k
 
     // ---- scale, causal mask, running maximum
     const int key0 = tile * BLOCK_N + 2 * (lane & 3);
-    // a tile needs the mask when it reaches beyond the first row's own key, or (window) when
-    // its first key lies outside the window of this warp's last row
+    // a tile needs the mask when it reaches beyond the first row's own key, or when its first
+    // key lies in front of what this warp's last row sees
     const bool needs_mask = tile * BLOCK_N + BLOCK_N - 1 > warp_pos_first ||
-                            (a.window > 0 && warp_pos_last - tile * BLOCK_N >= a.window);
+                            tile * BLOCK_N < warp_first_last;
+    if (a.softcap > 0.0f) {
+#pragma unroll
+      for (int n = 0; n < BLOCK_N / 8; ++n)
+        hx_level_off_fast(s[n], a.scale / a.softcap, a.softcap);
+    } else {
+#pragma unroll
+      for (int n = 0; n < BLOCK_N / 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[n][e] *= a.scale;
+    }
     float tile_max[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int n = 0; n < BLOCK_N / 8; ++n) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        float value = s[n][e] * a.scale;
+        float value = s[n][e];
         if (a.slopes != nullptr)
           value -= row_slope[e >> 1] *
                    static_cast<float>(((e & 2) ? q_pos1 : q_pos0) - (key0 + n * 8 + (e & 1)));
         if (needs_mask) {
           const int key = key0 + n * 8 + (e & 1);
           const int q_pos = (e & 2) ? q_pos1 : q_pos0;
-          if (key > q_pos ||
-              (a.window > 0 && q_pos - key >= a.window && key >= a.keep_first))
-            value = -INFINITY;
+          if (key > q_pos || (key < row_first[e >> 1] && key >= a.keep_first)) value = -INFINITY;
         }
         s[n][e] = value;
         tile_max[e >> 1] = fmaxf(tile_max[e >> 1], value);
@@ -340,7 +354,7 @@ __global__ __launch_bounds__(THREADS, D <= 128 ? 3 : 1) void prefill_attention_k
       tile_max[r] = fmaxf(tile_max[r], __shfl_xor_sync(0xffffffffu, tile_max[r], 1));
       tile_max[r] = fmaxf(tile_max[r], __shfl_xor_sync(0xffffffffu, tile_max[r], 2));
       const float new_max = fmaxf(row_max[r], tile_max[r]);
-      // new_max is finite from the first tile on: key 0 is visible to every row
+      // (without a window or chunks new_max is finite from the first tile on)
       correction[r] = row_max[r] == -INFINITY ? 0.0f : __expf(row_max[r] - new_max);
       row_max[r] = new_max;
       row_sum[r] *= correction[r];
@@ -462,8 +476,10 @@ int prefill_attention(const void* q, int ldq, const void* k_cache,
                                          int kv_heads, int head_dim, int page_size, int num_pages,
                                          float scale, int min_query_len, int window,
                                          int keep_first, int pack, int* status, cudaStream_t stream,
-                      const float* sinks = nullptr, const float* slopes = nullptr) {
+                      const float* sinks = nullptr, const float* slopes = nullptr, int chunk = 0,
+                      float softcap = 0.0f) {
   HX_REQUIRE(window >= 0 && keep_first >= 0, "hx_prefill_attention: bad window");
+  HX_REQUIRE(chunk >= 0 && softcap >= 0.0f, "hx_prefill_attention: bad chunk or softcap");
   if (window == 0) keep_first = 0;
   HX_REQUIRE(hx_prefill_attention_supports(head_dim, page_size),
              "hx_prefill_attention: head_dim %d with pages of %d is not supported (head sizes in "
@@ -484,7 +500,7 @@ int prefill_attention(const void* q, int ldq, const void* k_cache,
                 static_cast<const __nv_bfloat16*>(v_cache), request_start, request_context,
                 request_table_row, block_tables, table_stride, static_cast<__nv_bfloat16*>(out),
                 ldo, requests, heads, kv_heads, page_size, num_pages, scale, min_query_len, status,
-                window, keep_first, pack, sinks, slopes};
+                window, keep_first, pack, sinks, slopes, chunk, softcap};
   int rc = HX_ERR_UNSUPPORTED;
   switch (head_dim) {
     case 16: rc = launch<16>(a, tile_bound, stream); break;
@@ -563,8 +579,8 @@ HX_API int hx_prefill_attention(const void* q, int ldq, const void* k_cache, con
                                        num_pages, scale, min_query_len, 0, 0, status, stream);
 }
 
-// The same with the optional per-head sinks and distance slopes (null: none); pack_heads != 0
-// takes the kernel whose rows are a token's heads (hx_prefill_attention_packed).
+// The same with the optional per-head sinks and distance slopes (null: none), chunks (0: none)
+// and a level the scores run into (0: none; see PrefillArgs); pack_heads != 0 takes the kernel whose rows are a token's heads (hx_prefill_attention_packed).
 HX_API int hx_prefill_attention_biased(const void* q, int ldq, const void* k_cache,
                                        const void* v_cache, const int* request_start,
                                        const int* request_context, const int* request_table_row,
@@ -573,7 +589,8 @@ HX_API int hx_prefill_attention_biased(const void* q, int ldq, const void* k_cac
                                        int kv_heads, int head_dim, int page_size, int num_pages,
                                        float scale, int min_query_len, int window,
                                        int keep_first, int pack_heads, const float* sinks,
-                                       const float* slopes, int* status, cudaStream_t stream) {
+                                       const float* slopes, int chunk, float softcap, int* status,
+                                       cudaStream_t stream) {
   HX_REQUIRE(!pack_heads || hx_prefill_attention_packed_tokens(heads, kv_heads) > 0,
              "hx_prefill_attention_biased: %d heads on %d key/value heads do not pack", heads,
              kv_heads);
@@ -581,5 +598,5 @@ HX_API int hx_prefill_attention_biased(const void* q, int ldq, const void* k_cac
                            request_table_row, block_tables, table_stride, out, ldo, requests,
                            tile_bound, heads, kv_heads, head_dim, page_size, num_pages, scale,
                            min_query_len, window, keep_first, pack_heads ? heads / kv_heads : 1,
-                           status, stream, sinks, slopes);
+                           status, stream, sinks, slopes, chunk, softcap);
 }

@@ -98,6 +98,8 @@ struct TcPrefillArgs {
   // position i is lowered by slopes[h] * (i - j).
   const float* sinks = nullptr;
   const float* slopes = nullptr;
+  int chunk = 0;          // > 0: positions see each other only inside chunks of this many
+  float softcap = 0.0f;   // > 0: the scaled score s becomes softcap * tanh(s / softcap)
 };
 
 template <int D>
@@ -173,13 +175,13 @@ __global__ __launch_bounds__(THREADS, 1) void prefill_attention_tc_kernel(TcPref
   const int row0 = tile_in_request * LANES * BLOCK_M;         // first query row of the CTA
   const int rows_here = min(LANES * BLOCK_M, q_len - row0);
   const int last_key = context + row0 + rows_here - 1;        // last key any row here sees
-  // With a window the CTA walks the key tiles that hold kept first keys and then the tiles
-  // from the one with the first key its FIRST row sees through the window; `skipped` tiles lie
+  // With a window or chunks the CTA walks the key tiles that hold kept first keys and then the
+  // tiles from the one with the first key its FIRST row sees; `skipped` tiles lie
   // between the two runs.  Every loop below counts TURNS: turn t works on key tile
   // tile_at(t); rings and barriers go by turns, positions and pages by key tiles.  Keys from
   // keep_first up to first_needed are seen by no row of the CTA: their pages may have been
   // given back and are not read.
-  const int first_needed = a.window > 0 ? max(0, context + row0 - a.window + 1) : 0;
+  const int first_needed = hx_first_seen(context + row0, a.window, a.chunk);
   const int kept_tiles =
       a.window > 0 ? min((a.keep_first + BLOCK_N - 1) / BLOCK_N, first_needed / BLOCK_N) : 0;
   const int skipped = first_needed / BLOCK_N - kept_tiles;
@@ -488,6 +490,7 @@ __global__ __launch_bounds__(THREADS, 1) void prefill_attention_tc_kernel(TcPref
     float row_max = -INFINITY;      // the reference of this row's exponentials, in log2 units
     float row_sum = 0.0f;
     const float scale_log2 = a.scale * 1.4426950408889634f;
+    const int row_first = hx_first_seen(q_position, a.window, a.chunk);     // first key this row sees
     // a slope per position of distance, in the same log2 units (0: none)
     const float slope_log2 = a.slopes != nullptr ? a.slopes[head] * 1.4426950408889634f : 0.0f;
     bool ok = true;
@@ -521,7 +524,13 @@ __global__ __launch_bounds__(THREADS, 1) void prefill_attention_tc_kernel(TcPref
 #pragma unroll
         for (int c = 0; c < 4; ++c)
 #pragma unroll
-          for (int i = 0; i < 16; ++i) p[c * 16 + i] = __uint_as_float(r[c][i]) * scale_log2;
+          for (int i = 0; i < 16; ++i) p[c * 16 + i] = __uint_as_float(r[c][i]);
+      }
+      if (a.softcap > 0.0f) {
+        hx_level_off_fast(p, a.scale / a.softcap, a.softcap * 1.4426950408889634f);
+      } else {
+#pragma unroll
+        for (int i = 0; i < BLOCK_N; ++i) p[i] *= scale_log2;
       }
       const int key0 = tile_at(tile) * BLOCK_N;
       if (a.slopes != nullptr) {
@@ -535,11 +544,11 @@ __global__ __launch_bounds__(THREADS, 1) void prefill_attention_tc_kernel(TcPref
         for (int i = 0; i < BLOCK_N; ++i)
           if (key0 + i > q_position) p[i] = -INFINITY;
       }
-      if (a.window > 0 && q_position - key0 >= a.window) {
-        // keys of the tile lie outside this row's window: they count only when kept
+      if (key0 < row_first) {
+        // keys of the tile lie in front of what this row sees: they count only when kept
 #pragma unroll
         for (int i = 0; i < BLOCK_N; ++i)
-          if (q_position - (key0 + i) >= a.window && key0 + i >= a.keep_first) p[i] = -INFINITY;
+          if (key0 + i < row_first && key0 + i >= a.keep_first) p[i] = -INFINITY;
       }
       float part_max[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -621,7 +630,7 @@ __global__ __launch_bounds__(THREADS, 1) void prefill_attention_tc_kernel(TcPref
       const int first_stale = last_key + 1 - key0;
       const int unseen_from = a.keep_first - key0;      // tile-relative; may be negative
       const int unseen_to = first_needed - key0;        // exclusive
-      const bool has_unseen = a.window > 0 && unseen_to > 0 && unseen_from < BLOCK_N &&
+      const bool has_unseen = unseen_to > 0 && unseen_from < BLOCK_N &&
                               unseen_from < unseen_to;
       if (first_stale < BLOCK_N || has_unseen) {
         ok = wait_for(&v_full[tile % V_STAGES], static_cast<uint32_t>(tile / V_STAGES) & 1u);
@@ -726,7 +735,8 @@ HX_API int hx_prefill_attention_tc_supports(int head_dim, int page_size) {
 
 // The arguments of hx_prefill_attention; tile_bound bounds the number of 256-token query tiles
 // (a larger bound only launches CTAs that leave at once).
-// ... and with the optional per-head sinks and distance slopes (see TcPrefillArgs; null: none).
+// ... and with the optional per-head sinks and distance slopes (null: none), chunks (0: none)
+// and a level the scores run into (0: none); see TcPrefillArgs.
 HX_API int hx_prefill_attention_tc_biased(const void* q, int ldq, const void* k_cache,
                                           const void* v_cache, const int* request_start,
                                           const int* request_context,
@@ -735,8 +745,9 @@ HX_API int hx_prefill_attention_tc_biased(const void* q, int ldq, const void* k_
                                           int tile_bound, int heads, int kv_heads, int head_dim,
                                           int page_size, int num_pages, float scale,
                                           int min_query_len, int window, int keep_first,
-                                          const float* sinks, const float* slopes, int* status,
-                                          cudaStream_t stream) {
+                                          const float* sinks, const float* slopes, int chunk,
+                                          float softcap, int* status, cudaStream_t stream) {
+  HX_REQUIRE(chunk >= 0 && softcap >= 0.0f, "hx_prefill_attention_tc: bad chunk or softcap");
   HX_REQUIRE(window >= 0 && keep_first >= 0, "hx_prefill_attention_tc: bad window");
   if (window == 0) keep_first = 0;
   HX_REQUIRE(hx_prefill_attention_tc_supports(head_dim, page_size),
@@ -758,7 +769,7 @@ HX_API int hx_prefill_attention_tc_biased(const void* q, int ldq, const void* k_
                   static_cast<const __nv_bfloat16*>(v_cache), request_start, request_context,
                   request_table_row, block_tables, table_stride, static_cast<__nv_bfloat16*>(out),
                   ldo, requests, heads, kv_heads, page_size, num_pages, scale, min_query_len, status,
-                  window, keep_first, sinks, slopes};
+                  window, keep_first, sinks, slopes, chunk, softcap};
   int rc;
   switch (head_dim) {
     case 64: rc = launch<64>(a, tile_bound, stream); break;
@@ -785,7 +796,7 @@ HX_API int hx_prefill_attention_tc_windowed(const void* q, int ldq, const void* 
                                         request_table_row, block_tables, table_stride, out, ldo,
                                         requests, tile_bound, heads, kv_heads, head_dim, page_size,
                                         num_pages, scale, min_query_len, window, keep_first,
-                                        nullptr, nullptr, status, stream);
+                                        nullptr, nullptr, 0, 0.0f, status, stream);
 }
 
 // Every earlier key (no window).

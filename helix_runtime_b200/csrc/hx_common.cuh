@@ -169,6 +169,48 @@ __host__ __device__ __forceinline__ size_t hx_cache_offset(int page, int kv_head
   return ((page_head * (head_dim / chunk) + dim / chunk) * page_size + slot) * chunk + dim % chunk;
 }
 
+// Which keys a query sees.  The query at `position` sees no key behind itself and none in front
+// of this one: the start of its window of `window` positions (0: no window) and the start of the
+// chunk of `chunk` positions, counted from position 0, that it lies in (0: no chunks).  The
+// first key seen never moves back as the position grows.
+__host__ __device__ __forceinline__ int hx_first_seen(int position, int window, int chunk) {
+  int first = window > 0 && position >= window ? position - window + 1 : 0;
+  if (chunk > 0) {
+    const int start = position - position % chunk;
+    first = start > first ? start : first;
+  }
+  return first;
+}
+
+// x[i] = outer * tanh(inner * x[i]): scores that level off at +-outer.  Where all of a thread's
+// arguments are small (the usual case: scores well below the cap) the first five terms of
+// tanh's series do, whose remainder is below 2e-8 there; otherwise tanh(z) = 1 - 2 / (1 + e^2z)
+// with the hardware exponential, off by about 2^-23.
+template <int N>
+__device__ __forceinline__ void hx_level_off_fast(float (&x)[N], float inner, float outer) {
+  float top = 0.0f;
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    x[i] *= inner;
+    top = fmaxf(top, fabsf(x[i]));
+  }
+  if (top < 0.3f) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const float z = x[i] * x[i];
+      float series = fmaf(z, 62.0f / 2835.0f, -17.0f / 315.0f);
+      series = fmaf(series, z, 2.0f / 15.0f);
+      series = fmaf(series, z, -1.0f / 3.0f);
+      series = fmaf(series, z, 1.0f);
+      x[i] = outer * x[i] * series;
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+      x[i] = outer * (1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * x[i])));
+  }
+}
+
 // The requests that bring at least `min_len` tokens to a step are cut into tiles of `rows`
 // tokens, and the tiles are numbered in the order of the requests.  Which request holds tile
 // number `tile`, which of its tiles is it, and how many has it?  Every lane of a (whole,

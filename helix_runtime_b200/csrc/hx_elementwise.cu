@@ -37,7 +37,7 @@ void hx_count_launches(int kernels) { g_hx_launches.fetch_add(kernels, std::memo
 // counts once, when it is captured).
 HX_API long long hx_launch_count() { return g_hx_launches.load(std::memory_order_relaxed); }
 
-HX_API int hx_abi_version() { return 9; }
+HX_API int hx_abi_version() { return 10; }
 
 // Streaming multiprocessors of the current device (asked once per device); 0 with a message
 // when the device cannot be asked.  Launch sizes that should fill the GPU come from here.
@@ -541,7 +541,8 @@ HX_API int hx_swiglu(float* gate_up, void* act, int out_dtype, int tokens, int i
 // src/kernels/cuda/transformer.cu:100-119); the reference's separate cache append
 // (src/kv_cache/cuda_paged.cpp:561-577) is fused in.
 //
-// qkv row: [q heads | k heads | v heads], each head `head_dim` wide.
+// qkv row: [q heads | k heads | v heads], each head `head_dim` wide; with `shared_values` there
+// are no v heads in the row and the values are the keys as projected, before the rotation.
 // pairing 0: pairs (2p, 2p+1); pairing 1: pairs (p, p + rotary_dim/2).
 // cache layer (keys and values alike): [page][kv_head][head_dim / chunk][slot][chunk],
 // see hx_cache_offset.
@@ -563,7 +564,7 @@ __global__ void rope_append_kernel(T* __restrict__ qkv, int ld, const int* __res
                                    int heads, int kv_heads, int head_dim, int rotary_dim,
                                    int pairing, int page_size, int num_pages, int* status,
                                    float* __restrict__ accum, int ld_accum,
-                                   int release_successor) {
+                                   int release_successor, int shared_values) {
   // The attention kernel that follows fills the GPU with one resident grid of warps that
   // all start on equal runs of work; let in early, they would all leave the wait in the same
   // instant and stay in step, fetching and computing in bursts (measured: twice the time at
@@ -605,7 +606,7 @@ __global__ void rope_append_kernel(T* __restrict__ qkv, int ld, const int* __res
   // coordinate of a v head.
   const int pairs_per_head = head_dim / 2;
   const int first_head = blockIdx.y * ROPE_HEADS_PER_BLOCK;
-  const int total_heads = heads + 2 * kv_heads;
+  const int total_heads = heads + (shared_values ? 1 : 2) * kv_heads;
   const int last_head = min(first_head + ROPE_HEADS_PER_BLOCK, total_heads);
   for (int head = first_head; head < last_head; ++head) {
     T* vec = row + static_cast<size_t>(head) * head_dim;
@@ -637,6 +638,14 @@ __global__ void rope_append_kernel(T* __restrict__ qkv, int ld, const int* __res
         } else {
           a = hx_to_float<T>(vec[i0]);
           b = hx_to_float<T>(vec[i1]);
+        }
+        if (shared_values && head >= heads && page >= 0) {
+          const int kv_head = head - heads;
+          const int chunk = hx_cache_chunk(sizeof(T), head_dim);
+          v_cache[hx_cache_offset(page, kv_head, slot, i0, kv_heads, page_size, head_dim, chunk)] =
+              hx_from_float<T>(a);
+          v_cache[hx_cache_offset(page, kv_head, slot, i1, kv_heads, page_size, head_dim, chunk)] =
+              hx_from_float<T>(b);
         }
         if (rotate) {
           const float c = cos_row[pair];
@@ -691,7 +700,7 @@ __global__ void rope_append_pieces_kernel(
     __nv_bfloat16* __restrict__ v_cache, int write_cache, const float* __restrict__ cos_table,
     const float* __restrict__ sin_table, int table_positions, int heads, int kv_heads,
     int head_dim, int rotary_dim, int pairing, int page_size, int num_pages, int* status,
-    float* __restrict__ accum, int ld_accum, int release_successor) {
+    float* __restrict__ accum, int ld_accum, int release_successor, int shared_values) {
   // with many tokens the attention kernel that follows is launched when this one is done
   // (see above)
   if (release_successor) hx_pdl_trigger();
@@ -704,7 +713,7 @@ __global__ void rope_append_pieces_kernel(
   const int item = blockIdx.y * blockDim.x + threadIdx.x;
   const int head = item / pieces_per_head;
   const int piece = item - head * pieces_per_head;
-  if (head >= heads + 2 * kv_heads) {
+  if (head >= heads + (shared_values ? 1 : 2) * kv_heads) {
     hx_pdl_wait();      // a grid must not be seen complete before its predecessor is
     return;
   }
@@ -762,6 +771,17 @@ __global__ void rope_append_pieces_kernel(
     }
   };
 
+  // a key piece as projected is the value's piece too
+  auto store_shared = [&](int d0, const float (&x)[8]) {
+    if (!shared_values || head < heads || page < 0) return;
+    uint4 packed;
+    __nv_bfloat162* pairs = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) pairs[i] = __floats2bfloat162_rn(x[2 * i], x[2 * i + 1]);
+    *reinterpret_cast<uint4*>(v_cache + hx_cache_offset(page, head - heads, slot, d0, kv_heads,
+                                                        page_size, head_dim, 8)) = packed;
+  };
+
   const int d0 = piece * 8;
   const int half = rotary_dim / 2;
   const bool rotates = head < heads + kv_heads && d0 < rotary_dim;
@@ -772,6 +792,7 @@ __global__ void rope_append_pieces_kernel(
     if (accum == nullptr && head < heads) return;
     float x[8];
     load(d0, x);
+    store_shared(d0, x);
     store(d0, x);
     return;
   }
@@ -803,6 +824,7 @@ __global__ void rope_append_pieces_kernel(
     hx_pdl_wait();
     float x[8];
     load(d0, x);
+    store_shared(d0, x);
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const float a = x[2 * i], b = x[2 * i + 1];
@@ -826,6 +848,8 @@ __global__ void rope_append_pieces_kernel(
     float x[8], y[8];
     load(d0, x);
     load(d0 + half, y);
+    store_shared(d0, x);
+    store_shared(d0 + half, y);
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
       const float a = x[i], b = y[i];
@@ -837,36 +861,39 @@ __global__ void rope_append_pieces_kernel(
   }
 }
 
-HX_API int hx_rope_append(void* qkv, int dtype, int ld, const int* positions,
+// shared_values != 0: a row is [q heads | k heads]; a key head's projection, before the
+// rotation, goes to the value cache too.
+HX_API int hx_rope_append_shared(void* qkv, int dtype, int ld, const int* positions,
                           const int* token_request, const int* request_table_row,
                           const int* block_tables, int table_stride, void* k_cache, void* v_cache,
                           int write_cache, const float* cos_table, const float* sin_table,
                           int table_positions, int tokens, int heads, int kv_heads, int head_dim,
                           int rotary_dim, int pairing, int page_size, int num_pages, int* status,
-                          float* accum, int ld_accum, cudaStream_t stream) {
+                          float* accum, int ld_accum, int shared_values, cudaStream_t stream) {
+  const int row_heads = heads + (shared_values ? 1 : 2) * kv_heads;
   HX_REQUIRE(tokens >= 0 && heads > 0 && kv_heads > 0, "hx_rope_append: bad sizes");
   HX_REQUIRE(head_dim > 0 && head_dim % 2 == 0, "hx_rope_append: head_dim %d must be even", head_dim);
   HX_REQUIRE(rotary_dim >= 0 && rotary_dim <= head_dim && rotary_dim % 2 == 0,
              "hx_rope_append: rotary_dim %d must be even and at most head_dim %d", rotary_dim,
              head_dim);
   HX_REQUIRE(pairing == 0 || pairing == 1, "hx_rope_append: unknown pairing %d", pairing);
-  HX_REQUIRE(ld >= (heads + 2 * kv_heads) * head_dim, "hx_rope_append: row stride too small");
+  HX_REQUIRE(ld >= row_heads * head_dim, "hx_rope_append: row stride too small");
   HX_REQUIRE(!write_cache || (page_size > 0 && num_pages > 0 && k_cache && v_cache),
              "hx_rope_append: cache arguments missing");
   HX_REQUIRE(rotary_dim == 0 || table_positions > 0, "hx_rope_append: empty rotary table");
-  HX_REQUIRE(accum == nullptr || ld_accum >= (heads + 2 * kv_heads) * head_dim,
+  HX_REQUIRE(accum == nullptr || ld_accum >= row_heads * head_dim,
              "hx_rope_append: accumulator stride too small");
   if (tokens == 0) return HX_OK;
   const int release_successor = tokens <= HX_ROPE_RELEASE_TOKENS ? 1 : 0;
   const int threads = head_dim / 2 >= 64 ? 64 : 32;
-  const dim3 grid(tokens, (heads + 2 * kv_heads + ROPE_HEADS_PER_BLOCK - 1) / ROPE_HEADS_PER_BLOCK);
+  const dim3 grid(tokens, (row_heads + ROPE_HEADS_PER_BLOCK - 1) / ROPE_HEADS_PER_BLOCK);
   HX_REQUIRE(grid.y <= 65535, "hx_rope_append: too many heads");
   const int half = rotary_dim / 2;
   const bool whole_pieces =
       dtype == HX_BF16 && head_dim % 8 == 0 && ld % 8 == 0 && (accum == nullptr || ld_accum % 4 == 0) &&
       (pairing == 0 || half % 8 == 0);
   if (whole_pieces) {
-    const int items = (heads + 2 * kv_heads) * (head_dim / 8);
+    const int items = row_heads * (head_dim / 8);
     const int block = items >= 256 ? 256 : ((items + 31) / 32) * 32;
     const dim3 piece_grid(tokens, (items + block - 1) / block);
     HX_REQUIRE(piece_grid.y <= 65535, "hx_rope_append: too many heads");
@@ -875,16 +902,30 @@ HX_API int hx_rope_append(void* qkv, int dtype, int ld, const int* positions,
               block_tables, table_stride, static_cast<__nv_bfloat16*>(k_cache),
               static_cast<__nv_bfloat16*>(v_cache), write_cache, cos_table, sin_table,
               table_positions, heads, kv_heads, head_dim, rotary_dim, pairing, page_size, num_pages,
-              status, accum, ld_accum, release_successor);
+              status, accum, ld_accum, release_successor, shared_values);
   } else if (dtype == HX_F32) {
-    hx_launch(rope_append_kernel<float>, grid, threads, 0, stream,  static_cast<float*>(qkv), ld, positions, token_request, request_table_row, block_tables, table_stride, static_cast<float*>(k_cache), static_cast<float*>(v_cache), write_cache, cos_table, sin_table, table_positions, heads, kv_heads, head_dim, rotary_dim, pairing, page_size, num_pages, status, accum, ld_accum, release_successor);
+    hx_launch(rope_append_kernel<float>, grid, threads, 0, stream,  static_cast<float*>(qkv), ld, positions, token_request, request_table_row, block_tables, table_stride, static_cast<float*>(k_cache), static_cast<float*>(v_cache), write_cache, cos_table, sin_table, table_positions, heads, kv_heads, head_dim, rotary_dim, pairing, page_size, num_pages, status, accum, ld_accum, release_successor, shared_values);
   } else if (dtype == HX_BF16) {
-    hx_launch(rope_append_kernel<__nv_bfloat16>, grid, threads, 0, stream,  static_cast<__nv_bfloat16*>(qkv), ld, positions, token_request, request_table_row, block_tables, table_stride, static_cast<__nv_bfloat16*>(k_cache), static_cast<__nv_bfloat16*>(v_cache), write_cache, cos_table, sin_table, table_positions, heads, kv_heads, head_dim, rotary_dim, pairing, page_size, num_pages, status, accum, ld_accum, release_successor);
+    hx_launch(rope_append_kernel<__nv_bfloat16>, grid, threads, 0, stream,  static_cast<__nv_bfloat16*>(qkv), ld, positions, token_request, request_table_row, block_tables, table_stride, static_cast<__nv_bfloat16*>(k_cache), static_cast<__nv_bfloat16*>(v_cache), write_cache, cos_table, sin_table, table_positions, heads, kv_heads, head_dim, rotary_dim, pairing, page_size, num_pages, status, accum, ld_accum, release_successor, shared_values);
   } else {
     HX_REQUIRE(false, "hx_rope_append: unknown dtype %d", dtype);
   }
   HX_CHECK_LAUNCH("hx_rope_append");
   return HX_OK;
+}
+
+HX_API int hx_rope_append(void* qkv, int dtype, int ld, const int* positions,
+                          const int* token_request, const int* request_table_row,
+                          const int* block_tables, int table_stride, void* k_cache, void* v_cache,
+                          int write_cache, const float* cos_table, const float* sin_table,
+                          int table_positions, int tokens, int heads, int kv_heads, int head_dim,
+                          int rotary_dim, int pairing, int page_size, int num_pages, int* status,
+                          float* accum, int ld_accum, cudaStream_t stream) {
+  return hx_rope_append_shared(qkv, dtype, ld, positions, token_request, request_table_row,
+                               block_tables, table_stride, k_cache, v_cache, write_cache, cos_table,
+                               sin_table, table_positions, tokens, heads, kv_heads, head_dim,
+                               rotary_dim, pairing, page_size, num_pages, status, accum, ld_accum, 0,
+                               stream);
 }
 
 // ------------------------------------------------- tokens of a step queued ahead

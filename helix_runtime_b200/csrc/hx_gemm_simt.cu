@@ -21,7 +21,7 @@ template <typename T, int EPI>
 __global__ __launch_bounds__(256) void gemm_simt_kernel(const T* __restrict__ x, int ldx,
                                                         const T* __restrict__ w, int ldw,
                                                         void* __restrict__ out, int ldo, int tokens,
-                                                        int features, int depth) {
+                                                        int features, int depth, float softcap) {
   __shared__ float xs[BK][BM + 4];
   __shared__ float ws[BK][BN + 4];
   hx_pdl_prologue();
@@ -77,7 +77,8 @@ __global__ __launch_bounds__(256) void gemm_simt_kernel(const T* __restrict__ x,
       if (EPI == EPI_STORE) {
         static_cast<T*>(out)[index] = hx_from_float<T>(acc[i][j]);
       } else if (EPI == EPI_STORE_F32) {
-        static_cast<float*>(out)[index] = acc[i][j];
+        static_cast<float*>(out)[index] =
+            softcap > 0.0f ? softcap * tanhf(acc[i][j] / softcap) : acc[i][j];
       } else {
         static_cast<float*>(out)[index] += acc[i][j];
       }
@@ -87,19 +88,19 @@ __global__ __launch_bounds__(256) void gemm_simt_kernel(const T* __restrict__ x,
 
 template <typename T>
 int launch(const void* x, int ldx, const void* w, int ldw, void* out, int ldo, int tokens,
-           int features, int depth, int epilogue, cudaStream_t stream) {
+           int features, int depth, int epilogue, float softcap, cudaStream_t stream) {
   const dim3 grid((features + BN - 1) / BN, (tokens + BM - 1) / BM);
   const T* xp = static_cast<const T*>(x);
   const T* wp = static_cast<const T*>(w);
   switch (epilogue) {
     case EPI_STORE:
-      hx_launch(gemm_simt_kernel<T, EPI_STORE>, grid, 256, 0, stream, xp, ldx, wp, ldw, out, ldo, tokens, features, depth);
+      hx_launch(gemm_simt_kernel<T, EPI_STORE>, grid, 256, 0, stream, xp, ldx, wp, ldw, out, ldo, tokens, features, depth, softcap);
       break;
     case EPI_STORE_F32:
-      hx_launch(gemm_simt_kernel<T, EPI_STORE_F32>, grid, 256, 0, stream, xp, ldx, wp, ldw, out, ldo, tokens, features, depth);
+      hx_launch(gemm_simt_kernel<T, EPI_STORE_F32>, grid, 256, 0, stream, xp, ldx, wp, ldw, out, ldo, tokens, features, depth, softcap);
       break;
     case EPI_ADD_F32:
-      hx_launch(gemm_simt_kernel<T, EPI_ADD_F32>, grid, 256, 0, stream, xp, ldx, wp, ldw, out, ldo, tokens, features, depth);
+      hx_launch(gemm_simt_kernel<T, EPI_ADD_F32>, grid, 256, 0, stream, xp, ldx, wp, ldw, out, ldo, tokens, features, depth, softcap);
       break;
     default:
       hx_set_error("hx_gemm_simt: unknown epilogue %d", epilogue);
@@ -111,22 +112,32 @@ int launch(const void* x, int ldx, const void* w, int ldw, void* out, int ldo, i
 }  // namespace
 
 // epilogue 0: out (compute dtype) = x w^T; 1: out (float32) = x w^T; 2: out (float32) += x w^T
-HX_API int hx_gemm_simt(const void* x, int ldx, const void* w, int ldw, void* out, int ldo,
-                        int dtype, int tokens, int features, int depth, int epilogue,
-                        cudaStream_t stream) {
+// softcap > 0 (epilogue 1 only): the sums run into a level, softcap * tanh(x w^T / softcap)
+HX_API int hx_gemm_simt_softcapped(const void* x, int ldx, const void* w, int ldw, void* out,
+                                   int ldo, int dtype, int tokens, int features, int depth,
+                                   int epilogue, float softcap, cudaStream_t stream) {
+  HX_REQUIRE(softcap >= 0.0f && (softcap == 0.0f || epilogue == EPI_STORE_F32),
+             "hx_gemm_simt: a softcap belongs to a float32 store");
   HX_REQUIRE(tokens >= 0 && features > 0 && depth > 0, "hx_gemm_simt: bad sizes");
   HX_REQUIRE(ldx >= depth && ldw >= depth && ldo >= features, "hx_gemm_simt: bad strides");
   HX_REQUIRE((tokens + BM - 1) / BM <= 65535, "hx_gemm_simt: too many rows (%d)", tokens);
   if (tokens == 0) return HX_OK;
   int rc;
   if (dtype == HX_F32) {
-    rc = launch<float>(x, ldx, w, ldw, out, ldo, tokens, features, depth, epilogue, stream);
+    rc = launch<float>(x, ldx, w, ldw, out, ldo, tokens, features, depth, epilogue, softcap, stream);
   } else if (dtype == HX_BF16) {
-    rc = launch<__nv_bfloat16>(x, ldx, w, ldw, out, ldo, tokens, features, depth, epilogue, stream);
+    rc = launch<__nv_bfloat16>(x, ldx, w, ldw, out, ldo, tokens, features, depth, epilogue, softcap, stream);
   } else {
     HX_REQUIRE(false, "hx_gemm_simt: unknown dtype %d", dtype);
   }
   if (rc != HX_OK) return rc;
   HX_CHECK_LAUNCH("hx_gemm_simt");
   return HX_OK;
+}
+
+HX_API int hx_gemm_simt(const void* x, int ldx, const void* w, int ldw, void* out, int ldo,
+                        int dtype, int tokens, int features, int depth, int epilogue,
+                        cudaStream_t stream) {
+  return hx_gemm_simt_softcapped(x, ldx, w, ldw, out, ldo, dtype, tokens, features, depth, epilogue,
+                                 0.0f, stream);
 }

@@ -43,7 +43,8 @@ constexpr int THREADS = 192;
 
 enum Epilogue : int {
   EPI_STORE_BF16 = 0, EPI_STORE_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU = 3,
-  EPI_ROPE_APPEND = 4      // persistent kernel only, see RopeArgs
+  EPI_ROPE_APPEND = 4,     // persistent kernel only, see RopeArgs
+  EPI_BLOCK_GATES = 6      // persistent kernel only, see BlockGateArgs
 };
 
 // Where the [128 rows x 64 k] box of the weights that begins at row `row`, k-block `kb`, is.
@@ -60,13 +61,19 @@ __device__ __forceinline__ void load_weight_box(void* dst, const CUtensorMap* ma
   }
 }
 
+// A float32 store may let the sums run into a level: cap * tanh(x / cap) (cap 0: as they are).
+__device__ __forceinline__ float level_off(float x, float cap) {
+  return cap > 0.0f ? cap * tanhf(x / cap) : x;
+}
+
 // One epilogue warp's share of a finished tile: its 32 features (tensor-memory lanes) for all
 // BN token columns, 16 columns at a time.  With SwiGLU the up accumulator sits BN columns on.
 template <int BN, int EPI>
 __device__ __forceinline__ void write_tile(void* out, int ldo, int tokens, int features,
                                            uint32_t lane_address, int feature, int token0,
                                            int activation, float gate_limit,
-                                           const float* gate_bias, const float* up_bias) {
+                                           const float* gate_bias, const float* up_bias,
+                                           float softcap) {
   const bool feature_ok = feature < features;
   // this thread's feature is one row of the gate and one of the up matrix: one bias each
   const float gate_b = EPI == EPI_SWIGLU && gate_bias != nullptr && feature_ok ? gate_bias[feature] : 0.0f;
@@ -92,7 +99,7 @@ __device__ __forceinline__ void write_tile(void* out, int ldo, int tokens, int f
           if (EPI == EPI_STORE_BF16 || EPI == EPI_SWIGLU) {
             static_cast<__nv_bfloat16*>(out)[index] = __float2bfloat16_rn(acc[j]);
           } else if (EPI == EPI_STORE_F32) {
-            static_cast<float*>(out)[index] = acc[j];
+            static_cast<float*>(out)[index] = level_off(acc[j], softcap);
           } else {
             // a reduction at the memory side: nothing to wait for.  With one writer per
             // element the sum is still deterministic.
@@ -148,6 +155,7 @@ struct GemmArgs {
   // gated epilogue: float32 biases of the gate and the up rows, [features] each (null: none)
   const float* gate_bias = nullptr;
   const float* up_bias = nullptr;
+  float softcap = 0.0f;       // float32 store: see level_off
 };
 
 template <int BN, int EPI>
@@ -284,7 +292,8 @@ __global__ __launch_bounds__(THREADS) void gemm_tc_kernel(
         tc_fence_after();
         const uint32_t lane_address = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16);
         write_tile<BN, EPI>(args.out, args.ldo, args.tokens, args.features, lane_address, feature,
-                            token0, args.activation, args.gate_limit, args.gate_bias, args.up_bias);
+                            token0, args.activation, args.gate_limit, args.gate_bias, args.up_bias,
+                            args.softcap);
       }
     }
   }
@@ -352,6 +361,24 @@ struct RopeArgs {
   const float* sin_table;
   int table_positions;
   int heads, kv_heads, head_dim, rotary_dim, page_size, num_pages;
+  int shared_values;           // no v heads: the values are the keys before the rotation
+};
+
+// A block-diagonal product whose epilogue turns its sums into the decay and the push of a gated
+// linear recurrence (see hx_gated_recurrence.cu).  Block b of the channels multiplies columns
+// [b * size, (b + 1) * size) of the token rows with its own two square matrices, rows [2 b size,
+// 2 b size + size) of the weights (the recurrence gate) and the `size` rows behind them (the
+// input gate); a tile holds 128 channels of one block, both gates of a channel in one thread.
+struct BlockGateArgs {
+  const __nv_bfloat16* u;      // the token rows again: the input gate multiplies them
+  int ld_u;
+  const float* r_bias;         // [channels]
+  const float* i_bias;
+  const float* rate;
+  float* decay;                // [tokens, channels]: a - 1
+  float* push;                 // [tokens, channels]: sqrt(1 - a^2) i u
+  int size, channels;
+  int tiles;                   // 128-channel tiles of a block
 };
 
 #ifndef HX_GEMM_STREAM_K
@@ -382,6 +409,8 @@ struct PersistentArgs {
   // gated epilogue: float32 biases of the gate and the up rows, [features] each (null: none)
   const float* gate_bias = nullptr;
   const float* up_bias = nullptr;
+  float softcap = 0.0f;       // float32 store: see level_off
+  BlockGateArgs gates = BlockGateArgs{};      // EPI_BLOCK_GATES only
 };
 
 // What a CTA works on at a time: a tile, or (`partial`) a run of k-blocks of a tile that
@@ -464,7 +493,7 @@ template <int EPI>
 __device__ __forceinline__ void write_row(void* out, int ldo, int features, uint32_t lane_address,
                                           int token, int tokens, int feature0, int activation,
                                           float gate_limit, const float* gate_bias,
-                                          const float* up_bias) {
+                                          const float* up_bias, float softcap) {
   using Element = typename std::conditional<EPI == EPI_STORE_BF16 || EPI == EPI_SWIGLU,
                                             __nv_bfloat16, float>::type;
   constexpr int kColumns = EPI == EPI_SWIGLU ? BM : 2 * BM;
@@ -491,6 +520,10 @@ __device__ __forceinline__ void write_row(void* out, int ldo, int features, uint
       }
 #pragma unroll
       for (int j = 0; j < 16; ++j) acc[j] = hx_gated_fast(acc[j], up[j], activation, gate_limit);
+    }
+    if (EPI == EPI_STORE_F32 && softcap > 0.0f) {
+#pragma unroll
+      for (int j = 0; j < 16; ++j) acc[j] = level_off(acc[j], softcap);
     }
     if (token >= tokens) continue;
     Element* row = static_cast<Element*>(out) + static_cast<size_t>(token) * ldo + feature0 + column;
@@ -571,6 +604,16 @@ __device__ __forceinline__ void write_row_rope(const PersistentArgs& a, uint32_t
     const int d0 = inside - head * r.head_dim;
 #pragma unroll
     for (int j = 0; j < 16; ++j) x[j] = __bfloat162float(__float2bfloat16_rn(x[j]));
+    if (r.shared_values && is_key && page >= 0) {
+      uint4 packed[2];
+      __nv_bfloat162* pairs = reinterpret_cast<__nv_bfloat162*>(packed);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) pairs[j] = __floats2bfloat162_rn(x[2 * j], x[2 * j + 1]);
+      *reinterpret_cast<uint4*>(r.v_cache + hx_cache_offset(page, head, slot, d0, r.kv_heads,
+                                                            r.page_size, r.head_dim, 8)) = packed[0];
+      *reinterpret_cast<uint4*>(r.v_cache + hx_cache_offset(page, head, slot, d0 + 8, r.kv_heads,
+                                                            r.page_size, r.head_dim, 8)) = packed[1];
+    }
     if ((is_query || is_key) && d0 < r.rotary_dim) {
       // the eight angles of this piece: four 16-byte loads where the table's rows allow it
       // (every lane reads another row of the table, so the number of loads is what counts)
@@ -618,6 +661,49 @@ __device__ __forceinline__ void write_row_rope(const PersistentArgs& a, uint32_t
   }
 }
 
+// The gates' epilogue for this thread's token: channels [channel0, channel0 + 128) of block
+// `block`, as far as the block has them.
+__device__ __forceinline__ void write_row_gates(const BlockGateArgs& g, uint32_t lane_address,
+                                                int token, int tokens, int block, int channel0) {
+  const bool live = token < tokens;
+  const __nv_bfloat16* u_row = g.u + static_cast<size_t>(live ? token : 0) * g.ld_u;
+#pragma unroll 1
+  for (int column = 0; column < BM; column += 16) {
+    const int left = g.size - channel0 - column;      // channels of the block from here on
+    if (left <= 0) break;                              // uniform over the warp
+    float r[16], i[16];
+    tmem_load16(lane_address + column, r);
+    tmem_load16(lane_address + BM + column, i);
+    if (!live) continue;
+    // sizes are multiples of 8, so a run of eight channels is there or not as a whole
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      if (half * 8 >= left) continue;
+      const int c = block * g.size + channel0 + column + half * 8;
+      const uint4 packed = *reinterpret_cast<const uint4*>(u_row + c);
+      const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&packed);
+      float d[8], p[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float2 pair = __bfloat1622float2(pairs[j / 2]);
+        const float u = (j & 1) ? pair.y : pair.x;
+        const float r_gate =
+            __fdividef(1.0f, 1.0f + __expf(-(r[half * 8 + j] + __ldg(g.r_bias + c + j))));
+        const float i_gate =
+            __fdividef(1.0f, 1.0f + __expf(-(i[half * 8 + j] + __ldg(g.i_bias + c + j))));
+        d[j] = expm1f(-__ldg(g.rate + c + j) * r_gate);
+        p[j] = sqrtf(-d[j] * (2.0f + d[j])) * i_gate * u;
+      }
+      float4* decay = reinterpret_cast<float4*>(g.decay + static_cast<size_t>(token) * g.channels + c);
+      float4* push = reinterpret_cast<float4*>(g.push + static_cast<size_t>(token) * g.channels + c);
+      decay[0] = make_float4(d[0], d[1], d[2], d[3]);
+      decay[1] = make_float4(d[4], d[5], d[6], d[7]);
+      push[0] = make_float4(p[0], p[1], p[2], p[3]);
+      push[1] = make_float4(p[4], p[5], p[6], p[7]);
+    }
+  }
+}
+
 // The piece of a tile that a partial unit computed: added to the float32 output with atomic
 // adds (four values at a time where the row allows).
 __device__ __forceinline__ void add_row_atomically(float* out, int ldo, int features,
@@ -652,7 +738,7 @@ __global__ __launch_bounds__(THREADS) void gemm_tc_persistent_kernel(
   using Config = PersistentConfig;
   constexpr int STAGES = Config::kStages;
   // features of the output per tile, and where the second half of the N operand comes from
-  constexpr int FEATURES = EPI == EPI_SWIGLU ? BM : 2 * BM;
+  constexpr int FEATURES = EPI == EPI_SWIGLU || EPI == EPI_BLOCK_GATES ? BM : 2 * BM;
 
   hx_pdl_trigger();
   extern __shared__ uint8_t smem_raw[];
@@ -700,8 +786,15 @@ __global__ __launch_bounds__(THREADS) void gemm_tc_persistent_kernel(
           if (group < 0) kb_end = unit.kb_begin;
           else group_row0 = group * args.group_rows;
         }
-        const int feature0 = group_row0 + unit.feature_tile * FEATURES;
-        const int second_half = EPI == EPI_SWIGLU ? args.up_row_offset + feature0 : feature0 + BM;
+        int feature0 = group_row0 + unit.feature_tile * FEATURES;
+        int second_half = EPI == EPI_SWIGLU ? args.up_row_offset + feature0 : feature0 + BM;
+        int k0 = 0;      // first column of the token rows
+        if (EPI == EPI_BLOCK_GATES) {
+          const int block = unit.feature_tile / args.gates.tiles;
+          feature0 = block * 2 * args.gates.size + (unit.feature_tile - block * args.gates.tiles) * BM;
+          second_half = feature0 + args.gates.size;
+          k0 = block * args.gates.size;
+        }
         const int token0 = unit.token_tile * BM;
         for (int kb = unit.kb_begin; kb < kb_end; ++kb, ++fill) {
           const int s = fill % STAGES;
@@ -713,7 +806,7 @@ __global__ __launch_bounds__(THREADS) void gemm_tc_persistent_kernel(
           }
           uint8_t* stage = smem + s * Config::kStageBytes;
           mbar_expect_tx(&full_bar[s], Config::kStageBytes);
-          const int k = kb * BK;
+          const int k = k0 + kb * BK;
           tma_load_2d(stage, &map_x, &full_bar[s], k, token0);
           load_weight_box(stage + Config::kBytesA, &map_w, &full_bar[s], feature0, kb, args.k_tiles);
           load_weight_box(stage + Config::kBytesA + BM * BK * 2, &map_w, &full_bar[s], second_half,
@@ -804,6 +897,11 @@ __global__ __launch_bounds__(THREADS) void gemm_tc_persistent_kernel(
       if constexpr (EPI == EPI_ROPE_APPEND) {
         write_row_rope(args, lane_base + buffer * Config::kBufferColumns,
                        unit.token_tile * BM + quarter * 32 + lane, unit.feature_tile * FEATURES);
+      } else if constexpr (EPI == EPI_BLOCK_GATES) {
+        const int block = unit.feature_tile / args.gates.tiles;
+        write_row_gates(args.gates, lane_base + buffer * Config::kBufferColumns,
+                        unit.token_tile * BM + quarter * 32 + lane, args.tokens, block,
+                        (unit.feature_tile - block * args.gates.tiles) * BM);
       } else if (EPI == EPI_ADD_F32 && unit.partial) {
         add_row_atomically(static_cast<float*>(args.out), args.ldo, args.features,
                            lane_base + buffer * Config::kBufferColumns,
@@ -814,7 +912,7 @@ __global__ __launch_bounds__(THREADS) void gemm_tc_persistent_kernel(
                        lane_base + buffer * Config::kBufferColumns,
                        unit.token_tile * BM + quarter * 32 + lane, args.tokens,
                        unit.feature_tile * FEATURES, args.activation, args.gate_limit,
-                       args.gate_bias, args.up_bias);
+                       args.gate_bias, args.up_bias, args.softcap);
       }
       // every lane's tcgen05.ld has completed (the loads are waited for where they are
       // issued): hand the accumulator back
@@ -972,7 +1070,9 @@ int launch_persistent(const CUtensorMap& map_w, const CUtensorMap& map_x, Persis
     configured = true;
   }
   constexpr int kFeatures = EPI == EPI_SWIGLU ? BM : 2 * BM;
-  const int feature_tiles = (args.features + kFeatures - 1) / kFeatures;
+  const int feature_tiles = EPI == EPI_BLOCK_GATES
+                                ? args.gates.channels / args.gates.size * args.gates.tiles
+                                : (args.features + kFeatures - 1) / kFeatures;
   args.token_tiles = (args.tokens + BM - 1) / BM;
   const long long tiles = static_cast<long long>(args.token_tiles) * feature_tiles;
   HX_REQUIRE(tiles < (1ll << 30), "hx_gemm_tc: too many tiles");
@@ -1005,6 +1105,7 @@ int launch_persistent_epilogue(int epilogue, const CUtensorMap& map_w, const CUt
     case EPI_ADD_F32: return launch_persistent<EPI_ADD_F32>(map_w, map_x, args, stream);
     case EPI_SWIGLU: return launch_persistent<EPI_SWIGLU>(map_w, map_x, args, stream);
     case EPI_ROPE_APPEND: return launch_persistent<EPI_ROPE_APPEND>(map_w, map_x, args, stream);
+    case EPI_BLOCK_GATES: return launch_persistent<EPI_BLOCK_GATES>(map_w, map_x, args, stream);
     default:
       hx_set_error("hx_gemm_tc: unknown epilogue %d", epilogue);
       return HX_ERR_ARGUMENT;
@@ -1041,8 +1142,10 @@ static int gemm_tc(const void* x, int ldx, int x_capacity_rows, const void* w, i
                    int weight_rows, void* out, int ldo, int tokens, int features, int depth,
                    int epilogue, int activation, float gate_limit, const float* gate_bias,
                    const float* up_bias, int up_row_offset, int k_splits, int weight_tiles,
-                   int* status, cudaStream_t stream) {
+                   int* status, cudaStream_t stream, float softcap = 0.0f) {
   if (weight_tiles) ldw = 8;      // not a stride of anything here
+  HX_REQUIRE(softcap >= 0.0f && (softcap == 0.0f || epilogue == EPI_STORE_F32),
+             "hx_gemm_tc: a softcap belongs to a float32 store");
   HX_REQUIRE(!weight_tiles || epilogue != EPI_SWIGLU || up_row_offset % BM == 0,
              "hx_gemm_tc: with tiled weights the up rows must start on a multiple of %d", BM);
   HX_REQUIRE(hx_gemm_tc_supports(tokens, features, depth, ldx, ldw),
@@ -1084,7 +1187,7 @@ static int gemm_tc(const void* x, int ldx, int x_capacity_rows, const void* w, i
   if (persistent) {
     PersistentArgs args{out, ldo, tokens, features, depth, up_row_offset, k_tiles, 0, 0,
                         total_k_blocks, status, RopeArgs{}, -1, activation, nullptr, 0,
-                        gate_limit, gate_bias, up_bias};
+                        gate_limit, gate_bias, up_bias, softcap};
     rc = launch_persistent_epilogue(epilogue, map_w, map_x, args, stream);
     if (rc != HX_OK) return rc;
     HX_CHECK_LAUNCH("hx_gemm_tc");
@@ -1094,7 +1197,7 @@ static int gemm_tc(const void* x, int ldx, int x_capacity_rows, const void* w, i
   const int per_split = (total_k_blocks + k_splits - 1) / k_splits;
   k_splits = (total_k_blocks + per_split - 1) / per_split;
   GemmArgs args{out, ldo, tokens, features, depth, up_row_offset, per_split, k_tiles, status,
-                activation, nullptr, 0, gate_limit, gate_bias, up_bias};
+                activation, nullptr, 0, gate_limit, gate_bias, up_bias, softcap};
   const dim3 grid((tokens + bn - 1) / bn, (features + BM - 1) / BM, k_splits);
   HX_REQUIRE(grid.y <= 65535, "hx_gemm_tc: too many features (%d)", features);
 
@@ -1123,6 +1226,16 @@ HX_API int hx_gemm_tc(const void* x, int ldx, int x_capacity_rows, const void* w
   return gemm_tc(x, ldx, x_capacity_rows, w, ldw, weight_rows, out, ldo, tokens, features, depth,
                  epilogue, activation, 0.0f, nullptr, nullptr, up_row_offset, k_splits,
                  weight_tiles, status, stream);
+}
+
+// The product with a float32 store whose sums run into a level: out = cap * tanh(x w^T / cap).
+HX_API int hx_gemm_tc_softcapped(const void* x, int ldx, int x_capacity_rows, const void* w,
+                                 int ldw, int weight_rows, float* out, int ldo, int tokens,
+                                 int features, int depth, float softcap, int weight_tiles,
+                                 int* status, cudaStream_t stream) {
+  return gemm_tc(x, ldx, x_capacity_rows, w, ldw, weight_rows, out, ldo, tokens, features, depth,
+                 EPI_STORE_F32, HX_GATE_SILU, 0.0f, nullptr, nullptr, 0, 1, weight_tiles, status,
+                 stream, softcap);
 }
 
 // The product with the gated epilogue for every HxGateActivation and with float32 biases on
@@ -1247,22 +1360,24 @@ HX_API int hx_gemm_tc_rope_append_min_tokens() { return 65; }
 // `positions` on mean what they mean to hx_rope_append, with adjacent pairs; x, w, ldx, ldw,
 // x_capacity_rows, weight_rows and weight_tiles what they mean to hx_gemm_tc.  Needs more
 // than 64 tokens, bfloat16, head_dim a multiple of 16 and 16-byte aligned out and caches.
-HX_API int hx_gemm_tc_rope_append(const void* x, int ldx, int x_capacity_rows, const void* w,
+// shared_values != 0: w = [q heads | k heads], and the keys before the rotation are the values.
+HX_API int hx_gemm_tc_rope_append_shared(const void* x, int ldx, int x_capacity_rows, const void* w,
                                   int ldw, int weight_rows, void* out, int ldo, int tokens,
                                   int depth, int weight_tiles, const int* positions,
                                   const int* token_request, const int* request_table_row,
                                   const int* block_tables, int table_stride, void* k_cache,
                                   void* v_cache, const float* cos_table, const float* sin_table,
                                   int table_positions, int heads, int kv_heads, int head_dim,
-                                  int rotary_dim, int page_size, int num_pages, int* status,
-                                  cudaStream_t stream) {
+                                  int rotary_dim, int page_size, int num_pages, int shared_values,
+                                  int* status, cudaStream_t stream) {
+  const int row_heads = heads + (shared_values ? 1 : 2) * kv_heads;
   if (weight_tiles) ldw = 8;      // not a stride of anything here
   HX_REQUIRE(heads > 0 && kv_heads > 0 && head_dim > 0 && head_dim % 16 == 0,
              "hx_gemm_tc_rope_append: head_dim %d must be a multiple of 16", head_dim);
-  HX_REQUIRE(static_cast<long long>(heads + 2 * kv_heads) * head_dim <= weight_rows,
-             "hx_gemm_tc_rope_append: %d + 2 x %d heads of %d exceed the %d weight rows", heads,
-             kv_heads, head_dim, weight_rows);
-  const int features = (heads + 2 * kv_heads) * head_dim;
+  HX_REQUIRE(static_cast<long long>(row_heads) * head_dim <= weight_rows,
+             "hx_gemm_tc_rope_append: %d heads of %d exceed the %d weight rows", row_heads, head_dim,
+             weight_rows);
+  const int features = row_heads * head_dim;
   HX_REQUIRE(tokens >= hx_gemm_tc_rope_append_min_tokens(),
              "hx_gemm_tc_rope_append: %d tokens; it takes prompt portions of at least %d", tokens,
              hx_gemm_tc_rope_append_min_tokens());
@@ -1308,10 +1423,59 @@ HX_API int hx_gemm_tc_rope_append(const void* x, int ldx, int x_capacity_rows, c
                                table_stride, static_cast<__nv_bfloat16*>(k_cache),
                                static_cast<__nv_bfloat16*>(v_cache), cos_table, sin_table,
                                table_positions, heads, kv_heads, head_dim, rotary_dim, page_size,
-                               num_pages}};
+                               num_pages, shared_values}};
   rc = launch_persistent_epilogue(EPI_ROPE_APPEND, map_w, map_x, args, stream);
   if (rc != HX_OK) return rc;
   HX_CHECK_LAUNCH("hx_gemm_tc_rope_append");
+  return HX_OK;
+}
+
+HX_API int hx_gemm_tc_rope_append(const void* x, int ldx, int x_capacity_rows, const void* w,
+                                  int ldw, int weight_rows, void* out, int ldo, int tokens,
+                                  int depth, int weight_tiles, const int* positions,
+                                  const int* token_request, const int* request_table_row,
+                                  const int* block_tables, int table_stride, void* k_cache,
+                                  void* v_cache, const float* cos_table, const float* sin_table,
+                                  int table_positions, int heads, int kv_heads, int head_dim,
+                                  int rotary_dim, int page_size, int num_pages, int* status,
+                                  cudaStream_t stream) {
+  return hx_gemm_tc_rope_append_shared(x, ldx, x_capacity_rows, w, ldw, weight_rows, out, ldo,
+                                       tokens, depth, weight_tiles, positions, token_request,
+                                       request_table_row, block_tables, table_stride, k_cache,
+                                       v_cache, cos_table, sin_table, table_positions, heads,
+                                       kv_heads, head_dim, rotary_dim, page_size, num_pages, 0,
+                                       status, stream);
+}
+
+// hx_block_gates (see hx_gated_recurrence.cu) on the tensor cores: bfloat16, blocks of a multiple of
+// 8 channels, rows of u [u_capacity_rows][ld_u] with ld_u a multiple of 8.
+HX_API int hx_gemm_tc_block_gates(const void* u, int ld_u, int u_capacity_rows, const void* w,
+                                  const float* r_bias, const float* i_bias, const float* rate,
+                                  float* decay, float* push, int tokens, int blocks, int size,
+                                  int* status, cudaStream_t stream) {
+  HX_REQUIRE(tokens >= 0 && blocks > 0 && size > 0 && size % 8 == 0,
+             "hx_gemm_tc_block_gates: blocks of %d channels are not supported (multiples of 8)", size);
+  HX_REQUIRE(ld_u >= blocks * size && ld_u % 8 == 0 && (reinterpret_cast<uintptr_t>(u) & 15) == 0 &&
+                 (reinterpret_cast<uintptr_t>(w) & 15) == 0 &&
+                 (reinterpret_cast<uintptr_t>(decay) & 15) == 0 &&
+                 (reinterpret_cast<uintptr_t>(push) & 15) == 0,
+             "hx_gemm_tc_block_gates: operands must be 16-byte aligned");
+  HX_REQUIRE(u_capacity_rows >= tokens, "hx_gemm_tc_block_gates: buffer rows %d < tokens %d",
+             u_capacity_rows, tokens);
+  HX_REQUIRE(r_bias && i_bias && rate && status, "hx_gemm_tc_block_gates: an operand is missing");
+  if (tokens == 0) return HX_OK;
+  CUtensorMap map_w, map_x;
+  int rc = get_tensor_map(w, static_cast<uint64_t>(blocks) * 2 * size, size, size, BM, &map_w);
+  if (rc != HX_OK) return rc;
+  rc = get_tensor_map(u, u_capacity_rows, static_cast<uint64_t>(blocks) * size, ld_u, BM, &map_x);
+  if (rc != HX_OK) return rc;
+  PersistentArgs args{nullptr, 0, tokens, 2 * blocks * size, size, 0, 0, 0, 0,
+                      (size + BK - 1) / BK, status, RopeArgs{}, -1, HX_GATE_SILU, nullptr, 0};
+  args.gates = BlockGateArgs{static_cast<const __nv_bfloat16*>(u), ld_u, r_bias, i_bias, rate, decay,
+                             push, size, blocks * size, (size + BM - 1) / BM};
+  rc = launch_persistent_epilogue(EPI_BLOCK_GATES, map_w, map_x, args, stream);
+  if (rc != HX_OK) return rc;
+  HX_CHECK_LAUNCH("hx_gemm_tc_block_gates");
   return HX_OK;
 }
 

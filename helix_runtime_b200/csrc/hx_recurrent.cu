@@ -74,7 +74,21 @@ struct FilterArgs {
   const int* token_request;
   const int* request_slot;
   const int* request_start;
+  // Optional.  in_bias [channels]: added to every input before the filter (inputs in front of the
+  // sequence stay zero).  accum [tokens, ld_accum], already offset: the inputs are these float32
+  // sums, rounded as the projection's own store rounds them, instead of `raw`.
+  const float* in_bias = nullptr;
+  const float* accum = nullptr;
+  int ld_accum = 0;
 };
+
+template <typename T>
+__device__ __forceinline__ float filter_input(const FilterArgs<T>& a, int token, int c, float in_bias) {
+  const float x = a.accum != nullptr
+                      ? hx_to_float<T>(hx_from_float<T>(a.accum[static_cast<size_t>(token) * a.ld_accum + c]))
+                      : hx_to_float<T>(a.raw[static_cast<size_t>(token) * a.ld_raw + c]);
+  return x + in_bias;
+}
 
 __device__ __forceinline__ float filter_finish(float y, int silu) {
   return silu ? hx_silu(y) : y;
@@ -96,10 +110,11 @@ __global__ __launch_bounds__(256) void causal_filter_kernel(const FilterArgs<T> 
   const int reach = a.taps - 1;
   const float* w = a.taps_weight + static_cast<size_t>(c) * a.taps;
   const float b = a.bias != nullptr ? a.bias[c] : 0.0f;
+  const float in_bias = a.in_bias != nullptr ? a.in_bias[c] : 0.0f;
   if (index >= reach) {
     float y = b;
     for (int j = 0; j < a.taps; ++j)
-      y = fmaf(w[j], hx_to_float<T>(a.raw[static_cast<size_t>(token - reach + j) * a.ld_raw + c]), y);
+      y = fmaf(w[j], filter_input(a, token - reach + j, c, in_bias), y);
     a.out[static_cast<size_t>(token) * a.ld_out + c] = hx_from_float<T>(filter_finish(y, a.silu));
     return;
   }
@@ -112,7 +127,7 @@ __global__ __launch_bounds__(256) void causal_filter_kernel(const FilterArgs<T> 
     for (int j = 0; j < a.taps; ++j) {
       const int place = i - reach + j;       // relative to the portion's start
       const float u = place >= 0
-                          ? hx_to_float<T>(a.raw[static_cast<size_t>(start + place) * a.ld_raw + c])
+                          ? filter_input(a, start + place, c, in_bias)
                           : state[static_cast<size_t>(place + reach) * a.channels];
       y = fmaf(w[j], u, y);
     }
@@ -123,9 +138,172 @@ __global__ __launch_bounds__(256) void causal_filter_kernel(const FilterArgs<T> 
   for (int r = 0; r < reach; ++r) {
     const int place = count - reach + r;
     state[static_cast<size_t>(r) * a.channels] =
-        place >= 0 ? hx_to_float<T>(a.raw[static_cast<size_t>(start + place) * a.ld_raw + c])
+        place >= 0 ? filter_input(a, start + place, c, in_bias)
                    : state[static_cast<size_t>(place + reach) * a.channels];
   }
+}
+
+// The same for bfloat16 rows made of whole 16-byte pieces and up to FILTER_FAST_TAPS taps: a
+// thread takes one piece (8 channels) of `run` consecutive tokens of the batch, fetches the
+// filter's weights once and keeps a row of inputs for the tokens behind it.
+constexpr int FILTER_FAST_TAPS = 4;
+
+__device__ __forceinline__ void filter_input8(const FilterArgs<__nv_bfloat16>& a, int token, int c,
+                                              const float (&in_bias)[8], float (&x)[8]) {
+  if (a.accum != nullptr) {
+    const float4* source =
+        reinterpret_cast<const float4*>(a.accum + static_cast<size_t>(token) * a.ld_accum + c);
+    const float4 lo = source[0], hi = source[1];
+    const float raw[8] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
+#pragma unroll
+    for (int i = 0; i < 8; ++i) x[i] = __bfloat162float(__float2bfloat16_rn(raw[i])) + in_bias[i];
+    return;
+  }
+  const uint4 packed = *reinterpret_cast<const uint4*>(a.raw + static_cast<size_t>(token) * a.ld_raw + c);
+  const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&packed);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 v = __bfloat1622float2(pairs[i]);
+    x[2 * i] = v.x + in_bias[2 * i];
+    x[2 * i + 1] = v.y + in_bias[2 * i + 1];
+  }
+}
+
+template <int TAPS>
+__global__ __launch_bounds__(256) void causal_filter_pieces_kernel(const FilterArgs<__nv_bfloat16> a,
+                                                                   int tokens, int run) {
+  constexpr int REACH = TAPS - 1;
+  hx_pdl_trigger();
+  const int first = blockIdx.x * run;
+  const int last = min(first + run, tokens);      // exclusive
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
+  if (c >= a.channels) {
+    hx_pdl_wait();      // a grid must not be seen complete before its predecessor is
+    return;
+  }
+  // weights, biases and the step's own description do not depend on the kernel before
+  float w[TAPS][8], b[8], in_bias[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j][i] = a.taps_weight[static_cast<size_t>(c + i) * TAPS + j];
+    b[i] = a.bias != nullptr ? a.bias[c + i] : 0.0f;
+    in_bias[i] = a.in_bias != nullptr ? a.in_bias[c + i] : 0.0f;
+  }
+  int request = a.token_request[first];
+  int start = a.request_start[request];
+  int end = a.request_start[request + 1];
+  int slot = a.request_slot[request];
+  hx_pdl_wait();
+
+  auto emit = [&](int token, const float (&y)[8]) {
+    uint4 packed;
+    __nv_bfloat162* pairs = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      pairs[i] = __floats2bfloat162_rn(filter_finish(y[2 * i], a.silu), filter_finish(y[2 * i + 1], a.silu));
+    *reinterpret_cast<uint4*>(a.out + static_cast<size_t>(token) * a.ld_out + c) = packed;
+  };
+  // rows[j]: the inputs of batch row token - REACH + j, used only by tokens that lie at least
+  // REACH tokens into their portion (rows of another request are never used: not fetched)
+  float rows[TAPS][8];
+#pragma unroll
+  for (int j = 0; j < REACH; ++j) {
+    if (first - REACH + j >= start) {
+      filter_input8(a, first - REACH + j, c, in_bias, rows[j]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) rows[j][i] = 0.0f;
+    }
+  }
+  for (int token = first; token < last; ++token) {
+    filter_input8(a, token, c, in_bias, rows[REACH]);
+    if (token >= end) {
+      request = a.token_request[token];
+      start = a.request_start[request];
+      end = a.request_start[request + 1];
+      slot = a.request_slot[request];
+    }
+    const int index = token - start;
+    if (index >= REACH) {
+      float y[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        y[i] = b[i];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) y[i] = fmaf(w[j][i], rows[j][i], y[i]);
+      }
+      emit(token, y);
+    } else if (index == 0) {
+      // the portion's first token: the tokens whose filter reaches behind the portion, then
+      // the new state (see the scalar kernel)
+      const int count = end - start;
+      float* state = a.state + static_cast<size_t>(slot) * a.state_stride + c;
+      const int behind = count < REACH ? count : REACH;
+      for (int t = 0; t < behind; ++t) {
+        float y[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) y[i] = b[i];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+          const int place = t - REACH + j;
+          float x[8];
+          if (place >= 0) {
+            filter_input8(a, start + place, c, in_bias, x);
+          } else {
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+              x[i] = state[static_cast<size_t>(place + REACH) * a.channels + i];
+          }
+#pragma unroll
+          for (int i = 0; i < 8; ++i) y[i] = fmaf(w[j][i], x[i], y[i]);
+        }
+        emit(start + t, y);
+      }
+      for (int r = 0; r < REACH; ++r) {
+        const int place = count - REACH + r;
+        float x[8];
+        if (place >= 0) {
+          filter_input8(a, start + place, c, in_bias, x);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 8; ++i) x[i] = state[static_cast<size_t>(place + REACH) * a.channels + i];
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) state[static_cast<size_t>(r) * a.channels + i] = x[i];
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < REACH; ++j)
+#pragma unroll
+      for (int i = 0; i < 8; ++i) rows[j][i] = rows[j + 1][i];
+  }
+}
+
+bool filter_pieces_apply(const FilterArgs<__nv_bfloat16>& a) {
+  auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  return a.taps <= FILTER_FAST_TAPS && a.channels % 8 == 0 && a.ld_out % 8 == 0 && aligned(a.out) &&
+         (a.accum != nullptr ? a.ld_accum % 4 == 0 && aligned(a.accum)
+                             : a.ld_raw % 8 == 0 && aligned(a.raw));
+}
+
+int launch_filter(const FilterArgs<__nv_bfloat16>& a, int tokens, cudaStream_t stream) {
+  if (!filter_pieces_apply(a)) {
+    hx_launch(causal_filter_kernel<__nv_bfloat16>, dim3(tokens, (a.channels + 255) / 256), 256, 0,
+              stream, a);
+    return HX_OK;
+  }
+  const int run = tokens >= 1024 ? 8 : (tokens >= 256 ? 2 : 1);
+  const int pieces = a.channels / 8;
+  const int block = pieces >= 256 ? 256 : ((pieces + 31) / 32) * 32;
+  const dim3 grid((tokens + run - 1) / run, (pieces + block - 1) / block);
+  switch (a.taps) {
+    case 1: hx_launch(causal_filter_pieces_kernel<1>, grid, block, 0, stream, a, tokens, run); break;
+    case 2: hx_launch(causal_filter_pieces_kernel<2>, grid, block, 0, stream, a, tokens, run); break;
+    case 3: hx_launch(causal_filter_pieces_kernel<3>, grid, block, 0, stream, a, tokens, run); break;
+    default: hx_launch(causal_filter_pieces_kernel<4>, grid, block, 0, stream, a, tokens, run); break;
+  }
+  return HX_OK;
 }
 
 // ------------------------------------------------------------ state-space recurrence
@@ -801,31 +979,46 @@ int tile_for(int floats_per_token) {
 // Floats a head's matrix of `rows` x `columns` takes in a request's state row.
 HX_API int hx_scan_state_floats(int columns, int rows) { return state_floats(columns, rows); }
 
-HX_API int hx_causal_filter(const void* raw, int ld_raw, void* out, int ld_out, int dtype,
-                            const float* taps_weight, const float* bias, float* state,
-                            long long state_stride, int taps, int channels, int silu, int tokens,
-                            const int* token_request, const int* request_slot,
-                            const int* request_start, cudaStream_t stream) {
+// ... with an optional bias on the inputs and with inputs that may lie in float32 sums (see
+// FilterArgs): raw or accum is given, the other null.
+HX_API int hx_causal_filter_biased(const void* raw, int ld_raw, const float* accum, int ld_accum,
+                                   const float* in_bias, void* out, int ld_out, int dtype,
+                                   const float* taps_weight, const float* bias, float* state,
+                                   long long state_stride, int taps, int channels, int silu,
+                                   int tokens, const int* token_request, const int* request_slot,
+                                   const int* request_start, cudaStream_t stream) {
+  HX_REQUIRE((raw != nullptr) != (accum != nullptr),
+             "hx_causal_filter: give the projected rows or their sums");
+  HX_REQUIRE((channels + 255) / 256 <= 65535, "hx_causal_filter: rows too wide");
   HX_REQUIRE(tokens >= 0 && channels > 0 && taps >= 1, "hx_causal_filter: bad sizes");
   HX_REQUIRE(taps == 1 || state != nullptr, "hx_causal_filter: a filter of %d taps needs state", taps);
   if (tokens == 0) return HX_OK;
-  const dim3 grid(tokens, (channels + 255) / 256);
   if (dtype == HX_F32) {
     FilterArgs<float> a{static_cast<const float*>(raw), ld_raw, static_cast<float*>(out), ld_out,
                         taps_weight, bias, state, state_stride, taps, channels, silu,
-                        token_request, request_slot, request_start};
-    hx_launch(causal_filter_kernel<float>, grid, 256, 0, stream, a);
+                        token_request, request_slot, request_start, in_bias, accum, ld_accum};
+    hx_launch(causal_filter_kernel<float>, dim3(tokens, (channels + 255) / 256), 256, 0, stream, a);
   } else if (dtype == HX_BF16) {
     FilterArgs<__nv_bfloat16> a{static_cast<const __nv_bfloat16*>(raw), ld_raw,
                                 static_cast<__nv_bfloat16*>(out), ld_out, taps_weight, bias, state,
                                 state_stride, taps, channels, silu, token_request, request_slot,
-                                request_start};
-    hx_launch(causal_filter_kernel<__nv_bfloat16>, grid, 256, 0, stream, a);
+                                request_start, in_bias, accum, ld_accum};
+    launch_filter(a, tokens, stream);
   } else {
     HX_REQUIRE(false, "hx_causal_filter: unknown dtype %d", dtype);
   }
   HX_CHECK_LAUNCH("hx_causal_filter");
   return HX_OK;
+}
+
+HX_API int hx_causal_filter(const void* raw, int ld_raw, void* out, int ld_out, int dtype,
+                            const float* taps_weight, const float* bias, float* state,
+                            long long state_stride, int taps, int channels, int silu, int tokens,
+                            const int* token_request, const int* request_slot,
+                            const int* request_start, cudaStream_t stream) {
+  return hx_causal_filter_biased(raw, ld_raw, nullptr, 0, nullptr, out, ld_out, dtype, taps_weight,
+                                 bias, state, state_stride, taps, channels, silu, tokens,
+                                 token_request, request_slot, request_start, stream);
 }
 
 HX_API int hx_state_space_scan(const void* x, const void* b, const void* c, int ld, const void* dt,

@@ -199,10 +199,10 @@ class Engine:
         device = require_cuda(model.device)
         kv_needs, state_needs = model.cache_needs()
         # the most positions a request holds pages for at once: all of them in a layer that
-        # keeps every key; in a windowed layer the window, its kept first keys, the portion
-        # a step feeds and the page being filled
-        held = max((model.max_positions if need.window is None else
-                    min(model.max_positions, need.window + need.keep_first
+        # keeps every key; in a windowed or chunked layer the window or chunk, its kept first
+        # keys, the portion a step feeds and the page being filled
+        held = max((model.max_positions if need.reach is None else
+                    min(model.max_positions, need.reach + need.keep_first
                         + config.max_tokens_per_iteration + 2 * config.page_size)
                     for need in kv_needs.values()), default=model.max_positions)
         pages_per_request = -(-held // config.page_size)
@@ -215,8 +215,8 @@ class Engine:
             page_bytes = fixed_bytes = 0
             for need in kv_needs.values():
                 layer_page = 2 * need.kv_heads * need.head_dim * element * config.page_size
-                if need.window is not None and need.window in fixed:
-                    fixed_bytes += layer_page * fixed[need.window]
+                if need.bounded and need.reach in fixed:
+                    fixed_bytes += layer_page * fixed[need.reach]
                 else:
                     page_bytes += layer_page
             free_bytes, _ = torch.cuda.mem_get_info(device)

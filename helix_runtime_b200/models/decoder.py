@@ -231,6 +231,7 @@ class DecoderModel:
             view.page_size = group.page_size
             view.num_pages = group.pool.num_pages
             view.window = group.need.window
+            view.chunk = group.need.chunk
         if owner in cache.states:
             view.state = cache.state(owner)
         return view

@@ -80,6 +80,12 @@ def _declare(library: ctypes.CDLL) -> None:
         _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int,
         _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
         _c_ptr, _c_ptr, _c_int, _c_ptr]
+    library.hx_rope_append_shared.argtypes = [*library.hx_rope_append.argtypes[:-1], _c_int, _c_ptr]
+    library.hx_gemm_simt_softcapped.argtypes = [_c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int,
+                                                _c_int, _c_int, _c_int, _c_int, _c_float, _c_ptr]
+    library.hx_gemm_tc_softcapped.argtypes = [_c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr,
+                                              _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_ptr,
+                                              _c_ptr]
     library.hx_gemm_simt.argtypes = [_c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_int,
                                      _c_int, _c_int, _c_int, _c_ptr]
     library.hx_gemm_tc.argtypes = [_c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int,
@@ -94,6 +100,8 @@ def _declare(library: ctypes.CDLL) -> None:
         _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int,
         _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr]
     library.hx_gemm_tc_rope_append.restype = _c_int
+    library.hx_gemm_tc_rope_append_shared.argtypes = [
+        *library.hx_gemm_tc_rope_append.argtypes[:-2], _c_int, _c_ptr, _c_ptr]
     library.hx_gemm_tc_rope_append_min_tokens.argtypes = []
     library.hx_gemm_tc_rope_append_min_tokens.restype = _c_int
     library.hx_gemm_tc_supports.argtypes = [_c_int] * 5
@@ -150,6 +158,25 @@ def _declare(library: ctypes.CDLL) -> None:
     library.hx_causal_filter.argtypes = [_c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr,
                                          _c_ptr, _c_longlong, _c_int, _c_int, _c_int, _c_int, _c_ptr,
                                          _c_ptr, _c_ptr, _c_ptr]
+    library.hx_causal_filter_biased.argtypes = [
+        _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr,
+        _c_longlong, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr]
+    library.hx_block_gates.argtypes = [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
+                                       _c_int, _c_int, _c_int, _c_int, _c_ptr]
+    library.hx_gemm_tc_block_gates.argtypes = [_c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
+                                               _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr]
+    library.hx_gated_scan.argtypes = [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr,
+                                      _c_longlong, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr,
+                                      _c_int, _c_ptr]
+    library.hx_gated_recurrence_supports.argtypes = [_c_int]
+    library.hx_gated_recurrence_step.argtypes = [
+        _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr,
+        _c_ptr, _c_longlong, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr]
+    for name in ("hx_rope_append_shared", "hx_gemm_simt_softcapped", "hx_gemm_tc_softcapped",
+                 "hx_gemm_tc_rope_append_shared", "hx_causal_filter_biased", "hx_block_gates",
+                 "hx_gemm_tc_block_gates", "hx_gated_scan", "hx_gated_recurrence_supports",
+                 "hx_gated_recurrence_step"):
+        getattr(library, name).restype = _c_int
     library.hx_scan_state_floats.argtypes = [_c_int, _c_int]
     library.hx_scan_state_floats.restype = _c_int
     library.hx_state_space_scan.argtypes = [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_int,
@@ -221,11 +248,13 @@ def _declare(library: ctypes.CDLL) -> None:
     library.hx_paged_attention_biased.argtypes = [
         _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr,
         _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-        _c_int, _c_int, _c_float, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr]
+        _c_int, _c_int, _c_float, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_float, _c_ptr, _c_ptr]
     library.hx_prefill_attention_biased.argtypes = [
-        *library.hx_prefill_attention_windowed.argtypes[:-2], _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr]
+        *library.hx_prefill_attention_windowed.argtypes[:-2], _c_int, _c_ptr, _c_ptr, _c_int,
+        _c_float, _c_ptr, _c_ptr]
     library.hx_prefill_attention_tc_biased.argtypes = [
-        *library.hx_prefill_attention_windowed.argtypes[:-2], _c_ptr, _c_ptr, _c_ptr, _c_ptr]
+        *library.hx_prefill_attention_windowed.argtypes[:-2], _c_ptr, _c_ptr, _c_int, _c_float,
+        _c_ptr, _c_ptr]
     library.hx_prefill_attention_tc_biased.restype = _c_int
     library.hx_norm_residual_add.argtypes = [_c_ptr, _c_ptr, _c_ptr, _c_float, _c_float, _c_ptr,
                                              _c_int, _c_int, _c_int, _c_int, _c_ptr]
@@ -467,31 +496,34 @@ def rope_append(qkv: torch.Tensor, positions: torch.Tensor, token_request: torch
                 cos_table: torch.Tensor, sin_table: torch.Tensor, tokens: int, heads: int,
                 kv_heads: int, head_dim: int, rotary_dim: int, pairing: int, page_size: int,
                 num_pages: int, status: torch.Tensor,
-                accum: Optional[torch.Tensor] = None) -> None:
+                accum: Optional[torch.Tensor] = None, shared_values: bool = False) -> None:
     """Rotate q and k of ``qkv[:tokens]`` in place and write k, v into their pages.  With
     ``accum`` (float32 ``[rows, width]``) the projection is read from there instead, rounded
-    to the storage type, and ``accum`` is cleared."""
+    to the storage type, and ``accum`` is cleared.  ``shared_values``: the rows hold no values,
+    a key as projected (before the rotation) is its value."""
     write = k_cache is not None
-    _check(lib().hx_rope_append(
+    _check(lib().hx_rope_append_shared(
         qkv.data_ptr(), dtype_code(qkv.dtype), qkv.stride(0), positions.data_ptr(),
         token_request.data_ptr(), request_table_row.data_ptr(), block_tables.data_ptr(),
         block_tables.stride(0), _ptr(k_cache), _ptr(v_cache), 1 if write else 0,
         cos_table.data_ptr(), sin_table.data_ptr(), cos_table.shape[0], tokens, heads, kv_heads,
         head_dim, rotary_dim, pairing, page_size, num_pages, _ptr(status), _ptr(accum),
-        0 if accum is None else accum.stride(0), _stream()))
+        0 if accum is None else accum.stride(0), 1 if shared_values else 0, _stream()))
 
 
 def gemm_tc_supports(tokens: int, features: int, depth: int, ldx: int, ldw: int) -> bool:
     return bool(lib().hx_gemm_tc_supports(tokens, features, depth, ldx, ldw))
 
 
-def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tokens: int, epilogue: int) -> None:
-    """out[:tokens] (op)= x[:tokens] @ w.T on the CUDA cores (float32 or bfloat16 storage)."""
+def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tokens: int, epilogue: int,
+              softcap: float = 0.0) -> None:
+    """out[:tokens] (op)= x[:tokens] @ w.T on the CUDA cores (float32 or bfloat16 storage);
+    ``softcap`` > 0 with ``EPI_STORE_F32``: softcap * tanh(product / softcap) is stored."""
     assert x.dtype == w.dtype and x.stride(-1) == 1 and w.stride(-1) == 1 and out.stride(-1) == 1
     features, depth = w.shape
-    _check(lib().hx_gemm_simt(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(),
-                              out.stride(0), dtype_code(x.dtype), tokens, features, depth, epilogue,
-                              _stream()))
+    _check(lib().hx_gemm_simt_softcapped(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0),
+                                         out.data_ptr(), out.stride(0), dtype_code(x.dtype), tokens,
+                                         features, depth, epilogue, float(softcap), _stream()))
 
 
 WEIGHT_TILE_ROWS, WEIGHT_TILE_DEPTH = 128, 64
@@ -514,12 +546,13 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tokens: int, fe
             epilogue: int, status: torch.Tensor, up_row_offset: int = 0, k_splits: int = 1,
             weight_shape: Optional[Tuple[int, int]] = None, gate_activation: Optional[int] = None,
             gate_limit: float = 0.0, gate_bias: Optional[torch.Tensor] = None,
-            up_bias: Optional[torch.Tensor] = None) -> None:
+            up_bias: Optional[torch.Tensor] = None, softcap: float = 0.0) -> None:
     """out[:tokens, :features] (op)= x[:tokens] @ w.T on the tensor cores (bfloat16).  ``w``
     is the matrix ``[rows, depth]`` or its tiles from :func:`tile_weights` (then
     ``weight_shape`` gives rows and depth).  With ``gate_activation`` (any of GATE_ACTIVATIONS)
     the epilogue is that gated activation of ``[gate; up]`` whatever ``epilogue`` says, with the
-    optional float32 biases ``gate_bias`` and ``up_bias`` ``[features]`` added first."""
+    optional float32 biases ``gate_bias`` and ``up_bias`` ``[features]`` added first.
+    ``softcap`` > 0 with ``EPI_STORE_F32``: softcap * tanh(product / softcap) is stored."""
     _need(x, torch.bfloat16, "x")
     _need(w, torch.bfloat16, "w")
     tiled = w.dim() == 4
@@ -545,6 +578,14 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tokens: int, fe
                                       _ptr(up_bias), up_row_offset, 1 if tiled else 0,
                                       status.data_ptr(), _stream()))
         return
+    if softcap > 0.0:
+        if epilogue != EPI_STORE_F32 or k_splits != 1:
+            raise ValueError("a softcap belongs to a float32 store")
+        _check(lib().hx_gemm_tc_softcapped(x.data_ptr(), x.stride(0), x.shape[0], w.data_ptr(), ldw,
+                                           rows, out.data_ptr(), out.stride(0), tokens, features,
+                                           depth, float(softcap), 1 if tiled else 0,
+                                           status.data_ptr(), _stream()))
+        return
     _check(lib().hx_gemm_tc(x.data_ptr(), x.stride(0), x.shape[0], w.data_ptr(), ldw, rows,
                             out.data_ptr(), out.stride(0), tokens, features, depth, epilogue,
                             up_row_offset, k_splits, 1 if tiled else 0, status.data_ptr(),
@@ -562,11 +603,13 @@ def gemm_tc_rope_append(x: torch.Tensor, w: torch.Tensor, qkv: torch.Tensor, tok
                         cos_table: torch.Tensor, sin_table: torch.Tensor, heads: int,
                         kv_heads: int, head_dim: int, rotary_dim: int, page_size: int,
                         num_pages: int, status: torch.Tensor,
-                        weight_shape: Optional[Tuple[int, int]] = None) -> None:
+                        weight_shape: Optional[Tuple[int, int]] = None,
+                        shared_values: bool = False) -> None:
     """The fused QKV product of a prompt portion (more than 64 tokens, bfloat16) with the
     rotary encoding and the cache append as its epilogue: ``qkv[:tokens, :heads * head_dim]``
     receives the rotated queries (the key and value columns of ``qkv`` are NOT written), keys
-    (rotated) and values go to their pages.  Adjacent pairs; ``w`` as for :func:`gemm_tc`."""
+    (rotated) and values go to their pages.  Adjacent pairs; ``w`` as for :func:`gemm_tc`;
+    ``shared_values`` as for :func:`rope_append` (``w`` then holds the query and key rows)."""
     _need(x, torch.bfloat16, "x")
     _need(w, torch.bfloat16, "w")
     _need(qkv, torch.bfloat16, "qkv")
@@ -583,14 +626,14 @@ def gemm_tc_rope_append(x: torch.Tensor, w: torch.Tensor, qkv: torch.Tensor, tok
         rows, depth = w.shape
         ldw = w.stride(0)
     write = k_cache is not None
-    _check(lib().hx_gemm_tc_rope_append(
+    _check(lib().hx_gemm_tc_rope_append_shared(
         x.data_ptr(), x.stride(0), x.shape[0], w.data_ptr(), ldw, rows, qkv.data_ptr(),
         qkv.stride(0), tokens, depth, 1 if tiled else 0, positions.data_ptr(),
         token_request.data_ptr(), request_table_row.data_ptr(),
         _ptr(block_tables) if write else None,
         block_tables.stride(0) if write else 0, _ptr(k_cache), _ptr(v_cache),
         cos_table.data_ptr(), sin_table.data_ptr(), cos_table.shape[0], heads, kv_heads, head_dim,
-        rotary_dim, page_size, num_pages, status.data_ptr(), _stream()))
+        rotary_dim, page_size, num_pages, 1 if shared_values else 0, status.data_ptr(), _stream()))
 
 
 def attention_scratch_floats(tokens: int, heads: int, head_dim: int, max_splits: int,
@@ -613,7 +656,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                     request_start: Optional[torch.Tensor] = None, skip_query_len: int = 0,
                     arrivals: Optional[torch.Tensor] = None, keep_first: int = 0,
                     sinks: Optional[torch.Tensor] = None,
-                    slopes: Optional[torch.Tensor] = None) -> None:
+                    slopes: Optional[torch.Tensor] = None, chunk: int = 0,
+                    softcap: float = 0.0) -> None:
     """out[t, h*D:(h+1)*D] = attention of query (t, h) over its request's pages.  With
     ``skip_query_len > 0`` tokens of requests that bring at least that many tokens are left
     out (the tensor-core kernel takes them).  With a window, keys at positions below
@@ -622,7 +666,9 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     ``arrivals`` (int32, one counter per (token, head), zero on entry; the kernel leaves it
     zero).  ``sinks`` (float32 ``[heads]``): the softmax's denominator also holds
     ``exp(sinks[h])``, a term without key or value.  ``slopes`` (float32 ``[heads]``): the score
-    of key ``j`` for the query at position ``i`` is lowered by ``slopes[h] * (i - j)``."""
+    of key ``j`` for the query at position ``i`` is lowered by ``slopes[h] * (i - j)``.
+    ``chunk`` > 0: position ``i`` sees ``j`` only when ``i // chunk == j // chunk``.  ``softcap`` >
+    0: the scaled score ``s`` becomes ``softcap * tanh(s / softcap)``."""
     for per_head in (sinks, slopes):
         if per_head is not None:
             _need(per_head, torch.float32, "sinks and slopes")
@@ -640,7 +686,7 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         out.data_ptr(), out.stride(0),
         _ptr(partial), _ptr(arrivals), tokens, heads, kv_heads, head_dim, page_size, num_pages, window,
         int(keep_first), float(scale), split_keys, max_splits, _ptr(sinks), _ptr(slopes),
-        _ptr(status), _stream()))
+        int(chunk), float(softcap), _ptr(status), _stream()))
 
 
 PREFILL_TILE_ROWS = 64        # query rows of a CTA of the ``mma.sync`` prompt kernel
@@ -670,7 +716,8 @@ def prefill_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
                       query_lengths: Optional[Sequence[int]] = None, window: int = 0,
                       keep_first: int = 0, packed: bool = False,
                       sinks: Optional[torch.Tensor] = None,
-                      slopes: Optional[torch.Tensor] = None) -> None:
+                      slopes: Optional[torch.Tensor] = None, chunk: int = 0,
+                      softcap: float = 0.0) -> None:
     """Tensor-core attention (bfloat16) of every request that brings at least
     ``min_query_len`` tokens; ``tile_bound`` bounds the number of query tiles of 64 tokens
     (the tensor-memory kernel, whose tiles hold 256 tokens, needs no more).  A CTA that finds
@@ -683,9 +730,10 @@ def prefill_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     j < ``keep_first``; both kernels skip the tiles of keys that no row of a query tile sees.
     ``packed``: the ``mma.sync`` kernel with the heads of a key/value head side by side in a
     tile's rows (``prefill_attention_packed_tokens`` tokens a tile), which reads keys and
-    values once for all of them; it takes single decoded tokens as well.  ``sinks`` and
-    ``slopes`` as in :func:`paged_attention`; all three kernels take them."""
-    biased = sinks is not None or slopes is not None
+    values once for all of them; it takes single decoded tokens as well.  ``sinks``,
+    ``slopes``, ``chunk`` and ``softcap`` as in :func:`paged_attention`; all three kernels take
+    them."""
+    biased = sinks is not None or slopes is not None or chunk > 0 or softcap > 0.0
     for per_head in (sinks, slopes):
         if per_head is not None:
             _need(per_head, torch.float32, "sinks and slopes")
@@ -712,12 +760,13 @@ def prefill_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
         kv_heads, head_dim, page_size, num_pages, float(scale), min_query_len)
     if biased and tensor_memory:
         _check(lib().hx_prefill_attention_tc_biased(*arguments, int(window), int(keep_first),
-                                                    _ptr(sinks), _ptr(slopes), _ptr(status),
-                                                    _stream()))
+                                                    _ptr(sinks), _ptr(slopes), int(chunk),
+                                                    float(softcap), _ptr(status), _stream()))
     elif biased:
         _check(lib().hx_prefill_attention_biased(*arguments, int(window), int(keep_first),
                                                  1 if packed else 0, _ptr(sinks), _ptr(slopes),
-                                                 _ptr(status), _stream()))
+                                                 int(chunk), float(softcap), _ptr(status),
+                                                 _stream()))
     elif packed:
         _check(lib().hx_prefill_attention_packed(*arguments, int(window), int(keep_first),
                                                  _ptr(status), _stream()))
@@ -857,25 +906,119 @@ def scan_state_floats(columns: int, rows: int) -> int:
 def causal_filter(raw: torch.Tensor, out: torch.Tensor, taps: torch.Tensor,
                   bias: Optional[torch.Tensor], state: Optional[torch.Tensor], tokens: int,
                   silu: bool, token_request: torch.Tensor, request_slot: torch.Tensor,
-                  request_start: torch.Tensor) -> None:
+                  request_start: torch.Tensor, in_bias: Optional[torch.Tensor] = None,
+                  sums: bool = False) -> None:
     """out[t, c] = f(bias[c] + sum_j taps[c, j] * raw[t - (n - 1) + j, c]) along each request's
     tokens, ``f`` silu or nothing; ``raw`` (a view of the filtered columns) and ``out`` in the
     compute dtype.  ``state`` ``[slots, >= (n - 1) * channels]`` float32 holds each request's
-    last ``n - 1`` inputs and is updated."""
+    last ``n - 1`` inputs and is updated.  ``in_bias`` ``[channels]``: added to every input (not
+    to the zeros before the sequence).  ``sums``: ``raw`` is a view of float32 sums, rounded to the
+    compute dtype as a product's store would have."""
     _need(taps, torch.float32, "taps")
     channels, count = taps.shape
-    assert raw.dtype == out.dtype and raw.stride(-1) == 1 and out.stride(-1) == 1
+    assert raw.dtype == (torch.float32 if sums else out.dtype) and raw.stride(-1) == 1 and out.stride(-1) == 1
     assert raw.shape[1] == channels and out.shape[1] == channels and taps.is_contiguous()
     if bias is not None:
         _need(bias, torch.float32, "bias")
     if count > 1:
         _need(state, torch.float32, "state")
         assert state.shape[1] >= (count - 1) * channels
-    _check(lib().hx_causal_filter(raw.data_ptr(), raw.stride(0), out.data_ptr(), out.stride(0),
-                                  dtype_code(out.dtype), taps.data_ptr(), _ptr(bias), _ptr(state),
-                                  0 if state is None else state.stride(0), count, channels,
-                                  1 if silu else 0, tokens, token_request.data_ptr(),
-                                  request_slot.data_ptr(), request_start.data_ptr(), _stream()))
+    if in_bias is not None:
+        _need(in_bias, torch.float32, "in_bias")
+        assert in_bias.numel() == channels
+    _check(lib().hx_causal_filter_biased(
+        None if sums else raw.data_ptr(), 0 if sums else raw.stride(0),
+        raw.data_ptr() if sums else None, raw.stride(0) if sums else 0, _ptr(in_bias),
+        out.data_ptr(), out.stride(0), dtype_code(out.dtype), taps.data_ptr(), _ptr(bias),
+        _ptr(state), 0 if state is None else state.stride(0), count, channels, 1 if silu else 0,
+        tokens, token_request.data_ptr(), request_slot.data_ptr(), request_start.data_ptr(),
+        _stream()))
+
+
+def _gate_operands(u, weights, r_bias, i_bias, rate):
+    blocks, two, size, columns = weights.shape
+    assert two == 2 and columns == size and weights.is_contiguous() and weights.dtype == u.dtype
+    assert u.stride(-1) == 1 and u.shape[1] >= blocks * size
+    for name, vector in (("r_bias", r_bias), ("i_bias", i_bias), ("rate", rate)):
+        _need(vector, torch.float32, name)
+        assert vector.numel() == blocks * size and vector.is_contiguous()
+    return blocks, size
+
+
+def gated_recurrence_supports(size: int) -> bool:
+    """Whether the tensor-core kernels take blocks of ``size`` channels (bfloat16)."""
+    return bool(lib().hx_gated_recurrence_supports(size))
+
+
+def block_gates(u: torch.Tensor, weights: torch.Tensor, r_bias: torch.Tensor,
+                i_bias: torch.Tensor, rate: torch.Tensor, decay: torch.Tensor, push: torch.Tensor,
+                tokens: int, status: torch.Tensor, tensor_cores: Optional[bool] = None) -> None:
+    """``decay = a - 1`` and ``push = sqrt(1 - a^2) i u`` with ``log a = -rate r``: ``r`` and ``i``
+    are the sigmoids of the two square matrices of every block of channels, ``weights`` ``[blocks,
+    2, size, size]``, applied to the block's part of ``u`` (plus ``r_bias``, ``i_bias``).  ``decay``
+    and ``push`` float32 ``[rows, channels]``.  ``tensor_cores``: the tcgen05 kernel (default: where
+    it applies) or the CUDA-core one."""
+    blocks, size = _gate_operands(u, weights, r_bias, i_bias, rate)
+    for name, out in (("decay", decay), ("push", push)):
+        _need(out, torch.float32, name)
+        assert out.is_contiguous() and out.shape[1] == blocks * size
+    if tensor_cores is None:
+        tensor_cores = (u.dtype == torch.bfloat16 and gated_recurrence_supports(size)
+                        and u.stride(0) % 8 == 0)
+    if tensor_cores:
+        _check(lib().hx_gemm_tc_block_gates(
+            u.data_ptr(), u.stride(0), u.shape[0], weights.data_ptr(), r_bias.data_ptr(),
+            i_bias.data_ptr(), rate.data_ptr(), decay.data_ptr(), push.data_ptr(), tokens, blocks,
+            size, status.data_ptr(), _stream()))
+        return
+    _check(lib().hx_block_gates(u.data_ptr(), u.stride(0), weights.data_ptr(), r_bias.data_ptr(),
+                                i_bias.data_ptr(), rate.data_ptr(), decay.data_ptr(),
+                                push.data_ptr(), dtype_code(u.dtype), tokens, blocks, size,
+                                _stream()))
+
+
+def _other_branch(y: torch.Tensor, sums: bool):
+    """The other branch's rows, or the float32 sums that hold them: (y, ld_y, accum, ld_accum)."""
+    if sums:
+        _need(y, torch.float32, "the sums of both branches")
+        return None, 0, y.data_ptr(), y.stride(0)
+    return y.data_ptr(), y.stride(0), None, 0
+
+
+def gated_scan(decay: torch.Tensor, push: torch.Tensor, y: torch.Tensor, y_bias: torch.Tensor,
+               state: torch.Tensor, out: torch.Tensor, request_start: torch.Tensor,
+               request_slot: torch.Tensor, requests: int, sums: bool = False) -> None:
+    """Along each request's tokens and per channel ``S <- S + (decay S + push)``, ``out = S
+    gelu_tanh(y + y_bias)``.  ``state`` ``[slots, >= channels]`` float32 is read and updated.
+    ``sums``: ``y`` is the float32 buffer ``[rows, >= 2 channels]`` that holds the sums of both
+    branches (the other one's columns first); its rows are cleared."""
+    channels = y_bias.numel()
+    _need(y_bias, torch.float32, "y_bias")
+    _need(state, torch.float32, "state")
+    assert decay.is_contiguous() and push.is_contiguous() and decay.shape[1] == channels
+    _check(lib().hx_gated_scan(decay.data_ptr(), push.data_ptr(), *_other_branch(y, sums),
+                               y_bias.data_ptr(), state.data_ptr(), state.stride(0), out.data_ptr(),
+                               out.stride(0), dtype_code(out.dtype), channels,
+                               request_start.data_ptr(), request_slot.data_ptr(), requests,
+                               _stream()))
+
+
+def gated_recurrence_step(u: torch.Tensor, weights: torch.Tensor, r_bias: torch.Tensor,
+                          i_bias: torch.Tensor, rate: torch.Tensor, y: torch.Tensor,
+                          y_bias: torch.Tensor, state: torch.Tensor, out: torch.Tensor, tokens: int,
+                          token_request: torch.Tensor, request_slot: torch.Tensor,
+                          sums: bool = False) -> None:
+    """:func:`block_gates` and :func:`gated_scan` as one kernel, for a step in which every request
+    brings exactly one token (bfloat16)."""
+    blocks, size = _gate_operands(u, weights, r_bias, i_bias, rate)
+    _need(u, torch.bfloat16, "u")
+    _need(y_bias, torch.float32, "y_bias")
+    _need(state, torch.float32, "state")
+    _check(lib().hx_gated_recurrence_step(
+        u.data_ptr(), u.stride(0), weights.data_ptr(), r_bias.data_ptr(), i_bias.data_ptr(),
+        rate.data_ptr(), *_other_branch(y, sums), y_bias.data_ptr(), state.data_ptr(),
+        state.stride(0), out.data_ptr(), out.stride(0), tokens, blocks, size,
+        token_request.data_ptr(), request_slot.data_ptr(), _stream()))
 
 
 def state_space_scan(x: torch.Tensor, b: torch.Tensor, c: torch.Tensor, dt: torch.Tensor,

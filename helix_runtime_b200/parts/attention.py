@@ -26,8 +26,15 @@ Optional mechanisms, each a parameter (absent: as if it did not exist):
   ``sigmoid(g x)`` before the output projection (tensor ``g`` ``[heads*value_dim, hidden]``);
   with a filter the gate's projection is part of the fused product.
 
-* ``sinks`` (True): a learned number per head (tensor ``sink`` ``[heads]``) whose exponential
-  is one more term of the softmax's denominator; it has no key and no value.
+* ``sinks``: one more term of the softmax's denominator without key or value, the exponential
+  of a number per head: True, a learned one (tensor ``sink`` ``[heads]``); a number, that score
+  for every head (0.0: one is added to the denominator).
+* ``chunk``: position ``i`` sees ``j <= i`` only when both lie in the same chunk of that many
+  positions, counted from position 0; what lies in front of the running chunk is given back to
+  the page pool.
+* ``softcap``: the scaled score ``s`` becomes ``softcap * tanh(s / softcap)``.
+* ``values`` (``"keys"``): there is no value projection, a token's value is its key as projected,
+  before the rotation (the position encoding has to know, ``shared_values``).
 * ``distance_slopes`` (a number per head): the score of key ``j`` for the query at position
   ``i`` is lowered by ``slope_h * (i - j)``.
 
@@ -62,6 +69,7 @@ from ..config.spec import PartSpec
 from ..ops import library as ops
 from ..weights.loader import TensorRequest
 from .base import LayerCache, Mixer, StepContext, build_part, register_part
+from .position import stretched_frequencies
 from .linear import (STREAMING_MAX_TOKENS, Weight, is_weight_stream, project,
                      project_into_accumulator)
 
@@ -90,30 +98,6 @@ def rotary_row_permutation(heads: int, head_dim: int, rotary_dim: int) -> torch.
     return torch.tensor(order, dtype=torch.long)
 
 
-def stretched_frequencies(dims: int, theta: float, scaling: Optional[Mapping[str, float]]):
-    """Frequencies of the ``dims / 2`` rotated pairs (float64 tensor) and the factor on sine and
-    cosine.  Without ``scaling``: ``f_i = theta^(-2i / dims)`` and 1.  With ``scaling``
-    (``factor``, ``original``: the trained length, ``fast`` and ``slow``: turns over that
-    length) a pair that turns more often than ``fast`` keeps its frequency, one that turns less
-    than ``slow`` takes ``f_i / factor``, and the pairs between are blended linearly in the
-    pair's index: with ``pair(t) = dims ln(original / (2 pi t)) / (2 ln theta)``, ``lo =
-    max(floor(pair(fast)), 0)``, ``hi = min(ceil(pair(slow)), dims - 1)`` and ``r_i =
-    clamp((i - lo) / max(hi - lo, 0.001), 0, 1)`` the frequency is ``f_i / factor * r_i + f_i
-    (1 - r_i)``; sine and cosine are multiplied by ``0.1 ln(factor) + 1``."""
-    index = torch.arange(dims // 2, dtype=torch.float64)
-    plain = torch.pow(torch.tensor(float(theta), dtype=torch.float64), -2.0 * index / float(dims))
-    if not scaling:
-        return plain, 1.0
-    factor, original = float(scaling["factor"]), float(scaling["original"])
-
-    def pair_of(turns: float) -> float:
-        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
-    lo = max(math.floor(pair_of(float(scaling["fast"]))), 0)
-    hi = min(math.ceil(pair_of(float(scaling["slow"]))), dims - 1)
-    ramp = torch.clamp((index - lo) / max(hi - lo, 0.001), 0.0, 1.0)
-    return plain / factor * ramp + plain * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
-
-
 class PagedAttention(Mixer):
     pack_heads = False      # subclasses whose heads share few cached rows set this
     pack_always = True      # ... for every step; False: only for steps of single tokens
@@ -129,6 +113,12 @@ class PagedAttention(Mixer):
         window = spec.get("window")
         self.window: Optional[int] = int(window) if window else None
         self.keep_first = int(spec.get("keep_first") or 0) if self.window else 0
+        chunk = spec.get("chunk")
+        self.chunk: Optional[int] = int(chunk) if chunk else None
+        values = spec.get("values")
+        if values not in (None, "keys"):
+            raise ValueError(f"values {values!r}: a projection of their own (None) or 'keys'")
+        self.shared_values = values == "keys"
         self.value_dim = int(spec.get("value_dim") or self.head_dim)
         self.conv_taps = int(spec.get("short_conv") or 1)
         if self.conv_taps < 1:
@@ -138,11 +128,26 @@ class PagedAttention(Mixer):
             raise ValueError(f"output gate {gate!r} has no kernel; only 'sigmoid'")
         self.gated = gate is not None
         self._init_score_terms(spec)
+        if self.shared_values:
+            if self.value_dim != self.head_dim or self.conv_taps > 1 or self.gated:
+                raise ValueError("values that are the keys have the keys' size, and neither a "
+                                 "filter nor an output gate beside them")
+            # query heads that share a key/value head decode side by side in a tile's rows
+            self.pack_heads = self.heads // self.kv_heads >= 2
+            self.pack_always = False
         self.row_dim = self.head_dim
-        self.position = build_part("position", spec["position"], hidden_size)
+        position_spec = spec["position"]
+        if self.shared_values:
+            position_spec = PartSpec(position_spec.kind,
+                                     {**position_spec.params, "shared_values": True},
+                                     position_spec.tensors)
+        self.position = build_part("position", position_spec, hidden_size)
+        if getattr(self.position, "shared_values", False) != self.shared_values:
+            raise ValueError(f"position encoding {position_spec.kind!r} does not take values from "
+                             "the keys")
         wide = row_width(max(self.head_dim, self.value_dim))
         if wide != self.head_dim or self.value_dim != self.head_dim:
-            position = spec["position"]
+            position = position_spec
             padded = build_part("position", PartSpec(position.kind,
                                                      {**position.params, "row_dim": wide,
                                                       "value_dim": self.value_dim},
@@ -162,7 +167,7 @@ class PagedAttention(Mixer):
         self.o_columns = self.heads * self.value_dim
         self.q_size = self.heads * self.row_dim
         self.kv_size = self.kv_heads * self.row_dim
-        self.qkv_size = self.q_size + 2 * self.kv_size
+        self.qkv_size = self.q_size + (1 if self.shared_values else 2) * self.kv_size
         # with a filter the gate's projection rides in the fused product, behind q, k and v
         self.fused_gate = self.gated and self.conv_taps > 1
         self.projected_size = self.qkv_size + (self.q_size if self.fused_gate else 0)
@@ -177,7 +182,13 @@ class PagedAttention(Mixer):
 
     def _init_score_terms(self, spec: PartSpec) -> None:
         """The optional per-head terms of the scores: sinks and distance slopes."""
-        self.has_sinks = bool(spec.get("sinks", False))
+        sinks = spec.get("sinks", False)
+        self.sink_score: Optional[float] = \
+            float(sinks) if sinks is not None and not isinstance(sinks, bool) else None
+        self.has_sinks = bool(sinks) if isinstance(sinks, bool) else False
+        self.softcap = float(spec.get("softcap") or 0.0)
+        if not (math.isfinite(self.softcap) and self.softcap >= 0.0):
+            raise ValueError("softcap is a positive level the scores run into")
         slopes = spec.get("distance_slopes")
         if slopes is not None and len(slopes) != self.heads:
             raise ValueError("distance_slopes gives one slope per head")
@@ -194,12 +205,15 @@ class PagedAttention(Mixer):
         if self.has_sinks:
             self.sinks = tensors[self.names["sink"]].to(device=device, dtype=torch.float32) \
                 .contiguous()
+        elif self.sink_score is not None:
+            self.sinks = torch.full((self.heads,), self.sink_score, dtype=torch.float32,
+                                    device=device)
         if self.slope_values is not None:
             self.slopes = torch.tensor(self.slope_values, dtype=torch.float64) \
                 .to(torch.float32).to(device).contiguous()
 
     def kv_need(self) -> Optional[KvNeed]:
-        return KvNeed(self.kv_heads, self.row_dim, self.window, self.keep_first)
+        return KvNeed(self.kv_heads, self.row_dim, self.window, self.keep_first, self.chunk)
 
     def state_need(self) -> Optional[StateNeed]:
         if self.conv_taps <= 1:
@@ -211,11 +225,12 @@ class PagedAttention(Mixer):
         requests = [
             TensorRequest(self.names["q"], (self.q_rows, h)),
             TensorRequest(self.names["k"], (self.kv_rows, h)),
-            TensorRequest(self.names["v"], (self.v_rows, h)),
             TensorRequest(self.names["o"], (h, self.o_columns)),
             *self.position.tensor_requests(),
             *self._score_term_requests(),
         ]
+        if not self.shared_values:
+            requests.insert(2, TensorRequest(self.names["v"], (self.v_rows, h)))
         if self.gated:
             requests.append(TensorRequest(self.names["g"], (self.o_columns, h)))
         if self.conv_taps > 1:
@@ -237,7 +252,7 @@ class PagedAttention(Mixer):
     def bind(self, tensors: Mapping[str, torch.Tensor], dtype, device) -> None:
         q = tensors[self.names["q"]]
         k = tensors[self.names["k"]]
-        v = tensors[self.names["v"]]
+        v = None if self.shared_values else tensors[self.names["v"]]
         if (self.checkpoint_pairing is not None and self.position.pairing is not None
                 and self.checkpoint_pairing != self.position.pairing):
             if self.checkpoint_pairing == "half_split" and self.position.pairing == "adjacent":
@@ -254,11 +269,11 @@ class PagedAttention(Mixer):
             else:
                 raise ValueError(f"no row permutation from {self.checkpoint_pairing!r} to "
                                  f"{self.position.pairing!r}")
-        q, k, v = (self.widen_rows(q, self.heads), self.widen_rows(k, self.kv_heads),
-                   self.widen_rows(v, self.kv_heads, self.value_dim))
+        q, k = self.widen_rows(q, self.heads), self.widen_rows(k, self.kv_heads)
         o = self.widen_rows(tensors[self.names["o"]].t().contiguous(), self.heads,
                             self.value_dim).t()
-        fused = [q, k, v]
+        fused = [q, k] if v is None else \
+            [q, k, self.widen_rows(v, self.kv_heads, self.value_dim)]
         if self.gated:
             g = self.widen_rows(tensors[self.names["g"]], self.heads, self.value_dim)
             if self.fused_gate:
@@ -332,7 +347,7 @@ class PagedAttention(Mixer):
         (``heads`` rows of ``row_dim``), keys and values from the entry's pages, the result into
         ``context``.  Chooses the kernels by the step's make-up."""
         n = ctx.n_tokens
-        window = cache.window or 0
+        window, chunk = cache.window or 0, cache.chunk or 0
         kept = self.keep_first if window else 0
         # prompt portions of at least TENSOR_CORE_MIN_QUERY tokens go to a tensor-core
         # kernel (bfloat16, head sizes it has; with a window the ``mma.sync`` one); the rest,
@@ -353,7 +368,8 @@ class PagedAttention(Mixer):
                                   self.row_dim, cache.page_size, cache.num_pages, self.scale, 1,
                                   ctx.status, query_lengths=ctx.host_query_lengths,
                                   window=window, keep_first=kept, packed=True,
-                                  sinks=self.sinks, slopes=self.slopes)
+                                  sinks=self.sinks, slopes=self.slopes, chunk=chunk,
+                                  softcap=self.softcap)
             return
         if tensor_cores:
             ops.prefill_attention(qkv, cache.keys, cache.values, ctx.request_start,
@@ -362,10 +378,13 @@ class PagedAttention(Mixer):
                                   self.kv_heads, self.row_dim, cache.page_size, cache.num_pages,
                                   self.scale, TENSOR_CORE_MIN_QUERY, ctx.status,
                                   query_lengths=ctx.host_query_lengths, window=window,
-                                  keep_first=kept, sinks=self.sinks, slopes=self.slopes)
+                                  keep_first=kept, sinks=self.sinks, slopes=self.slopes,
+                                  chunk=chunk, softcap=self.softcap)
         if not tensor_cores or ctx.min_query_len < TENSOR_CORE_MIN_QUERY:
             longest = ctx.max_context_len if not window else \
                 min(ctx.max_context_len, window + kept)
+            if chunk:
+                longest = min(longest, chunk + kept)
             split_keys = self.split_keys_for(n, longest, ctx.attention_split_keys)
             max_splits = max(1, -(-longest // split_keys))
             floats = ops.attention_scratch_floats(n, self.heads, self.row_dim, max_splits,
@@ -380,7 +399,7 @@ class PagedAttention(Mixer):
                                 ctx.status, request_start=ctx.request_start,
                                 skip_query_len=TENSOR_CORE_MIN_QUERY if tensor_cores else 0,
                                 arrivals=arrivals, keep_first=kept, sinks=self.sinks,
-                                slopes=self.slopes)
+                                slopes=self.slopes, chunk=chunk, softcap=self.softcap)
 
     def forward(self, ctx: StepContext, cache: LayerCache, x: torch.Tensor,
                 residual: torch.Tensor) -> None:

@@ -107,6 +107,7 @@ class LayerCache:
     page_size: int = 0
     num_pages: int = 0
     window: Optional[int] = None
+    chunk: Optional[int] = None
     state: Optional[torch.Tensor] = None        # [state slot, *shape]
 
 

@@ -4,7 +4,9 @@ Embedding: ``hidden[t] = table[id[t]] * scale`` widened into the float32 residua
 (src/model/cpu_llama.cpp:21-27, 49); with the parameter ``norm`` (a norm's part spec) the
 looked-up rows pass that norm, float32 in and out.  Head: ``logits = x @ head.T`` in float32
 (src/model/cpu_llama.cpp:107); when the checkpoint has no head tensor and ties its
-embeddings the table stands in (tools/convert_hf_llama.py:497-510).
+embeddings the table stands in (tools/convert_hf_llama.py:497-510).  With the parameter
+``softcap`` the logits run into a level, ``softcap * tanh(logits / softcap)``, in the product's
+epilogue.
 """
 from __future__ import annotations
 
@@ -58,6 +60,7 @@ class LmHead(Part):
         self.vocab_size = int(spec["vocab_size"])
         self.name = spec.tensors["weight"]
         self.fallback = spec.tensors.get("tied_to") if spec.get("tied", False) else None
+        self.softcap = float(spec.get("softcap") or 0.0)       # 0: the logits as they are
         self.weight: Optional[Weight] = None
 
     def tensor_requests(self) -> List[TensorRequest]:
@@ -71,7 +74,7 @@ class LmHead(Part):
         return self.weight.nbytes()
 
     def forward(self, ctx: StepContext, x: torch.Tensor, logits: torch.Tensor, rows: int) -> None:
-        project(x, self.weight, logits, rows, ops.EPI_STORE_F32, ctx.status)
+        project(x, self.weight, logits, rows, ops.EPI_STORE_F32, ctx.status, softcap=self.softcap)
 
 
 register_part("embedding", "token_table", TokenEmbedding)

@@ -8,11 +8,17 @@ cache; the coordinates from ``head_dim`` on are carried along unrotated),
 src/kernels/cpu/reference.cpp:519-531; ``half_split``: pairs ``(p, p + rotary_dim/2)``),
 ``max_positions``.  The cos/sin table ``[max_positions, rotary_dim/2]`` is built once
 in double and cast to float32, as the reference builds its table
-(src/model/llama_common.cpp:37-46); the kernel rotates in float32.
+(src/model/llama_common.cpp:37-46); the kernel rotates in float32.  Two more, each optional:
+``scaling`` (frequencies stretched for contexts beyond a trained length and the factor on sine and
+cosine that goes with them, see :func:`stretched_frequencies`; the factor is part of the table)
+and ``shared_values`` (the rows hold no values: a key as projected, before the rotation, is its
+value).  Encodings with the same numbers on the same device share one table.
 """
 from __future__ import annotations
 
-from typing import Mapping, Optional
+import math
+import weakref
+from typing import Dict, Mapping, Optional, Tuple
 
 import torch
 
@@ -20,6 +26,53 @@ from ..config.spec import PartSpec
 from ..ops import library as ops
 from .base import LayerCache, PositionEncoding, StepContext, register_part
 from .linear import Weight, uses_tensor_cores
+
+
+def stretched_frequencies(dims: int, theta: float, scaling: Optional[Mapping[str, float]]):
+    """Frequencies of the ``dims / 2`` rotated pairs (float64 tensor) and the factor on sine and
+    cosine.  Without ``scaling``: ``f_i = theta^(-2i / dims)`` and 1.  With ``scaling``
+    (``factor``, ``original``: the trained length, ``fast`` and ``slow``: turns over that
+    length) a pair that turns more often than ``fast`` keeps its frequency, one that turns less
+    than ``slow`` takes ``f_i / factor``, and the pairs between are blended linearly in the
+    pair's index: with ``pair(t) = dims ln(original / (2 pi t)) / (2 ln theta)``, ``lo =
+    max(floor(pair(fast)), 0)``, ``hi = min(ceil(pair(slow)), dims - 1)`` and ``r_i =
+    clamp((i - lo) / max(hi - lo, 0.001), 0, 1)`` the frequency is ``f_i / factor * r_i + f_i
+    (1 - r_i)``; sine and cosine are multiplied by ``0.1 ln(factor) + 1``."""
+    index = torch.arange(dims // 2, dtype=torch.float64)
+    plain = torch.pow(torch.tensor(float(theta), dtype=torch.float64), -2.0 * index / float(dims))
+    if not scaling:
+        return plain, 1.0
+    factor, original = float(scaling["factor"]), float(scaling["original"])
+
+    def pair_of(turns: float) -> float:
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
+    lo = max(math.floor(pair_of(float(scaling["fast"]))), 0)
+    hi = min(math.ceil(pair_of(float(scaling["slow"]))), dims - 1)
+    ramp = torch.clamp((index - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return plain / factor * ramp + plain * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+
+
+# tables that are in use, by what they are made of: the layers of a model share theirs
+_TABLES: "weakref.WeakValueDictionary[Tuple, RotaryTable]" = weakref.WeakValueDictionary()
+
+
+class RotaryTable:
+    """Cosines and sines ``[positions, pairs]`` in float32, taken in double."""
+
+    def __init__(self, frequency: torch.Tensor, amplitude: float, positions: int, device) -> None:
+        angle = torch.arange(positions, dtype=torch.float64, device=device)[:, None] \
+            * frequency.to(device)[None, :]
+        self.cos = (torch.cos(angle) * amplitude).to(torch.float32).contiguous()
+        self.sin = (torch.sin(angle) * amplitude).to(torch.float32).contiguous()
+
+    @classmethod
+    def shared(cls, frequency: torch.Tensor, amplitude: float, positions: int, device) -> "RotaryTable":
+        key = (tuple(frequency.tolist()), float(amplitude), int(positions), str(device))
+        table = _TABLES.get(key)
+        if table is None:
+            table = _TABLES[key] = cls(frequency, amplitude, positions, device)
+        return table
+
 
 PAIRINGS = {"adjacent": 0, "half_split": 1}
 
@@ -42,18 +95,23 @@ class RotaryEncoding(PositionEncoding):
             raise ValueError("rotary_dim must be even and at most head_dim")
         if not self.theta > 0.0:
             raise ValueError("rotary theta must be positive")
+        self.scaling = spec.get("scaling")
+        # the reference holds theta as a float32 value (include/helix/model/llama.hpp:22)
+        self.exact_theta = bool(spec.get("exact_theta", False))
+        self.shared_values = bool(spec.get("shared_values", False))
+        self.table: Optional[RotaryTable] = None
         self.cos: Optional[torch.Tensor] = None
         self.sin: Optional[torch.Tensor] = None
 
     def bind(self, tensors: Mapping[str, torch.Tensor], dtype, device) -> None:
-        half = max(self.rotary_dim // 2, 1)
-        # the reference holds theta as a float32 value (include/helix/model/llama.hpp:22)
-        theta = float(torch.tensor(self.theta, dtype=torch.float32).item())
-        exponent = -2.0 * torch.arange(half, dtype=torch.float64) / float(max(self.rotary_dim, 1))
-        frequency = torch.pow(torch.tensor(theta, dtype=torch.float64), exponent)
-        angle = torch.arange(self.max_positions, dtype=torch.float64)[:, None] * frequency[None, :]
-        self.cos = torch.cos(angle).to(torch.float32).to(device).contiguous()
-        self.sin = torch.sin(angle).to(torch.float32).to(device).contiguous()
+        theta = self.theta if self.exact_theta else \
+            float(torch.tensor(self.theta, dtype=torch.float32).item())
+        if self.rotary_dim:
+            frequency, amplitude = stretched_frequencies(self.rotary_dim, theta, self.scaling)
+        else:
+            frequency, amplitude = torch.ones((1,), dtype=torch.float64), 1.0
+        self.table = RotaryTable.shared(frequency, amplitude, self.max_positions, device)
+        self.cos, self.sin = self.table.cos, self.table.sin
 
     def apply(self, ctx: StepContext, cache: LayerCache, qkv: torch.Tensor, heads: int,
               kv_heads: int, accum: Optional[torch.Tensor] = None) -> None:
@@ -65,8 +123,8 @@ class RotaryEncoding(PositionEncoding):
                         cache.block_tables, cache.keys if write else None,
                         cache.values if write else None, self.cos, self.sin, ctx.n_tokens, heads,
                         kv_heads, self.row_dim, self.rotary_dim, PAIRINGS[self.pairing],
-                        cache.page_size, cache.num_pages, ctx.status, accum=accum)
-
+                        cache.page_size, cache.num_pages, ctx.status, accum=accum,
+                        shared_values=self.shared_values)
 
     def project_and_apply(self, ctx: StepContext, cache: LayerCache, x: torch.Tensor,
                           weight: Weight, qkv: torch.Tensor, heads: int, kv_heads: int) -> bool:
@@ -76,7 +134,7 @@ class RotaryEncoding(PositionEncoding):
         consecutive coordinates of one token) and heads in steps of 16."""
         n = ctx.n_tokens
         if (self.pairing != "adjacent" or self.row_dim % 16
-                or weight.rows != (heads + 2 * kv_heads) * self.row_dim
+                or weight.rows != (heads + (1 if self.shared_values else 2) * kv_heads) * self.row_dim
                 or n < ops.gemm_tc_rope_append_min_tokens() or not uses_tensor_cores(x, weight, n)
                 or qkv.dtype != torch.bfloat16 or qkv.stride(0) % 8):
             return False
@@ -87,7 +145,7 @@ class RotaryEncoding(PositionEncoding):
                                 cache.keys if write else None, cache.values if write else None,
                                 self.cos, self.sin, heads, kv_heads, self.row_dim, self.rotary_dim,
                                 cache.page_size, cache.num_pages, ctx.status,
-                                weight_shape=weight.shape)
+                                weight_shape=weight.shape, shared_values=self.shared_values)
         return True
 
 

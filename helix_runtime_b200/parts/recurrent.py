@@ -1,7 +1,8 @@
 """Recurrent mixers: the selective state-space layer, the time-mixing layer with a decayed
-outer-product state, and a mixer that runs several mixers side by side.
+outer-product state, linear attention, the gated linear recurrence, and mixers that wrap or run
+others.
 
-All three keep per-request state in ONE float32 row per schedule entry (``StateNeed`` of a flat
+All of them keep per-request state in ONE float32 row per schedule entry (``StateNeed`` of a flat
 shape); a mixer cuts its row into the pieces it needs.  A step brings a portion of each
 request's tokens (cut anywhere, one token when decoding); the kernels carry the state from
 portion to portion, so the result does not depend on the cut.
@@ -37,6 +38,17 @@ coordinates), ``q_scale``, ``k_scale``, ``norm_weight`` (the head norm has a wei
 the weight, times ``silu(W_g x)``, then the output projection.  State: the filter's last inputs
 and the matrices.
 
+:class:`GatedRecurrence` (``gated_recurrence``).  A recurrence of one number per channel whose
+decay and input are gated, beside a branch that gates its output.  Parameters ``width`` (channels
+of either branch), ``blocks`` (equal parts of the channels), ``filter_taps``, ``decay_rate``
+(``c``).  ``y = gelu_tanh(W_y x + b_y)``; ``u`` is a causal per-channel filter with bias over ``W_x
+x + b_x``; per block ``r = sigmoid(R u + b_r)``, ``i = sigmoid(I u + b_i)``; ``log a = -c r
+softplus(decay)``, ``S_t = a S_(t-1) + sqrt(1 - a^2) i u``; the output projection reads ``S y``.
+Tensors ``y``, ``x`` ``[width, hidden]``, ``y_bias``, ``x_bias``, ``filter`` ``[width, taps]`` (the
+last tap on the token itself), ``filter_bias``, ``r``, ``i`` ``[blocks, width / blocks, width /
+blocks]``, ``r_bias``, ``i_bias`` ``[blocks, width / blocks]``, ``decay`` ``[width]``, ``o``.  State:
+the filter's last inputs and the numbers ``S``.
+
 :class:`InputFilter` (``input_filter``).  Parameters ``taps``, ``mixer`` (a part spec): the inner
 mixer reads ``x + conv(x)``, ``conv`` a causal per-channel filter over time (tensor ``filter``
 ``[hidden, taps]``, the last tap on the token itself); the last ``taps - 1`` inputs are state.
@@ -56,7 +68,8 @@ from ..config.spec import PartSpec
 from ..ops import library as ops
 from ..weights.loader import TensorRequest
 from .base import LayerCache, Mixer, StepContext, build_part, register_part
-from .linear import Weight, project
+from .linear import (STREAMING_MAX_TOKENS, Weight, is_weight_stream, project,
+                     project_into_accumulator)
 
 
 def _state_piece(cache: LayerCache, offset: int, size: int) -> torch.Tensor:
@@ -381,6 +394,100 @@ class LinearState(Mixer):
         project(gated, self.w_o, residual, n, ops.EPI_ADD_F32, ctx.status, ctx.ordered_sums)
 
 
+class GatedRecurrence(Mixer):
+    def __init__(self, spec: PartSpec, hidden_size: int) -> None:
+        super().__init__(spec, hidden_size)
+        self.width = int(spec["width"])
+        self.blocks = int(spec.get("blocks", 1))
+        if self.blocks < 1 or self.width % self.blocks:
+            raise ValueError("blocks must divide width")
+        self.block_size = self.width // self.blocks
+        self.taps = int(spec.get("filter_taps", 1))
+        if self.taps < 1:
+            raise ValueError("filter_taps counts the filter's taps: at least 1")
+        self.decay_rate = float(spec.get("decay_rate", 8.0))
+        self.filter_state = (self.taps - 1) * self.width
+        self.names = dict(spec.tensors)
+        self.w_in: Optional[Weight] = None
+        self.w_o: Optional[Weight] = None
+
+    def state_need(self) -> Optional[StateNeed]:
+        return StateNeed((self.filter_state + self.width,), torch.float32)
+
+    def tensor_requests(self) -> List[TensorRequest]:
+        h, w, square = self.hidden_size, self.width, (self.blocks, self.block_size, self.block_size)
+        return [TensorRequest(self.names["y"], (w, h)),
+                TensorRequest(self.names["y_bias"], (w,), role="scale"),
+                TensorRequest(self.names["x"], (w, h)),
+                TensorRequest(self.names["x_bias"], (w,), role="scale"),
+                TensorRequest(self.names["filter"], (w, self.taps), role="scale"),
+                TensorRequest(self.names["filter_bias"], (w,), role="scale"),
+                TensorRequest(self.names["r"], square),
+                TensorRequest(self.names["r_bias"], square[:2], role="scale"),
+                TensorRequest(self.names["i"], square),
+                TensorRequest(self.names["i_bias"], square[:2], role="scale"),
+                TensorRequest(self.names["decay"], (w,), role="scale"),
+                TensorRequest(self.names["o"], (h, w))]
+
+    def bind(self, tensors: Mapping[str, torch.Tensor], dtype, device) -> None:
+        def scale(role: str) -> torch.Tensor:
+            return tensors[self.names[role]].to(device=device, dtype=torch.float32) \
+                .reshape(-1).contiguous()
+        # both branches read the mixer's input: one product, the gating branch's rows first
+        self.w_in = Weight(torch.cat([tensors[self.names["y"]], tensors[self.names["x"]]], dim=0)
+                           .to(device=device, dtype=dtype).contiguous())
+        self.w_o = Weight(tensors[self.names["o"]].to(device=device, dtype=dtype).contiguous())
+        self.w_gates = torch.stack([tensors[self.names["r"]], tensors[self.names["i"]]], dim=1) \
+            .to(device=device, dtype=dtype).contiguous()
+        self.filter = tensors[self.names["filter"]].to(device=device, dtype=torch.float32).contiguous()
+        self.filter_bias, self.y_bias, self.x_bias = (scale("filter_bias"), scale("y_bias"),
+                                                      scale("x_bias"))
+        self.r_bias, self.i_bias = scale("r_bias"), scale("i_bias")
+        decay = tensors[self.names["decay"]].to(device=device, dtype=torch.float64)
+        self.rate = (self.decay_rate * torch.nn.functional.softplus(decay, threshold=700.0)) \
+            .to(torch.float32).contiguous()
+        self.tensor_cores = dtype == torch.bfloat16 and \
+            ops.gated_recurrence_supports(self.block_size)
+
+    def weight_bytes(self) -> int:
+        return self.w_in.nbytes() + self.w_o.nbytes() \
+            + self.w_gates.numel() * self.w_gates.element_size()
+
+    def forward(self, ctx: StepContext, cache: LayerCache, x: torch.Tensor,
+                residual: torch.Tensor) -> None:
+        n, w, get = ctx.n_tokens, self.width, ctx.workspace.get
+        sums = is_weight_stream(x, self.w_in, n)
+        if sums:
+            # few tokens: split-K into float32 sums, which the recurrence's kernel clears
+            rows = ctx.workspace.accumulator(f"gated_recurrence.rows/{w}",
+                                             (STREAMING_MAX_TOKENS, 2 * w))
+            project_into_accumulator(x, self.w_in, rows, n, ctx.status, ctx.ordered_sums)
+        else:
+            rows = get(f"gated_recurrence.rows/{w}", (ctx.capacity, -(-2 * w // 8) * 8), ctx.dtype)
+            project(x, self.w_in, rows, n, ops.EPI_STORE, ctx.status)
+        # rows of a width that keeps them 16-byte aligned
+        wide = -(-w // 8) * 8
+        u = get(f"gated_recurrence.filtered/{w}", (ctx.capacity, wide), ctx.dtype)
+        gated = get(f"gated_recurrence.gated/{w}", (ctx.capacity, wide), ctx.dtype)[:, :w]
+        ops.causal_filter(rows[:, w:2 * w], u[:, :w], self.filter, self.filter_bias,
+                          _state_piece(cache, 0, self.filter_state) if self.taps > 1 else None,
+                          n, False, ctx.token_request, ctx.request_slot, ctx.request_start,
+                          in_bias=self.x_bias, sums=sums)
+        state = _state_piece(cache, self.filter_state, w)
+        if self.tensor_cores and n == ctx.n_requests:
+            ops.gated_recurrence_step(u, self.w_gates, self.r_bias, self.i_bias, self.rate, rows,
+                                      self.y_bias, state, gated, n, ctx.token_request,
+                                      ctx.request_slot, sums=sums)
+        else:
+            decay = get(f"gated_recurrence.decay/{w}", (ctx.capacity, w), torch.float32)
+            push = get(f"gated_recurrence.push/{w}", (ctx.capacity, w), torch.float32)
+            ops.block_gates(u, self.w_gates, self.r_bias, self.i_bias, self.rate, decay, push, n,
+                            ctx.status)
+            ops.gated_scan(decay, push, rows, self.y_bias, state, gated, ctx.request_start,
+                           ctx.request_slot, ctx.n_requests, sums=sums)
+        project(gated, self.w_o, residual, n, ops.EPI_ADD_F32, ctx.status, ctx.ordered_sums)
+
+
 class InputFilter(Mixer):
     def __init__(self, spec: PartSpec, hidden_size: int) -> None:
         super().__init__(spec, hidden_size)
@@ -500,3 +607,4 @@ register_part("mixer", "time_mix", TimeMix)
 register_part("mixer", "side_by_side", SideBySide)
 register_part("mixer", "linear_state", LinearState)
 register_part("mixer", "input_filter", InputFilter)
+register_part("mixer", "gated_recurrence", GatedRecurrence)

@@ -147,6 +147,41 @@ int hx_causal_filter(const void* raw, int ld_raw, void* out, int ld_out, int dty
                      long long state_stride, int taps, int channels, int silu, int tokens,
                      const int* token_request, const int* request_slot, const int* request_start,
                      cudaStream_t stream);
+/* the same with a bias on the inputs (in_bias [channels] or NULL; the zeros in front of the
+ * sequence stay zeros) and with inputs that may lie in float32 sums: raw or accum is given, the
+ * other NULL; sums are rounded to `dtype` first */
+int hx_causal_filter_biased(const void* raw, int ld_raw, const float* accum, int ld_accum,
+                            const float* in_bias, void* out, int ld_out, int dtype,
+                            const float* taps_weight, const float* bias, float* state,
+                            long long state_stride, int taps, int channels, int silu, int tokens,
+                            const int* token_request, const int* request_slot,
+                            const int* request_start, cudaStream_t stream);
+/* a gated linear recurrence, one number per channel: decay = a - 1 and push = sqrt(1 - a^2) i u
+ * with log a = -rate[c] r; r, i = sigmoids of block b's two matrices w [blocks][2][size][size]
+ * applied to its part of u, plus biases; then S <- S + (decay S + push) along each request and
+ * out = S gelu_tanh(y + y_bias).  y [tokens][ld_y] in `dtype`, or NULL: accum [tokens][ld_accum]
+ * holds the float32 sums of y's columns and, behind them, of the filtered branch's; both are
+ * cleared.  state: one float per channel. */
+int hx_block_gates(const void* u, int ld_u, const void* w, const float* r_bias,
+                   const float* i_bias, const float* rate, float* decay, float* push, int dtype,
+                   int tokens, int blocks, int size, cudaStream_t stream);
+int hx_gated_scan(const float* decay, const float* push, const void* y, int ld_y, float* accum,
+                  int ld_accum, const float* y_bias, float* state, long long state_stride,
+                  void* out, int ld_out, int dtype, int channels, const int* request_start,
+                  const int* request_slot, int requests, cudaStream_t stream);
+/* bfloat16, `size` a multiple of 8 (supports returns 1): the gates on tcgen05, and gates, scan and
+ * output as one kernel for one token per request */
+int hx_gated_recurrence_supports(int size);
+int hx_gemm_tc_block_gates(const void* u, int ld_u, int u_capacity_rows, const void* w,
+                           const float* r_bias, const float* i_bias, const float* rate,
+                           float* decay, float* push, int tokens, int blocks, int size,
+                           int* status, cudaStream_t stream);
+int hx_gated_recurrence_step(const void* u, int ld_u, const void* w, const float* r_bias,
+                             const float* i_bias, const float* rate, const void* y, int ld_y,
+                             float* accum, int ld_accum, const float* y_bias, float* state,
+                             long long state_stride, void* out, int ld_out, int tokens, int blocks,
+                             int size, const int* token_request, const int* request_slot,
+                             cudaStream_t stream);
 /* floats that a head's rows x columns matrix takes in a state row (the kernels' own order) */
 int hx_scan_state_floats(int columns, int rows);
 /* per head: S = exp(-exp(a_log) d) S + d B x', y = S' C + skip x, d = softplus(dt + dt_bias);
@@ -328,6 +363,14 @@ int hx_rope_append(void* qkv, int dtype, int ld, const int* positions, const int
                    const float* sin_table, int table_positions, int tokens, int heads, int kv_heads,
                    int head_dim, int rotary_dim, int pairing, int page_size, int num_pages,
                    int* status, float* accum, int ld_accum, cudaStream_t stream);
+/* shared_values != 0: a row is [q heads | k heads], a key as projected is its value */
+int hx_rope_append_shared(void* qkv, int dtype, int ld, const int* positions,
+                          const int* token_request, const int* request_table_row,
+                          const int* block_tables, int table_stride, void* k_cache, void* v_cache,
+                          int write_cache, const float* cos_table, const float* sin_table,
+                          int table_positions, int tokens, int heads, int kv_heads, int head_dim,
+                          int rotary_dim, int pairing, int page_size, int num_pages, int* status,
+                          float* accum, int ld_accum, int shared_values, cudaStream_t stream);
 /* token_ids[i] = max(sampled[rows[i]], 0): a step takes its tokens from the output of the
  * step before it without a round trip to the host */
 int hx_feed_tokens(int* token_ids, const int* sampled, const int* rows, int count,
@@ -337,6 +380,14 @@ int hx_feed_tokens(int* token_ids, const int* sampled, const int* rows, int coun
 /* CUDA cores, float32 accumulate in a fixed order; both dtypes; the true 32-bit path */
 int hx_gemm_simt(const void* x, int ldx, const void* w, int ldw, void* out, int ldo, int dtype,
                  int tokens, int features, int depth, int epilogue, cudaStream_t stream);
+/* softcap > 0 with epilogue 1: out = softcap * tanh(product / softcap) */
+int hx_gemm_simt_softcapped(const void* x, int ldx, const void* w, int ldw, void* out, int ldo,
+                            int dtype, int tokens, int features, int depth, int epilogue,
+                            float softcap, cudaStream_t stream);
+int hx_gemm_tc_softcapped(const void* x, int ldx, int x_capacity_rows, const void* w, int ldw,
+                          int weight_rows, float* out, int ldo, int tokens, int features,
+                          int depth, float softcap, int weight_tiles, int* status,
+                          cudaStream_t stream);
 /* tcgen05 tensor cores, bfloat16 operands, float32 accumulate in tensor memory.
  * weight_tiles != 0: w holds the matrix as [ceil(rows / 128)][ceil(depth / 64)] tiles of
  * [128][64] elements, zero padded, each tile 16 contiguous kilobytes (ldw is ignored). */
@@ -357,6 +408,16 @@ int hx_gemm_tc_rope_append(const void* x, int ldx, int x_capacity_rows, const vo
                            const float* sin_table, int table_positions, int heads, int kv_heads,
                            int head_dim, int rotary_dim, int page_size, int num_pages, int* status,
                            cudaStream_t stream);
+/* shared_values != 0: w = [q heads | k heads], a key before the rotation is its value */
+int hx_gemm_tc_rope_append_shared(const void* x, int ldx, int x_capacity_rows, const void* w,
+                                  int ldw, int weight_rows, void* out, int ldo, int tokens,
+                                  int depth, int weight_tiles, const int* positions,
+                                  const int* token_request, const int* request_table_row,
+                                  const int* block_tables, int table_stride, void* k_cache,
+                                  void* v_cache, const float* cos_table, const float* sin_table,
+                                  int table_positions, int heads, int kv_heads, int head_dim,
+                                  int rotary_dim, int page_size, int num_pages, int shared_values,
+                                  int* status, cudaStream_t stream);
 
 /* hx_gemm_tc with the gated epilogue for every gate activation (see hx_biased_gated_activation)
  * and float32 biases on the gate and the up rows ([features] each, either may be null) */
@@ -405,7 +466,9 @@ int hx_paged_attention_kept(const void* q, int ldq, const void* k_cache, const v
                             int max_splits, int* status, cudaStream_t stream);
 /* the same with two optional float32 arrays per query head (null: absent): sinks: the softmax's
    denominator also holds exp(sinks[h]), a term without key or value; slopes: the score of key j
-   for the query at position i is lowered by slopes[h] * (i - j) */
+   for the query at position i is lowered by slopes[h] * (i - j); chunk > 0: position i sees j
+   only when i / chunk == j / chunk; softcap > 0: the scaled score s becomes softcap * tanh(s /
+   softcap), before slopes and mask */
 int hx_paged_attention_biased(const void* q, int ldq, const void* k_cache, const void* v_cache,
                               int dtype, const int* positions, const int* token_request,
                               const int* request_table_row, const int* block_tables,
@@ -414,7 +477,7 @@ int hx_paged_attention_biased(const void* q, int ldq, const void* k_cache, const
                               int heads, int kv_heads, int head_dim, int page_size, int num_pages,
                               int window, int keep_first, float scale, int split_keys,
                               int max_splits, const float* sinks, const float* slopes,
-                              int* status, cudaStream_t stream);
+                              int chunk, float softcap, int* status, cudaStream_t stream);
 /* the same with scratch built into the library: see hx_no_alloc.h beside the sources */
 int hx_paged_attention_no_alloc(const void* q, int ldq, const void* k_cache, const void* v_cache,
                                 int dtype, const int* positions, const int* token_request,
@@ -462,7 +525,8 @@ int hx_prefill_attention_biased(const void* q, int ldq, const void* k_cache, con
                                 int tile_bound, int heads, int kv_heads, int head_dim,
                                 int page_size, int num_pages, float scale, int min_query_len,
                                 int window, int keep_first, int pack_heads, const float* sinks,
-                                const float* slopes, int* status, cudaStream_t stream);
+                                const float* slopes, int chunk, float softcap, int* status,
+                                cudaStream_t stream);
 
 /* the same on tcgen05, scores and partial outputs in tensor memory (pages of 16, 32, 64) */
 int hx_prefill_attention_tc_supports(int head_dim, int page_size);
@@ -481,7 +545,8 @@ int hx_prefill_attention_tc_biased(const void* q, int ldq, const void* k_cache, 
                                    int tile_bound, int heads, int kv_heads, int head_dim,
                                    int page_size, int num_pages, float scale, int min_query_len,
                                    int window, int keep_first, const float* sinks,
-                                   const float* slopes, int* status, cudaStream_t stream);
+                                   const float* slopes, int chunk, float softcap, int* status,
+                                   cudaStream_t stream);
 /* the tcgen05 kernel with a window and kept first keys (see hx_prefill_attention_windowed) */
 int hx_prefill_attention_tc_windowed(const void* q, int ldq, const void* k_cache,
                                      const void* v_cache, const int* request_start,
