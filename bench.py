@@ -472,6 +472,34 @@ def rorovik_config(shape: dict, options):
                          max_positions=shape["max_position_embeddings"])
 
 
+def pizilix_config(shape: dict, options):
+    """The Pizilix design with the layer sizes of a Llama shape: the same width, feed-forward and
+    vocabulary.  Layers in turn: the gated linear recurrence (channels of the model's width in 16
+    blocks, a filter of four taps) and attention (the shape's heads on
+    a quarter as many key/value heads, chunks of ``--window`` or 1,024 positions, half of a head
+    rotated with stretched frequencies, scores that level off at 50, logits at 30); no repeated
+    stretch."""
+    import math
+
+    from helix_runtime_b200.config.pizilix import (ChunkedAttentionConfig, GatedRecurrenceConfig,
+                                                   PizilixConfig, PizilixLayerConfig)
+    from helix_runtime_b200.config.rekasun import DenseMlpConfig
+    from helix_runtime_b200.config.rorovik import RotaryScalingConfig
+    heads, dim, width = shape["num_attention_heads"], shape["head_dim"], shape["hidden_size"]
+    attention = ChunkedAttentionConfig(
+        heads=heads, kv_heads=options.kv_heads or max(1, heads // 4), dim=dim,
+        scale=1.0 / math.sqrt(dim), softcap=50.0, chunk=options.window or 1024, rot_base=500000.0,
+        rot_dims=dim // 2, scaling=RotaryScalingConfig(factor=8.0, original=1024, fast=32.0, slow=1.0))
+    recurrence = GatedRecurrenceConfig(width=width, blocks=16, conv=4)
+    mlp = DenseMlpConfig(shape["intermediate_size"])
+    layers = tuple(PizilixLayerConfig("attention", attention, mlp) if index % 2 else
+                   PizilixLayerConfig("rglru", recurrence, mlp)
+                   for index in range(shape["num_hidden_layers"]))
+    return PizilixConfig(vocab=shape["vocab_size"], width=width, norm_eps=shape["rms_norm_eps"],
+                         layers=layers, logit_softcap=30.0,
+                         max_positions=shape["max_position_embeddings"])
+
+
 def compare_designs(options, peaks, device) -> int:
     """``--compare``: the Rekasun design beside the Llama design at equal layer sizes
     (``--compare zuzadra``: and the Zuzadra design beside both), a few
@@ -540,7 +568,7 @@ def compare_designs(options, peaks, device) -> int:
             engine.run_until_done()
             step_bytes = model.weight_bytes_per_step() + batch * sum(
                 2 * need.kv_heads * need.head_dim * 2
-                * (context if need.window is None else min(context, need.window + need.keep_first))
+                * min(context, context - need.first_seen(context - 1) + need.keep_first)
                 for need in kv.values())
             # recurrent state is read and written once per request and step
             step_bytes += batch * sum(2 * int(np.prod(need.shape)) * need.dtype.itemsize
@@ -563,14 +591,16 @@ def compare_designs(options, peaks, device) -> int:
         row = {"hidden": shape["hidden_size"], "heads": shape["num_attention_heads"],
                "head_dim": shape["head_dim"], "intermediate": shape["intermediate_size"]}
         designs = [("llama", LlamaConfig(**shape))]
-        if options.compare != "rorovik":
+        if options.compare not in ("rorovik", "pizilix"):
             designs.append(("rekasun", rekasun_config(shape, options)))
-        if options.compare in ("zuzadra", "medolorn"):
+        if options.compare in ("zuzadra", "medolorn", "pizilix"):
             designs.append(("zuzadra", zuzadra_config(shape, options)))
         if options.compare in ("medolorn", "rorovik"):
             designs.append(("medolorn", medolorn_config(shape, options)))
-        if options.compare == "rorovik":
+        if options.compare in ("rorovik", "pizilix"):
             designs.append(("rorovik", rorovik_config(shape, options)))
+        if options.compare == "pizilix":
+            designs.append(("pizilix", pizilix_config(shape, options)))
         for design, config in designs:
             model = random_model(config, seed=0, dtype="bfloat16", device=device)
             row[design] = measure(model)
@@ -580,7 +610,8 @@ def compare_designs(options, peaks, device) -> int:
     print(json.dumps({
         "metric": "prefill and decode throughput, " + {"zuzadra": "Zuzadra and Rekasun",
                                                         "medolorn": "Medolorn, Zuzadra and Rekasun",
-                                                        "rorovik": "Rorovik and Medolorn"}
+                                                        "rorovik": "Rorovik and Medolorn",
+                                                        "pizilix": "Pizilix, Rorovik and Zuzadra"}
                   .get(options.compare, "Rekasun") +
                   " design beside Llama design (bf16)",
         "layers": layers, "prefill_tokens": PREFILL_TOKENS, "decode_context": context,
@@ -615,18 +646,20 @@ def main() -> int:
     parser.add_argument("--shape", choices=tuple(SHAPES), default="llama-2-7b",
                         help="layer sizes for --serving, --profile and --timeline (the contract "
                              "line is always the Llama-2-7B shape)")
-    parser.add_argument("--design", choices=("llama", "rekasun", "zuzadra", "medolorn", "rorovik"),
+    parser.add_argument("--design", choices=("llama", "rekasun", "zuzadra", "medolorn", "rorovik",
+                                           "pizilix"),
                         default="llama",
                         help="which decoder the layers of --shape are built as, for --profile "
                              "and --timeline (the contract line is always the Llama design)")
     parser.add_argument("--compare", nargs="?", const="rekasun", default=None,
-                        choices=("rekasun", "zuzadra", "medolorn", "rorovik"),
+                        choices=("rekasun", "zuzadra", "medolorn", "rorovik", "pizilix"),
                         help="prefill and decode throughput of the Rekasun design beside the "
                              "Llama design at equal layer sizes (a few layers of each --shape), "
                              "as one JSON line of its own; '--compare zuzadra' adds the Zuzadra "
                              "design as a third row, '--compare medolorn' the Medolorn design "
                              "as a fourth; '--compare rorovik' runs the Llama, Medolorn and "
-                             "Rorovik designs")
+                             "Rorovik designs, '--compare pizilix' the Llama, Zuzadra, Rorovik "
+                             "and Pizilix designs")
     parser.add_argument("--window", type=int, default=1024,
                         help="--design rekasun / --compare: keys a position sees behind itself")
     parser.add_argument("--keep-first", type=int, default=64,
@@ -687,6 +720,8 @@ def main() -> int:
         config = medolorn_config(shape, options)
     elif options.design == "rorovik":
         config = rorovik_config(shape, options)
+    elif options.design == "pizilix":
+        config = pizilix_config(shape, options)
     model = random_model(config, seed=0, dtype="bfloat16", device=device)
     rng = np.random.default_rng(0)
     out_dir = options.log_dir or tempfile.mkdtemp(prefix="helix_bench_")

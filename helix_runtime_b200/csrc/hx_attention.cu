@@ -27,6 +27,12 @@
 //    second product as two bfloat16 terms (hi + lo), so the softmax stays a float32
 //    quantity as far as the result can tell.
 //
+// Query heads that share a key/value head.  The tile's 8-column side has room for four of them:
+// with `group` = 2 to 4 a row of the streaming kernel is a token's group of up to four heads, one
+// per pair of columns (the pair holds the hi and lo part of that head's probabilities in the
+// second product), and keys and values are fetched and multiplied once for the group, in the
+// same number of instructions as for one head.
+//
 // Sharing a long context between warps.  The CUDA-core kernel cuts a context into splits of
 // `split_keys` keys, one warp each.  The streaming kernel lays all 32-key chunks of all rows
 // (token, head) end to end and gives every warp of a grid that fills the GPU once an equal
@@ -88,7 +94,25 @@ struct AttentionArgs {
   const float* slopes = nullptr;
   int chunk = 0;          // > 0: positions see each other only inside chunks of this many
   float softcap = 0.0f;   // > 0: the scaled score s becomes softcap * tanh(s / softcap)
+  // Streaming kernel: a row is a token's group of up to `group` query heads of one key/value head.
+  int group = 1;
+  int rows = 0;           // rows per token
+  int rows_per_kv = 0;    // rows of a key/value head
 };
+
+constexpr int MAX_GROUP = 4;
+
+// Row `row` of a token: its key/value head, its first query head and how many it holds.
+__device__ __forceinline__ int row_kv_head(const AttentionArgs& a, int row) {
+  return row / a.rows_per_kv;
+}
+__device__ __forceinline__ int row_first_head(const AttentionArgs& a, int row) {
+  const int kv_head = row / a.rows_per_kv;
+  return kv_head * (a.heads / a.kv_heads) + (row - kv_head * a.rows_per_kv) * a.group;
+}
+__device__ __forceinline__ int row_head_count(const AttentionArgs& a, int row) {
+  return min(a.group, a.heads / a.kv_heads - (row % a.rows_per_kv) * a.group);
+}
 
 // A finished row with maximum m, weight l and unnormalised sum o, and a sink s: the result is
 // o * factor with factor = e^(m - M) / (l e^(m - M) + e^(s - M)), M = max(m, s).
@@ -424,8 +448,8 @@ __device__ __forceinline__ int chunks_of(const AttentionArgs& a, int keys) {
   return n;
 }
 
-// A place in the flat list of chunks: rows (token, head) in ascending order, the chunks of a
-// row in ascending order of their keys.
+// A place in the flat list of chunks: rows (token, group of heads; `head` counts a token's rows)
+// in ascending order, the chunks of a row in ascending order of their keys.
 struct ChunkCursor {
   int token, head, chunk;
   int n;                  // chunks in a row of this token
@@ -442,7 +466,7 @@ __device__ __forceinline__ void cursor_next(const AttentionArgs& a, ChunkCursor&
   if (++c.chunk < c.n) return;
   c.chunk = 0;
   c.row_begin += c.n;
-  if (++c.head < a.heads) return;
+  if (++c.head < a.rows) return;
   c.head = 0;
   do {
     ++c.token;
@@ -461,8 +485,9 @@ __device__ __forceinline__ void cursor_next(const AttentionArgs& a, ChunkCursor&
 // chunk in its slot 0, that of a row that begins inside its range in slot 1.  All loads of a
 // batch of 32 parts are in flight together: the merge is a few round trips to the L2.
 template <typename T, int D, int STRIDE>
-__device__ void merge_parts(const AttentionArgs& a, int token, int head, long long row_begin,
-                            long long per_warp, int first_warp, int n_parts, int lane) {
+__device__ void merge_parts(const AttentionArgs& a, int token, int head, int member,
+                            long long row_begin, long long per_warp, int first_warp, int n_parts,
+                            int lane) {
   // Coordinates per lane: four consecutive ones for a head of 128; otherwise pairs, the
   // i-th pair of a lane at coordinate 2 lane + 64 i (lanes beyond the head hold zeros).
   constexpr int MERGE_LOADS = HX_MERGE_LOADS;      // parts whose loads are in flight together
@@ -471,7 +496,7 @@ __device__ void merge_parts(const AttentionArgs& a, int token, int head, long lo
   auto part_of = [&](int index) {
     const long long w = first_warp + index;
     const int slot = row_begin <= w * per_warp ? 0 : 1;
-    return a.partial + static_cast<size_t>(w * 2 + slot) * STRIDE;
+    return a.partial + static_cast<size_t>((w * 2 + slot) * a.group + member) * STRIDE;
   };
   auto load_slice = [&](const float* part, float (&o)[PER_LANE]) {
     if constexpr (QUADS) {
@@ -592,7 +617,7 @@ void paged_attention_stream_kernel(
       mine += __shfl_xor_sync(0xffffffffu, mine, offset);
     total = mine;
   }
-  total *= a.heads;
+  total *= a.rows;
   const long long per_warp = (total + n_warps - 1) / n_warps;
   const long long my_begin = me * per_warp;
   const long long my_end = min(my_begin + per_warp, total);
@@ -618,7 +643,7 @@ void paged_attention_stream_kernel(
           if (lane >= offset) inclusive += other;
         }
       }
-      const unsigned beyond = __ballot_sync(0xffffffffu, (before + inclusive) * a.heads > my_begin);
+      const unsigned beyond = __ballot_sync(0xffffffffu, (before + inclusive) * a.rows > my_begin);
       if (beyond != 0u) {
         const int source = __ffs(beyond) - 1;
         found = base + source;
@@ -632,7 +657,7 @@ void paged_attention_stream_kernel(
       }
     }
     at.token = found;
-    const long long inside = my_begin - before * a.heads;
+    const long long inside = my_begin - before * a.rows;
     at.head = static_cast<int>(inside / at.n);
     at.chunk = static_cast<int>(inside - static_cast<long long>(at.head) * at.n);
     at.row_begin = my_begin - at.chunk;
@@ -642,7 +667,6 @@ void paged_attention_stream_kernel(
   const int page_size = a.page_size;
   const int pages_per_chunk = KEYS / page_size;
   const uint32_t page_bytes = static_cast<uint32_t>(page_size) * D * 2;
-  const int heads_per_kv = a.heads / a.kv_heads;
   const uint8_t* k_cache = static_cast<const uint8_t*>(a.k_cache);
   const uint8_t* v_cache = static_cast<const uint8_t*>(a.v_cache);
   uint8_t* ring = stream_shared + static_cast<size_t>(warp) * RING * Config::kSlotBytes;
@@ -678,7 +702,7 @@ void paged_attention_stream_kernel(
     }
     uint8_t* slot_base = ring + static_cast<size_t>(slot) * Config::kSlotBytes;
     uint64_t* bar = &bars[slot];
-    const int kv_head = ahead.head / heads_per_kv;
+    const int kv_head = row_kv_head(a, ahead.head);
     int pages[kMaxPages];
     uint32_t expected = 0;
     unsigned bits = 0u;
@@ -739,9 +763,12 @@ void paged_attention_stream_kernel(
 
   // Both products put the cache on the 16-row side of the tensor-core tile, where none of it
   // is wasted, and the single query (or probability) vector on the 8-column side:
-  //   scores  S[16 keys x 8]  = K[16 keys x 16 d] q[16 d x 8]      (all 8 columns equal)
-  //   output  O[16 d x 8]    += V^T[16 d x 16 keys] P[16 keys x 8]  (column 0: hi part of the
-  //                                                    probabilities, column 1: lo part)
+  //   scores  S[16 keys x 8]  = K[16 keys x 16 d] q[16 d x 8]      (columns 2 h, 2 h + 1: the
+  //                                                    row's h-th head; one head: all equal)
+  //   output  O[16 d x 8]    += V^T[16 d x 16 keys] P[16 keys x 8]  (column 2 h: hi part of the
+  //                                                    probabilities, column 2 h + 1: lo part)
+  // so a lane's own head is the quad-th of the row, in the scores, the running sums and the
+  // output alike.
   // Where this lane's ldmatrix rows sit inside a slot half never changes from chunk to
   // chunk: work the offsets out once.  Keys (plain load): matrices (keys 0-7, d lo),
   // (keys 8-15, d lo), (keys 0-7, d hi), (keys 8-15, d hi) of a 16-key tile; values
@@ -760,9 +787,10 @@ void paged_attention_stream_kernel(
   }
 
   uint32_t q_frag[kDSteps][2];       // the query as B operand: d 16k + 2 quad (+8), +1
-  float o_acc[kDTiles][4];           // lanes with quad 0: d 16m + group (c0 hi, c1 lo), +8 (c2, c3)
+  float o_acc[kDTiles][4];           // head quad: d 16m + group (c0 hi, c1 lo), +8 (c2, c3)
   float running_max = -INFINITY;
   float running_sum = 0.0f;          // over this lane's own keys; lanes of a group hold copies
+  int row_head = 0, row_heads = 1;   // the row's first head and how many it holds
 #pragma unroll
   for (int k = 0; k < kDSteps; ++k) q_frag[k][0] = q_frag[k][1] = 0u;
 
@@ -770,8 +798,10 @@ void paged_attention_stream_kernel(
     const int slot = static_cast<int>(i % RING);
     if (i == 0 || at.chunk == 0) {
       // a row begins (or goes on from another warp's run): its query, an empty sum
+      row_head = row_first_head(a, at.head);
+      row_heads = row_head_count(a, at.head);
       const T* q = static_cast<const T*>(a.q) + static_cast<size_t>(at.token) * a.ldq +
-                   static_cast<size_t>(at.head) * D + 2 * quad;
+                   static_cast<size_t>(row_head + min(group >> 1, row_heads - 1)) * D + 2 * quad;
 #pragma unroll
       for (int k = 0; k < kDSteps; ++k) {
         q_frag[k][0] = *reinterpret_cast<const uint32_t*>(q + k * 16);
@@ -849,7 +879,7 @@ void paged_attention_stream_kernel(
     }
     if (a.slopes != nullptr) {
       // the distance from the row's own position (at.keys - 1) to key group + 8 j of the chunk
-      const float slope = a.slopes[at.head];
+      const float slope = a.slopes[row_head + min(quad, row_heads - 1)];
       const int distance0 = at.keys - 1 - block_key0 - group;
 #pragma unroll
       for (int j = 0; j < 2 * kTiles; ++j)
@@ -872,8 +902,10 @@ void paged_attention_stream_kernel(
     chunk_max = fmaxf(chunk_max, __shfl_xor_sync(0xffffffffu, chunk_max, 8));
     chunk_max = fmaxf(chunk_max, __shfl_xor_sync(0xffffffffu, chunk_max, 16));
     const float new_max = fmaxf(running_max, chunk_max);
-    if (new_max != -INFINITY) {
-      if (new_max != running_max) {      // the same in every lane
+    // (the heads of a row see the same keys, but the branch must be the warp's)
+    if (__any_sync(0xffffffffu, new_max != -INFINITY)) {
+      const float reference = new_max == -INFINITY ? 0.0f : new_max;
+      if (new_max != running_max) {      // the same in every lane of a head
         const float correction = running_max == -INFINITY ? 0.0f : __expf(running_max - new_max);
         running_max = new_max;
         running_sum *= correction;
@@ -886,7 +918,7 @@ void paged_attention_stream_kernel(
       uint32_t split[2 * kTiles];
 #pragma unroll
       for (int j = 0; j < 2 * kTiles; ++j) {
-        const float x = __expf(score[j] - new_max);
+        const float x = __expf(score[j] - reference);
         running_sum += x;
         const __nv_bfloat16 hi = __float2bfloat16_rn(x);
         const __nv_bfloat16 lo = __float2bfloat16_rn(x - __bfloat162float(hi));
@@ -895,9 +927,8 @@ void paged_attention_stream_kernel(
       }
       // ---- o += V^T p.  The B operand wants, in this lane, keys 2 quad, 2 quad + 1 (b0) and
       // 8 more (b1) of each tile: they sit in the lanes of groups 2 quad and 2 quad + 1.
-      // Even columns (group even) take the hi parts, odd columns the lo parts; only columns
-      // 0 and 1 are read back.
-      const int source = 8 * quad;                         // first lane of group 2 quad
+      // Even columns (group even) take the hi parts of head group / 2, odd columns the lo parts.
+      const int source = 8 * quad + (group >> 1);          // that head's lane of group 2 quad
       const uint32_t pick = (group & 1) ? 0x7632u : 0x5410u;      // lo halves : hi halves
 #pragma unroll
       for (int tile = 0; tile < kTiles; ++tile) {
@@ -932,10 +963,10 @@ void paged_attention_stream_kernel(
       row_sum += __shfl_xor_sync(0xffffffffu, row_sum, 16);
       const long long row_end = at.row_begin + at.n;
       if (at.row_begin >= my_begin && row_end <= my_end) {
-        if (quad == 0) {
-          const float inverse = sink_inverse(a, at.head, running_max, row_sum);
+        if (quad < row_heads) {
+          const float inverse = sink_inverse(a, row_head + quad, running_max, row_sum);
           T* out = static_cast<T*>(a.out) + static_cast<size_t>(at.token) * a.ldo +
-                   static_cast<size_t>(at.head) * D + group;
+                   static_cast<size_t>(row_head + quad) * D + group;
 #pragma unroll
           for (int m = 0; m < kDTiles; ++m) {
             out[m * 16] = __float2bfloat16_rn((o_acc[m][0] + o_acc[m][1]) * inverse);
@@ -944,28 +975,30 @@ void paged_attention_stream_kernel(
         }
       } else {
         const int my_slot = at.row_begin <= my_begin ? 0 : 1;
-        float* part = a.partial + static_cast<size_t>(me * 2 + my_slot) * Config::kPartStride;
-        if (quad == 0) {
+        if (quad < row_heads) {
+          float* part = a.partial +
+                        static_cast<size_t>((me * 2 + my_slot) * a.group + quad) * Config::kPartStride;
 #pragma unroll
           for (int m = 0; m < kDTiles; ++m) {
             part[m * 16 + group] = o_acc[m][0] + o_acc[m][1];
             part[m * 16 + group + 8] = o_acc[m][2] + o_acc[m][3];
           }
+          if (group == 0) *reinterpret_cast<float2*>(part + D) = make_float2(running_max, row_sum);
         }
-        if (lane == 0) *reinterpret_cast<float2*>(part + D) = make_float2(running_max, row_sum);
         __threadfence();
         __syncwarp();
         const int first_warp = static_cast<int>(at.row_begin / per_warp);
         const int n_parts = static_cast<int>((row_end - 1) / per_warp) - first_warp + 1;
-        const long long counter = static_cast<long long>(at.token) * a.heads + at.head;
+        const long long counter = static_cast<long long>(at.token) * a.rows + at.head;
         int arrived_count = 0;
         if (lane == 0) arrived_count = atomicAdd(a.arrivals + counter, 1);
         arrived_count = __shfl_sync(0xffffffffu, arrived_count, 0);
         if (arrived_count == n_parts - 1) {
           __threadfence();
           if (lane == 0) a.arrivals[counter] = 0;      // ready for the next call
-          merge_parts<T, D, Config::kPartStride>(a, at.token, at.head, at.row_begin, per_warp,
-                                                 first_warp, n_parts, lane);
+          for (int member = 0; member < row_heads; ++member)
+            merge_parts<T, D, Config::kPartStride>(a, at.token, row_head + member, member,
+                                                   at.row_begin, per_warp, first_warp, n_parts, lane);
         }
       }
     }
@@ -1002,7 +1035,7 @@ int launch_stream(const AttentionArgs& a, cudaStream_t stream) {
   }
   // one warp per chunk at most (the bound on chunks comes from the caller's split sizes)
   const long long chunk_bound =
-      static_cast<long long>(a.tokens) * a.heads *
+      static_cast<long long>(a.tokens) * a.rows *
       ((static_cast<long long>(a.split_keys) * a.max_splits + KEYS - 1) / KEYS);
   const long long warps = min(static_cast<long long>(resident_warps[device]), max(1ll, chunk_bound));
   const int blocks = static_cast<int>((warps + STREAM_WARPS - 1) / STREAM_WARPS);
@@ -1096,10 +1129,21 @@ HX_API long long hx_paged_attention_scratch_floats_for(int dtype, int tokens, in
   return hx_paged_attention_scratch_floats(tokens, heads, head_dim, max_splits);
 }
 
+// ... and for a caller that lets the streaming kernel take up to four query heads of a key/value
+// head at a time (hx_paged_attention_biased with group_heads != 0); 0: that kernel does not apply.
+HX_API long long hx_paged_attention_group_scratch_floats(int dtype, int head_dim, int page_size) {
+  AttentionArgs a{};
+  a.head_dim = head_dim;
+  a.page_size = page_size;
+  return stream_kernel_applies(a, dtype) ? 2ll * STREAM_MAX_WARPS * MAX_GROUP * (head_dim + 4) : 0;
+}
+
 // hx_paged_attention with kept first keys: a row at position p sees key j <= p when
 // p - j < window or j < keep_first (window 0: every earlier key, keep_first is then unused).
 // ... and with the optional per-head sinks and distance slopes (null: none), chunks (0: none)
-// and a level the scores run into (0: none); see AttentionArgs.
+// and a level the scores run into (0: none); see AttentionArgs.  group_heads != 0: where the
+// streaming kernel runs it takes the query heads of a key/value head up to four at a time
+// (`partial` then holds hx_paged_attention_group_scratch_floats() floats).
 HX_API int hx_paged_attention_biased(const void* q, int ldq, const void* k_cache,
                                      const void* v_cache, int dtype, const int* positions,
                                      const int* token_request, const int* request_table_row,
@@ -1109,7 +1153,8 @@ HX_API int hx_paged_attention_biased(const void* q, int ldq, const void* k_cache
                                      int kv_heads, int head_dim, int page_size, int num_pages,
                                      int window, int keep_first, float scale, int split_keys,
                                      int max_splits, const float* sinks, const float* slopes,
-                                     int chunk, float softcap, int* status, cudaStream_t stream) {
+                                     int chunk, float softcap, int group_heads, int* status,
+                                     cudaStream_t stream) {
   HX_REQUIRE(chunk >= 0 && softcap >= 0.0f, "hx_paged_attention: bad chunk or softcap");
   HX_REQUIRE(keep_first >= 0, "hx_paged_attention: keep_first must not be negative");
   if (window == 0) keep_first = 0;
@@ -1132,6 +1177,10 @@ HX_API int hx_paged_attention_biased(const void* q, int ldq, const void* k_cache
                   arrivals, tokens, heads, kv_heads, head_dim, page_size, num_pages, window,
                   keep_first, scale, split_keys, max_splits, status, sinks, slopes, chunk,
                   softcap};
+  const int share = heads / kv_heads;
+  if (group_heads) a.group = share < MAX_GROUP ? share : MAX_GROUP;
+  a.rows_per_kv = (share + a.group - 1) / a.group;
+  a.rows = kv_heads * a.rows_per_kv;
   const long long items = static_cast<long long>(tokens) * heads * max_splits;
   HX_REQUIRE(items / STREAM_WARPS < (1ll << 31) - 1, "hx_paged_attention: grid too large");
   int rc;
@@ -1160,8 +1209,8 @@ HX_API int hx_paged_attention_kept(const void* q, int ldq, const void* k_cache, 
                                    request_table_row, block_tables, table_stride, request_start,
                                    skip_query_len, out, ldo, partial, arrivals, tokens, heads,
                                    kv_heads, head_dim, page_size, num_pages, window, keep_first,
-                                   scale, split_keys, max_splits, nullptr, nullptr, 0, 0.0f, status,
-                                   stream);
+                                   scale, split_keys, max_splits, nullptr, nullptr, 0, 0.0f, 0,
+                                   status, stream);
 }
 
 HX_API int hx_paged_attention(const void* q, int ldq, const void* k_cache, const void* v_cache,

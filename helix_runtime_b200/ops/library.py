@@ -248,7 +248,10 @@ def _declare(library: ctypes.CDLL) -> None:
     library.hx_paged_attention_biased.argtypes = [
         _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr,
         _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-        _c_int, _c_int, _c_float, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_float, _c_ptr, _c_ptr]
+        _c_int, _c_int, _c_float, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_float, _c_int, _c_ptr,
+        _c_ptr]
+    library.hx_paged_attention_group_scratch_floats.argtypes = [_c_int] * 3
+    library.hx_paged_attention_group_scratch_floats.restype = _c_longlong
     library.hx_prefill_attention_biased.argtypes = [
         *library.hx_prefill_attention_windowed.argtypes[:-2], _c_int, _c_ptr, _c_ptr, _c_int,
         _c_float, _c_ptr, _c_ptr]
@@ -647,6 +650,12 @@ def attention_scratch_floats(tokens: int, heads: int, head_dim: int, max_splits:
         dtype_code(dtype), tokens, heads, head_dim, page_size, window, max_splits))
 
 
+def attention_group_scratch_floats(dtype: torch.dtype, head_dim: int, page_size: int) -> int:
+    """Floats of scratch ``paged_attention`` with ``group_heads`` needs; 0 where the streaming kernel
+    does not apply."""
+    return int(lib().hx_paged_attention_group_scratch_floats(dtype_code(dtype), head_dim, page_size))
+
+
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                     positions: torch.Tensor, token_request: torch.Tensor,
                     request_table_row: torch.Tensor, block_tables: torch.Tensor, out: torch.Tensor,
@@ -657,7 +666,7 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                     arrivals: Optional[torch.Tensor] = None, keep_first: int = 0,
                     sinks: Optional[torch.Tensor] = None,
                     slopes: Optional[torch.Tensor] = None, chunk: int = 0,
-                    softcap: float = 0.0) -> None:
+                    softcap: float = 0.0, group_heads: bool = False) -> None:
     """out[t, h*D:(h+1)*D] = attention of query (t, h) over its request's pages.  With
     ``skip_query_len > 0`` tokens of requests that bring at least that many tokens are left
     out (the tensor-core kernel takes them).  With a window, keys at positions below
@@ -668,7 +677,9 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     ``exp(sinks[h])``, a term without key or value.  ``slopes`` (float32 ``[heads]``): the score
     of key ``j`` for the query at position ``i`` is lowered by ``slopes[h] * (i - j)``.
     ``chunk`` > 0: position ``i`` sees ``j`` only when ``i // chunk == j // chunk``.  ``softcap`` >
-    0: the scaled score ``s`` becomes ``softcap * tanh(s / softcap)``."""
+    0: the scaled score ``s`` becomes ``softcap * tanh(s / softcap)``.  ``group_heads``: where the
+    streaming kernel runs it takes the query heads of a key/value head up to four at a time
+    (``partial`` as large as :func:`attention_group_scratch_floats` says)."""
     for per_head in (sinks, slopes):
         if per_head is not None:
             _need(per_head, torch.float32, "sinks and slopes")
@@ -676,9 +687,11 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     if arrivals is None:
         arrivals = torch.zeros(max(1, tokens * heads), dtype=torch.int32, device=q.device)
     if partial is None:
-        partial = torch.empty(attention_scratch_floats(tokens, heads, head_dim, max_splits,
-                                                       q.dtype, page_size, window),
-                              dtype=torch.float32, device=q.device)
+        floats = attention_scratch_floats(tokens, heads, head_dim, max_splits, q.dtype, page_size,
+                                          window)
+        if group_heads:
+            floats = max(floats, attention_group_scratch_floats(q.dtype, head_dim, page_size))
+        partial = torch.empty(floats, dtype=torch.float32, device=q.device)
     _check(lib().hx_paged_attention_biased(
         q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), dtype_code(q.dtype),
         positions.data_ptr(), token_request.data_ptr(), request_table_row.data_ptr(),
@@ -686,7 +699,7 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         out.data_ptr(), out.stride(0),
         _ptr(partial), _ptr(arrivals), tokens, heads, kv_heads, head_dim, page_size, num_pages, window,
         int(keep_first), float(scale), split_keys, max_splits, _ptr(sinks), _ptr(slopes),
-        int(chunk), float(softcap), _ptr(status), _stream()))
+        int(chunk), float(softcap), 1 if group_heads else 0, _ptr(status), _stream()))
 
 
 PREFILL_TILE_ROWS = 64        # query rows of a CTA of the ``mma.sync`` prompt kernel

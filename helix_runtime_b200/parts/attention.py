@@ -132,7 +132,7 @@ class PagedAttention(Mixer):
             if self.value_dim != self.head_dim or self.conv_taps > 1 or self.gated:
                 raise ValueError("values that are the keys have the keys' size, and neither a "
                                  "filter nor an output gate beside them")
-            # query heads that share a key/value head decode side by side in a tile's rows
+            # query heads that share a key/value head decode side by side
             self.pack_heads = self.heads // self.kv_heads >= 2
             self.pack_always = False
         self.row_dim = self.head_dim
@@ -358,8 +358,13 @@ class PagedAttention(Mixer):
                         and ops.prefill_attention_supports(self.row_dim, cache.page_size))
         # many heads on one cached row: the kernel whose rows are a token's heads reads the
         # row once for all of them, decoded tokens included
+        # (without pack_always, single tokens are the streaming kernel's wherever it applies: it
+        # takes up to four heads of a key/value head at a time and shares long contexts out)
+        group_floats = ops.attention_group_scratch_floats(ctx.dtype, self.row_dim, cache.page_size) \
+            if self.heads > self.kv_heads else 0
         if (self.pack_heads and ctx.dtype == torch.bfloat16
-                and (self.pack_always or ctx.max_query_len < TENSOR_CORE_MIN_QUERY)
+                and (self.pack_always or (ctx.max_query_len < TENSOR_CORE_MIN_QUERY
+                                          and not group_floats))
                 and ops.prefill_attention_supports(self.row_dim, cache.page_size)
                 and ops.prefill_attention_packed_tokens(self.heads, self.kv_heads) > 0):
             ops.prefill_attention(qkv, cache.keys, cache.values, ctx.request_start,
@@ -389,7 +394,8 @@ class PagedAttention(Mixer):
             max_splits = max(1, -(-longest // split_keys))
             floats = ops.attention_scratch_floats(n, self.heads, self.row_dim, max_splits,
                                                   ctx.dtype, cache.page_size, window)
-            partial = ctx.workspace.at_least("attention.partial", floats, torch.float32)
+            partial = ctx.workspace.at_least("attention.partial", max(floats, group_floats),
+                                             torch.float32)
             arrivals = ctx.workspace.accumulator(f"attention.arrivals/{self.heads}",
                                                  (ctx.capacity * self.heads,), torch.int32)
             ops.paged_attention(qkv, cache.keys, cache.values, ctx.positions, ctx.token_request,
@@ -399,7 +405,8 @@ class PagedAttention(Mixer):
                                 ctx.status, request_start=ctx.request_start,
                                 skip_query_len=TENSOR_CORE_MIN_QUERY if tensor_cores else 0,
                                 arrivals=arrivals, keep_first=kept, sinks=self.sinks,
-                                slopes=self.slopes, chunk=chunk, softcap=self.softcap)
+                                slopes=self.slopes, chunk=chunk, softcap=self.softcap,
+                                group_heads=group_floats > 0)
 
     def forward(self, ctx: StepContext, cache: LayerCache, x: torch.Tensor,
                 residual: torch.Tensor) -> None:
@@ -480,9 +487,8 @@ class NormedProjectionAttention(PagedAttention):
         if self.conv_taps > 1:
             raise ValueError("this part has no filter over time")
         self.spec = spec
-        # decoding: query heads that share a key/value head attend side by side in a tile's
-        # rows (the streaming kernel would read the shared keys once per query head); steps
-        # with prompt portions keep the kernels every attention part uses
+        # decoding: query heads that share a key/value head attend side by side, four at a time
+        # in the streaming kernel or, for page sizes it does not take, in a tile's rows
         self.pack_heads = self.heads // self.kv_heads >= 2
         self.pack_always = False
         self.head_gated = gate is not None

@@ -468,7 +468,10 @@ int hx_paged_attention_kept(const void* q, int ldq, const void* k_cache, const v
    denominator also holds exp(sinks[h]), a term without key or value; slopes: the score of key j
    for the query at position i is lowered by slopes[h] * (i - j); chunk > 0: position i sees j
    only when i / chunk == j / chunk; softcap > 0: the scaled score s becomes softcap * tanh(s /
-   softcap), before slopes and mask */
+   softcap), before slopes and mask.  group_heads != 0: the streaming kernel takes the query heads
+   of a key/value head up to four at a time; `partial` then holds group_scratch_floats() floats
+   (0: that kernel does not apply, and the flag changes nothing) */
+long long hx_paged_attention_group_scratch_floats(int dtype, int head_dim, int page_size);
 int hx_paged_attention_biased(const void* q, int ldq, const void* k_cache, const void* v_cache,
                               int dtype, const int* positions, const int* token_request,
                               const int* request_table_row, const int* block_tables,
@@ -477,7 +480,8 @@ int hx_paged_attention_biased(const void* q, int ldq, const void* k_cache, const
                               int heads, int kv_heads, int head_dim, int page_size, int num_pages,
                               int window, int keep_first, float scale, int split_keys,
                               int max_splits, const float* sinks, const float* slopes,
-                              int chunk, float softcap, int* status, cudaStream_t stream);
+                              int chunk, float softcap, int group_heads, int* status,
+                              cudaStream_t stream);
 /* the same with scratch built into the library: see hx_no_alloc.h beside the sources */
 int hx_paged_attention_no_alloc(const void* q, int ldq, const void* k_cache, const void* v_cache,
                                 int dtype, const int* positions, const int* token_request,

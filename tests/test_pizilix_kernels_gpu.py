@@ -73,7 +73,7 @@ def attention_case(rng, dtype, kernel, heads, kv_heads, head_dim, page_size, con
         ops.paged_attention(*common, dev(np.arange(context, total), torch.int32),
                             dev(np.zeros(new), torch.int32), slots, dev(tables, torch.int32), out,
                             None, new, heads, kv_heads, head_dim, page_size, num_pages, 0, scale,
-                            split_keys, max(1, -(-longest // split_keys)), status, **options)
+                            split_keys, max(1, -(-longest // split_keys)), status, group_heads=kernel == "grouped", **options)
     assert int(status.item()) == 0
     padded = np.concatenate([np.zeros((context, heads, head_dim)), queries])
     expected = plain.chunked_attention(padded, keys, values, scale, cap, chunk, sink)[context:]
@@ -85,7 +85,7 @@ def attention_case(rng, dtype, kernel, heads, kv_heads, head_dim, page_size, con
 @pytest.mark.parametrize("cap", [None, 2.0])
 def test_chunks_and_levels_in_portions_and_decoding(dtype, kernel, chunk, cap):
     rng = np.random.default_rng(27)
-    heads, kv_heads = (6, 2) if kernel != "packed" else (6, 1)
+    heads, kv_heads = {"packed": (6, 1), "grouped": (14, 2)}.get(kernel, (6, 2))
     for context, new in [(0, 150), (37, 90), (63, 1), (64, 1), (139, 1), (140, 1), (210, 17),
                          (15, 1), (0, 1), (100, 23), (250, 300)]:
         if kernel == "tcgen05" and new == 1:
@@ -152,6 +152,55 @@ def test_a_far_key_among_hundreds_of_its_chunk():
                                                1020 - new, new, 600, 100.0, dominant=(new - 1, 603))
             close(got, want, what=f"{kernel} new {new}", **bounds(dtype))
             assert np.abs(got[-1] - values[603, 0][None, :]).max() < 3e-2
+
+
+@pytest.mark.parametrize("heads,kv_heads", [(5, 1), (8, 4), (12, 3), (4, 4), (9, 1)])
+@pytest.mark.parametrize("chunk", [0, 300])
+def test_decoding_requests_of_very_different_lengths_in_groups_of_heads(heads, kv_heads, chunk):
+    """One token of each of twelve requests: rows are cut between warps anywhere."""
+    from helix_runtime_b200.ops import library as ops
+    rng = np.random.default_rng(heads + chunk)
+    dtype, head_dim, page_size, cap = torch.bfloat16, 64, 16, 3.0
+    positions = np.array([0, 1, 15, 16, 31, 299, 300, 301, 640, 1499, 7, 900])
+    count = len(positions)
+    pages = [int(p) // page_size + 1 for p in positions]
+    num_pages = sum(pages) + 2
+    order = list(rng.permutation(num_pages))
+    tables = np.full((count, max(pages)), -1, dtype=np.int32)
+    k_cache = np.full((num_pages, kv_heads, page_size, head_dim), np.nan, dtype=np.float32)
+    v_cache = np.full_like(k_cache, np.nan)
+    queries = held(rng.normal(size=(count, heads, head_dim)), dtype)
+    want, scale = [], 1.5 / math.sqrt(head_dim)
+    for request, position in enumerate(positions):
+        keys, values = (held(rng.normal(size=(position + 1, kv_heads, head_dim)), dtype)
+                        for _ in range(2))
+        for p in range(pages[request]):
+            lo, hi = p * page_size, min((p + 1) * page_size, position + 1)
+            if chunk and hi <= position // chunk * chunk:
+                continue
+            page = tables[request, p] = order.pop()
+            k_cache[page, :, :hi - lo] = keys[lo:hi].transpose(1, 0, 2)
+            v_cache[page, :, :hi - lo] = values[lo:hi].transpose(1, 0, 2)
+        first = position // chunk * chunk if chunk else 0
+        padded = np.concatenate([np.zeros((position - first, heads, head_dim)),
+                                 queries[request:request + 1]])
+        want.append(plain.chunked_attention(padded, keys[first:], values[first:], scale, cap,
+                                            None)[-1])
+    out = torch.full((count, heads * head_dim), float("nan"), dtype=dtype, device="cuda")
+    arrivals = torch.zeros(count * heads, dtype=torch.int32, device="cuda")
+    status = status_word()
+    for repeat in range(2):       # the second call finds the counters as the first left them
+        ops.paged_attention(dev(queries.reshape(count, -1), dtype),
+                            dev(to_cache_layout(k_cache, dtype), dtype),
+                            dev(to_cache_layout(v_cache, dtype), dtype),
+                            dev(positions, torch.int32), dev(np.arange(count), torch.int32),
+                            dev(np.arange(count), torch.int32), dev(tables, torch.int32), out, None,
+                            count, heads, kv_heads, head_dim, page_size, num_pages, 0, scale, 32, 48,
+                            status, arrivals=arrivals, sinks=device_tensor(np.zeros(heads)),
+                            chunk=chunk, softcap=cap, group_heads=True)
+        assert int(status.item()) == 0 and not arrivals.any()
+        close(host(out).reshape(count, heads, head_dim), np.stack(want), what="decoded",
+              **bounds(dtype))
 
 
 # ------------------------------------------------------------ rotation, values from the keys

@@ -99,7 +99,7 @@ def attention_case(rng, dtype, kernel, heads, kv_heads, head_dim, page_size, con
                             dev(np.zeros(new), torch.int32), slots, dev(tables, torch.int32), out,
                             None, new, heads, kv_heads, head_dim, page_size, num_pages,
                             window or 0, scale, split_keys, max_splits, status, sinks=sink_t,
-                            slopes=slope_t)
+                            slopes=slope_t, group_heads=kernel == "grouped")
     assert int(status.item()) == 0
     spread = np.arange(heads) // share
     expected = plain.sink_softmax_attention(
@@ -109,10 +109,11 @@ def attention_case(rng, dtype, kernel, heads, kv_heads, head_dim, page_size, con
     return host(out).reshape(new, heads, head_dim), expected, values
 
 
-# CUDA cores (float32), the streaming kernel (bfloat16), the ``mma.sync`` kernel with a head per
-# tile and with a token's heads per tile, the tcgen05 kernel (prompt portions only)
-KERNELS = [(torch.float32, "paged"), (torch.bfloat16, "paged"), (torch.bfloat16, "mma"),
-           (torch.bfloat16, "packed"), (torch.bfloat16, "tcgen05")]
+# CUDA cores (float32), the streaming kernel (bfloat16) with a head and with up to four per row,
+# the ``mma.sync`` kernel with a head per tile and with a token's heads per tile, the tcgen05
+# kernel (prompt portions only)
+KERNELS = [(torch.float32, "paged"), (torch.bfloat16, "paged"), (torch.bfloat16, "grouped"),
+           (torch.bfloat16, "mma"), (torch.bfloat16, "packed"), (torch.bfloat16, "tcgen05")]
 
 
 def sizes_for(kernel):
@@ -129,7 +130,7 @@ def bounds(dtype):
 @pytest.mark.parametrize("terms", ["sinks", "slopes", "both"])
 def test_sinks_and_slopes_in_portions_and_decoding(dtype, kernel, window, terms):
     rng = np.random.default_rng(17)
-    heads, kv_heads = (6, 2) if kernel != "packed" else (6, 1)
+    heads, kv_heads = {"packed": (6, 1), "grouped": (14, 2)}.get(kernel, (6, 2))
     sinks = rng.normal(size=heads) * 2.0 + 1.0 if terms != "slopes" else None
     slopes = 2.0 ** (-6.0 * (np.arange(heads) + 1) / heads) if terms != "sinks" else None
     for context, new in [(0, 150), (37, 90), (210, 17), (129, 1), (15, 1), (0, 1), (100, 23),
