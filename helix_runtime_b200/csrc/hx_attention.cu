@@ -485,9 +485,8 @@ __device__ __forceinline__ void cursor_next(const AttentionArgs& a, ChunkCursor&
 // chunk in its slot 0, that of a row that begins inside its range in slot 1.  All loads of a
 // batch of 32 parts are in flight together: the merge is a few round trips to the L2.
 template <typename T, int D, int STRIDE>
-__device__ void merge_parts(const AttentionArgs& a, int token, int head, int member,
-                            long long row_begin, long long per_warp, int first_warp, int n_parts,
-                            int lane) {
+__device__ void merge_parts(const AttentionArgs& a, int token, int head, long long row_begin,
+                            long long per_warp, int first_warp, int n_parts, int lane) {
   // Coordinates per lane: four consecutive ones for a head of 128; otherwise pairs, the
   // i-th pair of a lane at coordinate 2 lane + 64 i (lanes beyond the head hold zeros).
   constexpr int MERGE_LOADS = HX_MERGE_LOADS;      // parts whose loads are in flight together
@@ -496,7 +495,7 @@ __device__ void merge_parts(const AttentionArgs& a, int token, int head, int mem
   auto part_of = [&](int index) {
     const long long w = first_warp + index;
     const int slot = row_begin <= w * per_warp ? 0 : 1;
-    return a.partial + static_cast<size_t>((w * 2 + slot) * a.group + member) * STRIDE;
+    return a.partial + static_cast<size_t>(w * 2 + slot) * STRIDE;
   };
   auto load_slice = [&](const float* part, float (&o)[PER_LANE]) {
     if constexpr (QUADS) {
@@ -562,6 +561,93 @@ __device__ void merge_parts(const AttentionArgs& a, int token, int head, int mem
     if (d < D)
       *reinterpret_cast<__nv_bfloat162*>(out + d) =
           __floats2bfloat162_rn(acc[i] * inverse, acc[i + 1] * inverse);
+  }
+}
+
+// The same for a row of several heads, all of them at once: eight lanes per head, coordinates
+// 4 (lane % 8) + 32 j.  One round trip to the L2 then serves every head of the row.
+template <typename T, int D, int STRIDE>
+__device__ void merge_group_parts(const AttentionArgs& a, int token, int first_head, int heads,
+                                  long long row_begin, long long per_warp, int first_warp,
+                                  int n_parts, int lane) {
+  constexpr int PIECES = (D + 31) / 32;
+  constexpr int LOADS = D == 128 ? 4 : (PIECES >= 8 ? 1 : 8 / PIECES);     // parts in flight
+  const int member = lane >> 3, own = lane & 7;
+  const bool live = member < heads;
+  auto part_of = [&](int index) {
+    const long long w = first_warp + index;
+    const int slot = row_begin <= w * per_warp ? 0 : 1;
+    return a.partial + static_cast<size_t>((w * 2 + slot) * a.group + (live ? member : 0)) * STRIDE;
+  };
+  float total_max = -INFINITY, total_sum = 0.0f;
+  float acc[PIECES][4];
+#pragma unroll
+  for (int j = 0; j < PIECES; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[j][e] = 0.0f;
+  // maximum and weight of part base + own; the next eight parts' are on their way
+  auto weight_of = [&](int index) {
+    return index < n_parts ? __ldcg(reinterpret_cast<const float2*>(part_of(index) + D))
+                           : make_float2(-INFINITY, 0.0f);
+  };
+  float2 next = weight_of(own);
+  for (int base = 0; base < n_parts; base += 8) {
+    const float2 ml = next;
+    next = weight_of(base + 8 + own);
+    float batch_max = ml.x;
+#pragma unroll
+    for (int offset = 4; offset > 0; offset >>= 1)
+      batch_max = fmaxf(batch_max, __shfl_xor_sync(0xffffffffu, batch_max, offset));
+    const float new_max = fmaxf(total_max, batch_max);
+    const float rescale = total_max == -INFINITY ? 0.0f : __expf(total_max - new_max);
+    total_max = new_max;
+    total_sum *= rescale;
+#pragma unroll
+    for (int j = 0; j < PIECES; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[j][e] *= rescale;
+    const float factor = ml.x == -INFINITY ? 0.0f : __expf(ml.x - new_max);
+    const int here = min(8, n_parts - base);
+    for (int first = 0; first < here; first += LOADS) {
+      float4 o[LOADS][PIECES];
+#pragma unroll
+      for (int u = 0; u < LOADS; ++u)
+#pragma unroll
+        for (int j = 0; j < PIECES; ++j) {
+          o[u][j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+          if (first + u < here && own * 4 + j * 32 < D)
+            o[u][j] = __ldcg(reinterpret_cast<const float4*>(part_of(base + first + u) + own * 4 + j * 32));
+        }
+#pragma unroll
+      for (int u = 0; u < LOADS; ++u) {
+        if (first + u < here) {
+          const int source = (lane & 24) + first + u;
+          const float f = __shfl_sync(0xffffffffu, factor, source);
+          total_sum = fmaf(__shfl_sync(0xffffffffu, ml.y, source), f, total_sum);
+#pragma unroll
+          for (int j = 0; j < PIECES; ++j) {
+            acc[j][0] = fmaf(o[u][j].x, f, acc[j][0]);
+            acc[j][1] = fmaf(o[u][j].y, f, acc[j][1]);
+            acc[j][2] = fmaf(o[u][j].z, f, acc[j][2]);
+            acc[j][3] = fmaf(o[u][j].w, f, acc[j][3]);
+          }
+        }
+      }
+    }
+  }
+  if (!live) return;
+  const float inverse = sink_inverse(a, first_head + member, total_max, total_sum);
+  T* out = static_cast<T*>(a.out) + static_cast<size_t>(token) * a.ldo +
+           static_cast<size_t>(first_head + member) * D;
+#pragma unroll
+  for (int j = 0; j < PIECES; ++j) {
+    const int d = own * 4 + j * 32;
+    if (d < D) {
+      *reinterpret_cast<__nv_bfloat162*>(out + d) =
+          __floats2bfloat162_rn(acc[j][0] * inverse, acc[j][1] * inverse);
+      *reinterpret_cast<__nv_bfloat162*>(out + d + 2) =
+          __floats2bfloat162_rn(acc[j][2] * inverse, acc[j][3] * inverse);
+    }
   }
 }
 
@@ -996,9 +1082,14 @@ void paged_attention_stream_kernel(
         if (arrived_count == n_parts - 1) {
           __threadfence();
           if (lane == 0) a.arrivals[counter] = 0;      // ready for the next call
-          for (int member = 0; member < row_heads; ++member)
-            merge_parts<T, D, Config::kPartStride>(a, at.token, row_head + member, member,
-                                                   at.row_begin, per_warp, first_warp, n_parts, lane);
+          if (a.group == 1) {
+            merge_parts<T, D, Config::kPartStride>(a, at.token, row_head, at.row_begin, per_warp,
+                                                   first_warp, n_parts, lane);
+          } else {
+            merge_group_parts<T, D, Config::kPartStride>(a, at.token, row_head, row_heads,
+                                                         at.row_begin, per_warp, first_warp, n_parts,
+                                                         lane);
+          }
         }
       }
     }

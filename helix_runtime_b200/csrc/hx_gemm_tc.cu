@@ -43,8 +43,7 @@ constexpr int THREADS = 192;
 
 enum Epilogue : int {
   EPI_STORE_BF16 = 0, EPI_STORE_F32 = 1, EPI_ADD_F32 = 2, EPI_SWIGLU = 3,
-  EPI_ROPE_APPEND = 4,     // persistent kernel only, see RopeArgs
-  EPI_BLOCK_GATES = 6      // persistent kernel only, see BlockGateArgs
+  EPI_ROPE_APPEND = 4      // persistent kernel only, see RopeArgs
 };
 
 // Where the [128 rows x 64 k] box of the weights that begins at row `row`, k-block `kb`, is.
@@ -364,23 +363,6 @@ struct RopeArgs {
   int shared_values;           // no v heads: the values are the keys before the rotation
 };
 
-// A block-diagonal product whose epilogue turns its sums into the decay and the push of a gated
-// linear recurrence (see hx_gated_recurrence.cu).  Block b of the channels multiplies columns
-// [b * size, (b + 1) * size) of the token rows with its own two square matrices, rows [2 b size,
-// 2 b size + size) of the weights (the recurrence gate) and the `size` rows behind them (the
-// input gate); a tile holds 128 channels of one block, both gates of a channel in one thread.
-struct BlockGateArgs {
-  const __nv_bfloat16* u;      // the token rows again: the input gate multiplies them
-  int ld_u;
-  const float* r_bias;         // [channels]
-  const float* i_bias;
-  const float* rate;
-  float* decay;                // [tokens, channels]: a - 1
-  float* push;                 // [tokens, channels]: sqrt(1 - a^2) i u
-  int size, channels;
-  int tiles;                   // 128-channel tiles of a block
-};
-
 #ifndef HX_GEMM_STREAM_K
 #define HX_GEMM_STREAM_K 1      // 0: every unit of the persistent kernel is a whole tile
 #endif
@@ -410,7 +392,6 @@ struct PersistentArgs {
   const float* gate_bias = nullptr;
   const float* up_bias = nullptr;
   float softcap = 0.0f;       // float32 store: see level_off
-  BlockGateArgs gates = BlockGateArgs{};      // EPI_BLOCK_GATES only
 };
 
 // What a CTA works on at a time: a tile, or (`partial`) a run of k-blocks of a tile that
@@ -661,49 +642,6 @@ __device__ __forceinline__ void write_row_rope(const PersistentArgs& a, uint32_t
   }
 }
 
-// The gates' epilogue for this thread's token: channels [channel0, channel0 + 128) of block
-// `block`, as far as the block has them.
-__device__ __forceinline__ void write_row_gates(const BlockGateArgs& g, uint32_t lane_address,
-                                                int token, int tokens, int block, int channel0) {
-  const bool live = token < tokens;
-  const __nv_bfloat16* u_row = g.u + static_cast<size_t>(live ? token : 0) * g.ld_u;
-#pragma unroll 1
-  for (int column = 0; column < BM; column += 16) {
-    const int left = g.size - channel0 - column;      // channels of the block from here on
-    if (left <= 0) break;                              // uniform over the warp
-    float r[16], i[16];
-    tmem_load16(lane_address + column, r);
-    tmem_load16(lane_address + BM + column, i);
-    if (!live) continue;
-    // sizes are multiples of 8, so a run of eight channels is there or not as a whole
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      if (half * 8 >= left) continue;
-      const int c = block * g.size + channel0 + column + half * 8;
-      const uint4 packed = *reinterpret_cast<const uint4*>(u_row + c);
-      const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&packed);
-      float d[8], p[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const float2 pair = __bfloat1622float2(pairs[j / 2]);
-        const float u = (j & 1) ? pair.y : pair.x;
-        const float r_gate =
-            __fdividef(1.0f, 1.0f + __expf(-(r[half * 8 + j] + __ldg(g.r_bias + c + j))));
-        const float i_gate =
-            __fdividef(1.0f, 1.0f + __expf(-(i[half * 8 + j] + __ldg(g.i_bias + c + j))));
-        d[j] = expm1f(-__ldg(g.rate + c + j) * r_gate);
-        p[j] = sqrtf(-d[j] * (2.0f + d[j])) * i_gate * u;
-      }
-      float4* decay = reinterpret_cast<float4*>(g.decay + static_cast<size_t>(token) * g.channels + c);
-      float4* push = reinterpret_cast<float4*>(g.push + static_cast<size_t>(token) * g.channels + c);
-      decay[0] = make_float4(d[0], d[1], d[2], d[3]);
-      decay[1] = make_float4(d[4], d[5], d[6], d[7]);
-      push[0] = make_float4(p[0], p[1], p[2], p[3]);
-      push[1] = make_float4(p[4], p[5], p[6], p[7]);
-    }
-  }
-}
-
 // The piece of a tile that a partial unit computed: added to the float32 output with atomic
 // adds (four values at a time where the row allows).
 __device__ __forceinline__ void add_row_atomically(float* out, int ldo, int features,
@@ -738,7 +676,7 @@ __global__ __launch_bounds__(THREADS) void gemm_tc_persistent_kernel(
   using Config = PersistentConfig;
   constexpr int STAGES = Config::kStages;
   // features of the output per tile, and where the second half of the N operand comes from
-  constexpr int FEATURES = EPI == EPI_SWIGLU || EPI == EPI_BLOCK_GATES ? BM : 2 * BM;
+  constexpr int FEATURES = EPI == EPI_SWIGLU ? BM : 2 * BM;
 
   hx_pdl_trigger();
   extern __shared__ uint8_t smem_raw[];
@@ -786,15 +724,8 @@ __global__ __launch_bounds__(THREADS) void gemm_tc_persistent_kernel(
           if (group < 0) kb_end = unit.kb_begin;
           else group_row0 = group * args.group_rows;
         }
-        int feature0 = group_row0 + unit.feature_tile * FEATURES;
-        int second_half = EPI == EPI_SWIGLU ? args.up_row_offset + feature0 : feature0 + BM;
-        int k0 = 0;      // first column of the token rows
-        if (EPI == EPI_BLOCK_GATES) {
-          const int block = unit.feature_tile / args.gates.tiles;
-          feature0 = block * 2 * args.gates.size + (unit.feature_tile - block * args.gates.tiles) * BM;
-          second_half = feature0 + args.gates.size;
-          k0 = block * args.gates.size;
-        }
+        const int feature0 = group_row0 + unit.feature_tile * FEATURES;
+        const int second_half = EPI == EPI_SWIGLU ? args.up_row_offset + feature0 : feature0 + BM;
         const int token0 = unit.token_tile * BM;
         for (int kb = unit.kb_begin; kb < kb_end; ++kb, ++fill) {
           const int s = fill % STAGES;
@@ -806,7 +737,7 @@ __global__ __launch_bounds__(THREADS) void gemm_tc_persistent_kernel(
           }
           uint8_t* stage = smem + s * Config::kStageBytes;
           mbar_expect_tx(&full_bar[s], Config::kStageBytes);
-          const int k = k0 + kb * BK;
+          const int k = kb * BK;
           tma_load_2d(stage, &map_x, &full_bar[s], k, token0);
           load_weight_box(stage + Config::kBytesA, &map_w, &full_bar[s], feature0, kb, args.k_tiles);
           load_weight_box(stage + Config::kBytesA + BM * BK * 2, &map_w, &full_bar[s], second_half,
@@ -897,11 +828,6 @@ __global__ __launch_bounds__(THREADS) void gemm_tc_persistent_kernel(
       if constexpr (EPI == EPI_ROPE_APPEND) {
         write_row_rope(args, lane_base + buffer * Config::kBufferColumns,
                        unit.token_tile * BM + quarter * 32 + lane, unit.feature_tile * FEATURES);
-      } else if constexpr (EPI == EPI_BLOCK_GATES) {
-        const int block = unit.feature_tile / args.gates.tiles;
-        write_row_gates(args.gates, lane_base + buffer * Config::kBufferColumns,
-                        unit.token_tile * BM + quarter * 32 + lane, args.tokens, block,
-                        (unit.feature_tile - block * args.gates.tiles) * BM);
       } else if (EPI == EPI_ADD_F32 && unit.partial) {
         add_row_atomically(static_cast<float*>(args.out), args.ldo, args.features,
                            lane_base + buffer * Config::kBufferColumns,
@@ -1070,9 +996,7 @@ int launch_persistent(const CUtensorMap& map_w, const CUtensorMap& map_x, Persis
     configured = true;
   }
   constexpr int kFeatures = EPI == EPI_SWIGLU ? BM : 2 * BM;
-  const int feature_tiles = EPI == EPI_BLOCK_GATES
-                                ? args.gates.channels / args.gates.size * args.gates.tiles
-                                : (args.features + kFeatures - 1) / kFeatures;
+  const int feature_tiles = (args.features + kFeatures - 1) / kFeatures;
   args.token_tiles = (args.tokens + BM - 1) / BM;
   const long long tiles = static_cast<long long>(args.token_tiles) * feature_tiles;
   HX_REQUIRE(tiles < (1ll << 30), "hx_gemm_tc: too many tiles");
@@ -1105,7 +1029,6 @@ int launch_persistent_epilogue(int epilogue, const CUtensorMap& map_w, const CUt
     case EPI_ADD_F32: return launch_persistent<EPI_ADD_F32>(map_w, map_x, args, stream);
     case EPI_SWIGLU: return launch_persistent<EPI_SWIGLU>(map_w, map_x, args, stream);
     case EPI_ROPE_APPEND: return launch_persistent<EPI_ROPE_APPEND>(map_w, map_x, args, stream);
-    case EPI_BLOCK_GATES: return launch_persistent<EPI_BLOCK_GATES>(map_w, map_x, args, stream);
     default:
       hx_set_error("hx_gemm_tc: unknown epilogue %d", epilogue);
       return HX_ERR_ARGUMENT;
@@ -1445,38 +1368,6 @@ HX_API int hx_gemm_tc_rope_append(const void* x, int ldx, int x_capacity_rows, c
                                        v_cache, cos_table, sin_table, table_positions, heads,
                                        kv_heads, head_dim, rotary_dim, page_size, num_pages, 0,
                                        status, stream);
-}
-
-// hx_block_gates (see hx_gated_recurrence.cu) on the tensor cores: bfloat16, blocks of a multiple of
-// 8 channels, rows of u [u_capacity_rows][ld_u] with ld_u a multiple of 8.
-HX_API int hx_gemm_tc_block_gates(const void* u, int ld_u, int u_capacity_rows, const void* w,
-                                  const float* r_bias, const float* i_bias, const float* rate,
-                                  float* decay, float* push, int tokens, int blocks, int size,
-                                  int* status, cudaStream_t stream) {
-  HX_REQUIRE(tokens >= 0 && blocks > 0 && size > 0 && size % 8 == 0,
-             "hx_gemm_tc_block_gates: blocks of %d channels are not supported (multiples of 8)", size);
-  HX_REQUIRE(ld_u >= blocks * size && ld_u % 8 == 0 && (reinterpret_cast<uintptr_t>(u) & 15) == 0 &&
-                 (reinterpret_cast<uintptr_t>(w) & 15) == 0 &&
-                 (reinterpret_cast<uintptr_t>(decay) & 15) == 0 &&
-                 (reinterpret_cast<uintptr_t>(push) & 15) == 0,
-             "hx_gemm_tc_block_gates: operands must be 16-byte aligned");
-  HX_REQUIRE(u_capacity_rows >= tokens, "hx_gemm_tc_block_gates: buffer rows %d < tokens %d",
-             u_capacity_rows, tokens);
-  HX_REQUIRE(r_bias && i_bias && rate && status, "hx_gemm_tc_block_gates: an operand is missing");
-  if (tokens == 0) return HX_OK;
-  CUtensorMap map_w, map_x;
-  int rc = get_tensor_map(w, static_cast<uint64_t>(blocks) * 2 * size, size, size, BM, &map_w);
-  if (rc != HX_OK) return rc;
-  rc = get_tensor_map(u, u_capacity_rows, static_cast<uint64_t>(blocks) * size, ld_u, BM, &map_x);
-  if (rc != HX_OK) return rc;
-  PersistentArgs args{nullptr, 0, tokens, 2 * blocks * size, size, 0, 0, 0, 0,
-                      (size + BK - 1) / BK, status, RopeArgs{}, -1, HX_GATE_SILU, nullptr, 0};
-  args.gates = BlockGateArgs{static_cast<const __nv_bfloat16*>(u), ld_u, r_bias, i_bias, rate, decay,
-                             push, size, blocks * size, (size + BM - 1) / BM};
-  rc = launch_persistent_epilogue(EPI_BLOCK_GATES, map_w, map_x, args, stream);
-  if (rc != HX_OK) return rc;
-  HX_CHECK_LAUNCH("hx_gemm_tc_block_gates");
-  return HX_OK;
 }
 
 // ------------------------------------------------------------ the bounded wait, by itself

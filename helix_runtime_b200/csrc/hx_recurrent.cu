@@ -169,8 +169,8 @@ __device__ __forceinline__ void filter_input8(const FilterArgs<__nv_bfloat16>& a
   }
 }
 
-template <int TAPS>
-__global__ __launch_bounds__(256) void causal_filter_pieces_kernel(const FilterArgs<__nv_bfloat16> a,
+template <int TAPS, bool SUMS>
+__global__ __launch_bounds__(256, 2) void causal_filter_pieces_kernel(const FilterArgs<__nv_bfloat16> a,
                                                                    int tokens, int run) {
   constexpr int REACH = TAPS - 1;
   hx_pdl_trigger();
@@ -183,10 +183,22 @@ __global__ __launch_bounds__(256) void causal_filter_pieces_kernel(const FilterA
   }
   // weights, biases and the step's own description do not depend on the kernel before
   float w[TAPS][8], b[8], in_bias[8];
+  {
+    // the 8 * TAPS weights of the piece are contiguous
+    float flat[8 * TAPS];
+    const float4* source = reinterpret_cast<const float4*>(a.taps_weight + static_cast<size_t>(c) * TAPS);
+#pragma unroll
+    for (int v = 0; v < 2 * TAPS; ++v) {
+      const float4 x = __ldg(source + v);
+      flat[4 * v] = x.x; flat[4 * v + 1] = x.y; flat[4 * v + 2] = x.z; flat[4 * v + 3] = x.w;
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int i = 0; i < 8; ++i) w[j][i] = flat[i * TAPS + j];
+  }
 #pragma unroll
   for (int i = 0; i < 8; ++i) {
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) w[j][i] = a.taps_weight[static_cast<size_t>(c + i) * TAPS + j];
     b[i] = a.bias != nullptr ? a.bias[c + i] : 0.0f;
     in_bias[i] = a.in_bias != nullptr ? a.in_bias[c + i] : 0.0f;
   }
@@ -194,6 +206,7 @@ __global__ __launch_bounds__(256) void causal_filter_pieces_kernel(const FilterA
   int start = a.request_start[request];
   int end = a.request_start[request + 1];
   int slot = a.request_slot[request];
+  const bool wide_state = a.state_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(a.state) & 15) == 0;
   hx_pdl_wait();
 
   auto emit = [&](int token, const float (&y)[8]) {
@@ -201,23 +214,63 @@ __global__ __launch_bounds__(256) void causal_filter_pieces_kernel(const FilterA
     __nv_bfloat162* pairs = reinterpret_cast<__nv_bfloat162*>(&packed);
 #pragma unroll
     for (int i = 0; i < 4; ++i)
-      pairs[i] = __floats2bfloat162_rn(filter_finish(y[2 * i], a.silu), filter_finish(y[2 * i + 1], a.silu));
+      pairs[i] = a.silu ? __floats2bfloat162_rn(hx_silu_fast(y[2 * i]), hx_silu_fast(y[2 * i + 1]))
+                        : __floats2bfloat162_rn(y[2 * i], y[2 * i + 1]);
     *reinterpret_cast<uint4*>(a.out + static_cast<size_t>(token) * a.ld_out + c) = packed;
   };
   // rows[j]: the inputs of batch row token - REACH + j, used only by tokens that lie at least
-  // REACH tokens into their portion (rows of another request are never used: not fetched)
-  float rows[TAPS][8];
-#pragma unroll
-  for (int j = 0; j < REACH; ++j) {
-    if (first - REACH + j >= start) {
-      filter_input8(a, first - REACH + j, c, in_bias, rows[j]);
+  // REACH tokens into their portion (rows of another request are never used: not fetched).
+  // A row of raw inputs is kept packed; sums (few tokens) are rounded into the same form.  The
+  // input bias of a row inside the portion is part of the sum's start value.
+  auto packed_input = [&](int token) {
+    if constexpr (!SUMS) {
+      return *reinterpret_cast<const uint4*>(a.raw + static_cast<size_t>(token) * a.ld_raw + c);
     } else {
-#pragma unroll
-      for (int i = 0; i < 8; ++i) rows[j][i] = 0.0f;
+      const float4* source =
+          reinterpret_cast<const float4*>(a.accum + static_cast<size_t>(token) * a.ld_accum + c);
+      const float4 lo = source[0], hi = source[1];
+      uint4 packed;
+      __nv_bfloat162* pairs = reinterpret_cast<__nv_bfloat162*>(&packed);
+      pairs[0] = __floats2bfloat162_rn(lo.x, lo.y);
+      pairs[1] = __floats2bfloat162_rn(lo.z, lo.w);
+      pairs[2] = __floats2bfloat162_rn(hi.x, hi.y);
+      pairs[3] = __floats2bfloat162_rn(hi.z, hi.w);
+      return packed;
     }
+  };
+  auto tap = [&](const uint4& packed, int j, float (&y)[8]) {
+    const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&packed);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 v = __bfloat1622float2(pairs[i]);
+      y[2 * i] = fmaf(w[j][2 * i], v.x, y[2 * i]);
+      y[2 * i + 1] = fmaf(w[j][2 * i + 1], v.y, y[2 * i + 1]);
+    }
+  };
+  float inside[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    float sum = 0.0f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) sum += w[j][i];
+    inside[i] = fmaf(sum, in_bias[i], b[i]);
   }
+  uint4 rows[TAPS];
+#pragma unroll
+  for (int j = 0; j < REACH; ++j)
+    rows[j] = first - REACH + j >= start ? packed_input(first - REACH + j) : make_uint4(0u, 0u, 0u, 0u);
+  // the next tokens' inputs are in flight while a token is worked on
+  constexpr int AHEAD = SUMS ? 1 : 4;
+  uint4 ahead[AHEAD];
+#pragma unroll
+  for (int k = 0; k < AHEAD; ++k)
+    ahead[k] = first + k < last ? packed_input(first + k) : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll 1
   for (int token = first; token < last; ++token) {
-    filter_input8(a, token, c, in_bias, rows[REACH]);
+    rows[REACH] = ahead[0];
+#pragma unroll
+    for (int k = 0; k + 1 < AHEAD; ++k) ahead[k] = ahead[k + 1];
+    if (token + AHEAD < last) ahead[AHEAD - 1] = packed_input(token + AHEAD);
     if (token >= end) {
       request = a.token_request[token];
       start = a.request_start[request];
@@ -228,63 +281,99 @@ __global__ __launch_bounds__(256) void causal_filter_pieces_kernel(const FilterA
     if (index >= REACH) {
       float y[8];
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        y[i] = b[i];
+      for (int i = 0; i < 8; ++i) y[i] = inside[i];
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) y[i] = fmaf(w[j][i], rows[j][i], y[i]);
-      }
+      for (int j = 0; j < TAPS; ++j) tap(rows[j], j, y);
       emit(token, y);
     } else if (index == 0) {
       // the portion's first token: the tokens whose filter reaches behind the portion, then
       // the new state (see the scalar kernel)
       const int count = end - start;
       float* state = a.state + static_cast<size_t>(slot) * a.state_stride + c;
-      const int behind = count < REACH ? count : REACH;
-      for (int t = 0; t < behind; ++t) {
-        float y[8];
-#pragma unroll
-        for (int i = 0; i < 8; ++i) y[i] = b[i];
-#pragma unroll
-        for (int j = 0; j < TAPS; ++j) {
-          const int place = t - REACH + j;
-          float x[8];
-          if (place >= 0) {
-            filter_input8(a, start + place, c, in_bias, x);
-          } else {
-#pragma unroll
-            for (int i = 0; i < 8; ++i)
-              x[i] = state[static_cast<size_t>(place + REACH) * a.channels + i];
-          }
-#pragma unroll
-          for (int i = 0; i < 8; ++i) y[i] = fmaf(w[j][i], x[i], y[i]);
-        }
-        emit(start + t, y);
-      }
-      for (int r = 0; r < REACH; ++r) {
-        const int place = count - REACH + r;
-        float x[8];
+      // the input at a place of the portion, or in front of it the state's
+      auto input_at = [&](int place, float (&x)[8]) {
         if (place >= 0) {
           filter_input8(a, start + place, c, in_bias, x);
+        } else if (wide_state) {
+          const float4* source = reinterpret_cast<const float4*>(
+              state + static_cast<size_t>(place + REACH) * a.channels);
+          const float4 lo = source[0], hi = source[1];
+          x[0] = lo.x; x[1] = lo.y; x[2] = lo.z; x[3] = lo.w;
+          x[4] = hi.x; x[5] = hi.y; x[6] = hi.z; x[7] = hi.w;
         } else {
 #pragma unroll
           for (int i = 0; i < 8; ++i) x[i] = state[static_cast<size_t>(place + REACH) * a.channels + i];
         }
+      };
+      if (count == 1) {
+        // a decoded token: its filter reads the state and itself, and the state moves up by one
+        float x[TAPS][8], y[8];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) state[static_cast<size_t>(r) * a.channels + i] = x[i];
+        for (int j = 0; j < TAPS; ++j) input_at(j - REACH, x[j]);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          y[i] = b[i];
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j) y[i] = fmaf(w[j][i], x[j][i], y[i]);
+        }
+        emit(token, y);
+#pragma unroll
+        for (int r = 0; r < REACH; ++r) {
+          float* target = state + static_cast<size_t>(r) * a.channels;
+          if (wide_state) {
+            reinterpret_cast<float4*>(target)[0] =
+                make_float4(x[r + 1][0], x[r + 1][1], x[r + 1][2], x[r + 1][3]);
+            reinterpret_cast<float4*>(target)[1] =
+                make_float4(x[r + 1][4], x[r + 1][5], x[r + 1][6], x[r + 1][7]);
+          } else {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) target[i] = x[r + 1][i];
+          }
+        }
+      } else {
+        const int behind = count < REACH ? count : REACH;
+        for (int t = 0; t < behind; ++t) {
+          float y[8];
+#pragma unroll
+          for (int i = 0; i < 8; ++i) y[i] = b[i];
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j) {
+            float x[8];
+            input_at(t - REACH + j, x);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) y[i] = fmaf(w[j][i], x[i], y[i]);
+          }
+          emit(start + t, y);
+        }
+        for (int r = 0; r < REACH; ++r) {
+          float x[8];
+          input_at(count - REACH + r, x);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) state[static_cast<size_t>(r) * a.channels + i] = x[i];
+        }
       }
     }
 #pragma unroll
-    for (int j = 0; j < REACH; ++j)
-#pragma unroll
-      for (int i = 0; i < 8; ++i) rows[j][i] = rows[j + 1][i];
+    for (int j = 0; j < REACH; ++j) rows[j] = rows[j + 1];
   }
 }
 
 bool filter_pieces_apply(const FilterArgs<__nv_bfloat16>& a) {
   auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   return a.taps <= FILTER_FAST_TAPS && a.channels % 8 == 0 && a.ld_out % 8 == 0 && aligned(a.out) &&
+         aligned(a.taps_weight) &&
          (a.accum != nullptr ? a.ld_accum % 4 == 0 && aligned(a.accum)
                              : a.ld_raw % 8 == 0 && aligned(a.raw));
+}
+
+template <int TAPS>
+void launch_filter_pieces(const FilterArgs<__nv_bfloat16>& a, dim3 grid, int block, int tokens, int run,
+                          bool sums, cudaStream_t stream) {
+  if (sums) {
+    hx_launch(causal_filter_pieces_kernel<TAPS, true>, grid, block, 0, stream, a, tokens, run);
+  } else {
+    hx_launch(causal_filter_pieces_kernel<TAPS, false>, grid, block, 0, stream, a, tokens, run);
+  }
 }
 
 int launch_filter(const FilterArgs<__nv_bfloat16>& a, int tokens, cudaStream_t stream) {
@@ -293,15 +382,16 @@ int launch_filter(const FilterArgs<__nv_bfloat16>& a, int tokens, cudaStream_t s
               stream, a);
     return HX_OK;
   }
-  const int run = tokens >= 1024 ? 8 : (tokens >= 256 ? 2 : 1);
+  const int run = tokens >= 1024 ? 8 : (tokens >= 256 ? 4 : 1);
   const int pieces = a.channels / 8;
   const int block = pieces >= 256 ? 256 : ((pieces + 31) / 32) * 32;
   const dim3 grid((tokens + run - 1) / run, (pieces + block - 1) / block);
+  const bool sums = a.accum != nullptr;
   switch (a.taps) {
-    case 1: hx_launch(causal_filter_pieces_kernel<1>, grid, block, 0, stream, a, tokens, run); break;
-    case 2: hx_launch(causal_filter_pieces_kernel<2>, grid, block, 0, stream, a, tokens, run); break;
-    case 3: hx_launch(causal_filter_pieces_kernel<3>, grid, block, 0, stream, a, tokens, run); break;
-    default: hx_launch(causal_filter_pieces_kernel<4>, grid, block, 0, stream, a, tokens, run); break;
+    case 1: launch_filter_pieces<1>(a, grid, block, tokens, run, sums, stream); break;
+    case 2: launch_filter_pieces<2>(a, grid, block, tokens, run, sums, stream); break;
+    case 3: launch_filter_pieces<3>(a, grid, block, tokens, run, sums, stream); break;
+    default: launch_filter_pieces<4>(a, grid, block, tokens, run, sums, stream); break;
   }
   return HX_OK;
 }

@@ -163,8 +163,12 @@ def _declare(library: ctypes.CDLL) -> None:
         _c_longlong, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr]
     library.hx_block_gates.argtypes = [_c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
                                        _c_int, _c_int, _c_int, _c_int, _c_ptr]
-    library.hx_gemm_tc_block_gates.argtypes = [_c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr,
-                                               _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr]
+    library.hx_block_gates_tiled.argtypes = [
+        _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_longlong,
+        _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr]
+    library.hx_gated_scan_tiled.argtypes = [
+        _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_longlong,
+        _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr]
     library.hx_gated_scan.argtypes = [_c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr,
                                       _c_longlong, _c_ptr, _c_int, _c_int, _c_int, _c_ptr, _c_ptr,
                                       _c_int, _c_ptr]
@@ -174,7 +178,8 @@ def _declare(library: ctypes.CDLL) -> None:
         _c_ptr, _c_longlong, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr, _c_ptr, _c_ptr]
     for name in ("hx_rope_append_shared", "hx_gemm_simt_softcapped", "hx_gemm_tc_softcapped",
                  "hx_gemm_tc_rope_append_shared", "hx_causal_filter_biased", "hx_block_gates",
-                 "hx_gemm_tc_block_gates", "hx_gated_scan", "hx_gated_recurrence_supports",
+                 "hx_block_gates_tiled", "hx_gated_scan", "hx_gated_scan_tiled",
+                 "hx_gated_recurrence_supports",
                  "hx_gated_recurrence_step"):
         getattr(library, name).restype = _c_int
     library.hx_scan_state_floats.argtypes = [_c_int, _c_int]
@@ -959,31 +964,22 @@ def _gate_operands(u, weights, r_bias, i_bias, rate):
 
 
 def gated_recurrence_supports(size: int) -> bool:
-    """Whether the tensor-core kernels take blocks of ``size`` channels (bfloat16)."""
+    """Whether the tiled kernels and the one-kernel step take blocks of ``size`` channels
+    (bfloat16)."""
     return bool(lib().hx_gated_recurrence_supports(size))
 
 
 def block_gates(u: torch.Tensor, weights: torch.Tensor, r_bias: torch.Tensor,
                 i_bias: torch.Tensor, rate: torch.Tensor, decay: torch.Tensor, push: torch.Tensor,
-                tokens: int, status: torch.Tensor, tensor_cores: Optional[bool] = None) -> None:
+                tokens: int) -> None:
     """``decay = a - 1`` and ``push = sqrt(1 - a^2) i u`` with ``log a = -rate r``: ``r`` and ``i``
     are the sigmoids of the two square matrices of every block of channels, ``weights`` ``[blocks,
     2, size, size]``, applied to the block's part of ``u`` (plus ``r_bias``, ``i_bias``).  ``decay``
-    and ``push`` float32 ``[rows, channels]``.  ``tensor_cores``: the tcgen05 kernel (default: where
-    it applies) or the CUDA-core one."""
+    and ``push`` float32 ``[rows, channels]``."""
     blocks, size = _gate_operands(u, weights, r_bias, i_bias, rate)
     for name, out in (("decay", decay), ("push", push)):
         _need(out, torch.float32, name)
         assert out.is_contiguous() and out.shape[1] == blocks * size
-    if tensor_cores is None:
-        tensor_cores = (u.dtype == torch.bfloat16 and gated_recurrence_supports(size)
-                        and u.stride(0) % 8 == 0)
-    if tensor_cores:
-        _check(lib().hx_gemm_tc_block_gates(
-            u.data_ptr(), u.stride(0), u.shape[0], weights.data_ptr(), r_bias.data_ptr(),
-            i_bias.data_ptr(), rate.data_ptr(), decay.data_ptr(), push.data_ptr(), tokens, blocks,
-            size, status.data_ptr(), _stream()))
-        return
     _check(lib().hx_block_gates(u.data_ptr(), u.stride(0), weights.data_ptr(), r_bias.data_ptr(),
                                 i_bias.data_ptr(), rate.data_ptr(), decay.data_ptr(),
                                 push.data_ptr(), dtype_code(u.dtype), tokens, blocks, size,
@@ -1014,6 +1010,57 @@ def gated_scan(decay: torch.Tensor, push: torch.Tensor, y: torch.Tensor, y_bias:
                                out.stride(0), dtype_code(out.dtype), channels,
                                request_start.data_ptr(), request_slot.data_ptr(), requests,
                                _stream()))
+
+
+RECURRENCE_TILE = 64        # tokens of a tile of the tiled kernels
+
+
+def recurrence_tiles(query_lengths: Sequence[int]) -> int:
+    """Tiles of a step whose requests bring that many tokens each."""
+    return sum(-(-length // RECURRENCE_TILE) for length in query_lengths)
+
+
+def block_gates_tiled(u: torch.Tensor, weights: torch.Tensor, r_bias: torch.Tensor,
+                      i_bias: torch.Tensor, rate: torch.Tensor, decay: torch.Tensor,
+                      push: torch.Tensor, joined: torch.Tensor, state: torch.Tensor,
+                      before: torch.Tensor, request_start: torch.Tensor,
+                      request_slot: torch.Tensor, requests: int, tiles: int) -> None:
+    """:func:`block_gates` (bfloat16, blocks :func:`gated_recurrence_supports` takes) by tiles of 64
+    tokens of each request: ``joined`` ``[>= tiles, 2 channels]`` float32 receives every tile's
+    composition and ``before`` ``[>= requests, channels]`` the states as the step finds them, both
+    for :func:`gated_scan_tiled`."""
+    blocks, size = _gate_operands(u, weights, r_bias, i_bias, rate)
+    channels = blocks * size
+    _need(u, torch.bfloat16, "u")
+    for name, tensor, width in (("decay", decay, channels), ("push", push, channels),
+                                ("joined", joined, 2 * channels), ("before", before, channels)):
+        _need(tensor, torch.float32, name)
+        assert tensor.is_contiguous() and tensor.shape[1] == width
+    assert joined.shape[0] >= tiles and before.shape[0] >= requests
+    _need(state, torch.float32, "state")
+    _check(lib().hx_block_gates_tiled(
+        u.data_ptr(), u.stride(0), weights.data_ptr(), r_bias.data_ptr(), i_bias.data_ptr(),
+        rate.data_ptr(), decay.data_ptr(), push.data_ptr(), joined.data_ptr(), state.data_ptr(),
+        state.stride(0), before.data_ptr(), blocks, size, request_start.data_ptr(),
+        request_slot.data_ptr(), requests, tiles, _stream()))
+
+
+def gated_scan_tiled(decay: torch.Tensor, push: torch.Tensor, joined: torch.Tensor,
+                     before: torch.Tensor, y: torch.Tensor, y_bias: torch.Tensor,
+                     state: torch.Tensor, out: torch.Tensor, request_start: torch.Tensor,
+                     request_slot: torch.Tensor, requests: int, tiles: int,
+                     sums: bool = False) -> None:
+    """:func:`gated_scan` behind :func:`block_gates_tiled`: all tiles run at once."""
+    channels = y_bias.numel()
+    _need(y_bias, torch.float32, "y_bias")
+    _need(state, torch.float32, "state")
+    _need(out, torch.bfloat16, "out")
+    assert decay.is_contiguous() and push.is_contiguous() and decay.shape[1] == channels
+    _check(lib().hx_gated_scan_tiled(
+        decay.data_ptr(), push.data_ptr(), joined.data_ptr(), before.data_ptr(),
+        *_other_branch(y, sums), y_bias.data_ptr(), state.data_ptr(), state.stride(0),
+        out.data_ptr(), out.stride(0), channels, request_start.data_ptr(), request_slot.data_ptr(),
+        requests, tiles, _stream()))
 
 
 def gated_recurrence_step(u: torch.Tensor, weights: torch.Tensor, r_bias: torch.Tensor,

@@ -446,7 +446,7 @@ class GatedRecurrence(Mixer):
         decay = tensors[self.names["decay"]].to(device=device, dtype=torch.float64)
         self.rate = (self.decay_rate * torch.nn.functional.softplus(decay, threshold=700.0)) \
             .to(torch.float32).contiguous()
-        self.tensor_cores = dtype == torch.bfloat16 and \
+        self.tiled = dtype == torch.bfloat16 and \
             ops.gated_recurrence_supports(self.block_size)
 
     def weight_bytes(self) -> int:
@@ -474,17 +474,27 @@ class GatedRecurrence(Mixer):
                           n, False, ctx.token_request, ctx.request_slot, ctx.request_start,
                           in_bias=self.x_bias, sums=sums)
         state = _state_piece(cache, self.filter_state, w)
-        if self.tensor_cores and n == ctx.n_requests:
+        if self.tiled and n == ctx.n_requests:
             ops.gated_recurrence_step(u, self.w_gates, self.r_bias, self.i_bias, self.rate, rows,
                                       self.y_bias, state, gated, n, ctx.token_request,
                                       ctx.request_slot, sums=sums)
         else:
             decay = get(f"gated_recurrence.decay/{w}", (ctx.capacity, w), torch.float32)
             push = get(f"gated_recurrence.push/{w}", (ctx.capacity, w), torch.float32)
-            ops.block_gates(u, self.w_gates, self.r_bias, self.i_bias, self.rate, decay, push, n,
-                            ctx.status)
-            ops.gated_scan(decay, push, rows, self.y_bias, state, gated, ctx.request_start,
-                           ctx.request_slot, ctx.n_requests, sums=sums)
+            gates = (u, self.w_gates, self.r_bias, self.i_bias, self.rate, decay, push)
+            batch = (ctx.request_start, ctx.request_slot, ctx.n_requests)
+            if self.tiled:
+                tiles = ops.recurrence_tiles(ctx.host_query_lengths)
+                most = ctx.capacity // ops.RECURRENCE_TILE + ctx.request_slot.shape[0]
+                joined = get(f"gated_recurrence.joined/{w}", (most, 2 * w), torch.float32)
+                before = get(f"gated_recurrence.before/{w}", (ctx.request_slot.shape[0], w),
+                             torch.float32)
+                ops.block_gates_tiled(*gates, joined, state, before, *batch, tiles)
+                ops.gated_scan_tiled(decay, push, joined, before, rows, self.y_bias, state, gated,
+                                     *batch, tiles, sums=sums)
+            else:
+                ops.block_gates(*gates, n)
+                ops.gated_scan(decay, push, rows, self.y_bias, state, gated, *batch, sums=sums)
         project(gated, self.w_o, residual, n, ops.EPI_ADD_F32, ctx.status, ctx.ordered_sums)
 
 

@@ -169,13 +169,22 @@ int hx_gated_scan(const float* decay, const float* push, const void* y, int ld_y
                   int ld_accum, const float* y_bias, float* state, long long state_stride,
                   void* out, int ld_out, int dtype, int channels, const int* request_start,
                   const int* request_slot, int requests, cudaStream_t stream);
-/* bfloat16, `size` a multiple of 8 (supports returns 1): the gates on tcgen05, and gates, scan and
- * output as one kernel for one token per request */
+/* bfloat16, `size` a multiple of 8 (supports returns 1): gates and scan by tiles of 64 tokens of
+ * each request that all run at once (joined [tile_bound][channels] pairs, before [requests]
+ * [channels]: scratch between the two; tile_bound: tokens / 64 + requests is enough), and gates,
+ * scan and output as one kernel for one token per request */
 int hx_gated_recurrence_supports(int size);
-int hx_gemm_tc_block_gates(const void* u, int ld_u, int u_capacity_rows, const void* w,
-                           const float* r_bias, const float* i_bias, const float* rate,
-                           float* decay, float* push, int tokens, int blocks, int size,
-                           int* status, cudaStream_t stream);
+int hx_block_gates_tiled(const void* u, int ld_u, const void* w, const float* r_bias,
+                         const float* i_bias, const float* rate, float* decay, float* push,
+                         float* joined, const float* state, long long state_stride, float* before,
+                         int blocks, int size, const int* request_start, const int* request_slot,
+                         int requests, int tile_bound, cudaStream_t stream);
+int hx_gated_scan_tiled(const float* decay, const float* push, const float* joined,
+                        const float* before, const void* y, int ld_y, float* accum, int ld_accum,
+                        const float* y_bias, float* state, long long state_stride, void* out,
+                        int ld_out, int channels, const int* request_start,
+                        const int* request_slot, int requests, int tile_bound,
+                        cudaStream_t stream);
 int hx_gated_recurrence_step(const void* u, int ld_u, const void* w, const float* r_bias,
                              const float* i_bias, const float* rate, const void* y, int ld_y,
                              float* accum, int ld_accum, const float* y_bias, float* state,

@@ -3,8 +3,8 @@
 (CUDA cores, the streaming kernel, the ``mma.sync`` kernel with a head or a token's heads per
 tile, the tcgen05 kernel), the rotation and cache append with values that are the keys (on their
 own and as the product's epilogue), the filter with a bias on its inputs, the block-diagonal gates
-on the CUDA cores and on tcgen05, the scan, the one-kernel step, and products whose sums run into
-a level.  Sizes are ones the models of the other tests do not have.
+and the scan (token by token and by tiles of tokens), the one-kernel step, and products whose
+sums run into a level.  Sizes are ones the models of the other tests do not have.
 """
 from __future__ import annotations
 
@@ -384,25 +384,35 @@ def gate_arguments(case, dtype):
             device_tensor(case["rate"]))
 
 
-BLOCKS = [(3, 8), (2, 15), (5, 24), (1, 40), (2, 72), (3, 128), (2, 200), (1, 256), (4, 1)]
+BLOCKS = [(3, 8), (2, 15), (5, 24), (1, 40), (2, 72), (3, 128), (2, 200), (1, 256), (4, 1), (1, 344)]
 
 
-@pytest.mark.parametrize("dtype,tensor_cores", [(torch.float32, False), (torch.bfloat16, False),
-                                                (torch.bfloat16, True)])
+@pytest.mark.parametrize("dtype,tiled", [(torch.float32, False), (torch.bfloat16, False),
+                                         (torch.bfloat16, True)])
 @pytest.mark.parametrize("blocks,size", BLOCKS)
-def test_block_diagonal_gates(dtype, tensor_cores, blocks, size):
+def test_block_diagonal_gates(dtype, tiled, blocks, size):
     from helix_runtime_b200.ops import library as ops
-    if tensor_cores and not ops.gated_recurrence_supports(size):
+    if tiled and not ops.gated_recurrence_supports(size):
         pytest.skip("blocks of a multiple of 8 channels")
     rng = np.random.default_rng(blocks * 1000 + size)
     for tokens in (1, 70, 300):
         case = recurrence_case(rng, dtype, tokens, blocks, size)
         decay, push = (torch.full((tokens, blocks * size), float("nan"), device="cuda")
                        for _ in range(2))
-        status = status_word()
-        ops.block_gates(*gate_arguments(case, dtype), decay, push, tokens, status,
-                        tensor_cores=tensor_cores)
-        assert int(status.item()) == 0
+        if tiled:
+            # three requests, one of them a single token
+            starts = [0, tokens] if tokens == 1 else [0, 1, tokens - 5, tokens]
+            count = len(starts) - 1
+            joined = torch.full((tokens // 64 + count, 2 * blocks * size), float("nan"), device="cuda")
+            before = torch.full((count, blocks * size), float("nan"), device="cuda")
+            state = torch.randn((4, blocks * size + 3), device="cuda")
+            slots = dev([3, 1, 0][:count], torch.int32)
+            tiles = ops.recurrence_tiles(np.diff(starts))
+            ops.block_gates_tiled(*gate_arguments(case, dtype), decay, push, joined, state, before,
+                                  dev(starts, torch.int32), slots, count, tiles)
+            assert torch.equal(before, state[slots.long(), :blocks * size])
+        else:
+            ops.block_gates(*gate_arguments(case, dtype), decay, push, tokens)
         log_a = -case["r_gate"] * case["rate"]
         # a decay close to one keeps its digits: the error is relative to a - 1
         close(as_double(decay), np.expm1(log_a), 1e-9, 2e-5, f"{tokens} tokens: a - 1")
@@ -411,8 +421,8 @@ def test_block_diagonal_gates(dtype, tensor_cores, blocks, size):
 
 
 def run_scan(case, dtype, sizes, slot, state, from_sums, form):
-    """The recurrence over one sequence in portions; ``form``: gates and scan, or the one-kernel
-    step (portions of one token)."""
+    """The recurrence over one sequence in portions; ``form``: gates and scan, the same by
+    tiles, or the one-kernel step (portions of one token)."""
     from helix_runtime_b200.ops import library as ops
     u, weights, br, bi, rate = gate_arguments(case, dtype)
     channels = case["by"].size
@@ -434,10 +444,19 @@ def run_scan(case, dtype, sizes, slot, state, from_sums, form):
                                       dev([0], torch.int32), slots, sums=from_sums)
         else:
             decay, push = (torch.empty((count, channels), device="cuda") for _ in range(2))
-            ops.block_gates(u[part].contiguous(), weights, br, bi, rate, decay, push, count,
-                            status_word())
-            ops.gated_scan(decay, push, y, device_tensor(case["by"]), state, out,
-                           dev([0, count], torch.int32), slots, 1, sums=from_sums)
+            gates = (u[part].contiguous(), weights, br, bi, rate, decay, push)
+            starts = dev([0, count], torch.int32)
+            if form == "tiled":
+                tiles = ops.recurrence_tiles([count])
+                joined = torch.full((tiles, 2 * channels), float("nan"), device="cuda")
+                before = torch.full((1, channels), float("nan"), device="cuda")
+                ops.block_gates_tiled(*gates, joined, state, before, starts, slots, 1, tiles)
+                ops.gated_scan_tiled(decay, push, joined, before, y, device_tensor(case["by"]), state,
+                                     out, starts, slots, 1, tiles, sums=from_sums)
+            else:
+                ops.block_gates(*gates, count)
+                ops.gated_scan(decay, push, y, device_tensor(case["by"]), state, out, starts, slots,
+                               1, sums=from_sums)
         if from_sums:       # the rows that were read are clear, the row behind them is not touched
             assert not y[:count].any() and bool((y[count, channels:] == 3.0).all())
         rows.append(as_double(out))
@@ -450,15 +469,15 @@ def run_scan(case, dtype, sizes, slot, state, from_sums, form):
 def test_recurrence_in_portions(dtype, blocks, size, from_sums):
     from helix_runtime_b200.ops import library as ops
     rng = np.random.default_rng(size)
-    total = 260
+    total = 710
     case = recurrence_case(rng, dtype, total, blocks, size)
     states = plain.gated_linear_recurrence(case["u"], case["r_gate"], case["i_gate"], case["lam"])
     want = states * plain.gelu_tanh(case["y"] + case["by"])
     tolerance = (2e-5, 2e-5) if dtype == torch.float32 else (1e-2, 8e-3)
-    forms = [("scan", (total,)), ("scan", (64, 2, 3, 61, 130)), ("scan", (1,) * 4 + (2,) * 128),
-             ("scan", (63, 65, 7, 125))]
+    forms = [("scan", (total,)), ("scan", (64, 2, 3, 61, 580)), ("scan", (1,) * 4 + (2,) * 353),
+             ("scan", (63, 65, 7, 575))]
     if dtype == torch.bfloat16 and ops.gated_recurrence_supports(size):
-        forms.append(("step", (1,) * total))
+        forms += [("tiled", sizes) for _, sizes in forms] + [("step", (1,) * total)]
     for form, sizes in forms:
         state = torch.zeros((3, blocks * size + 5), device="cuda")
         state[0] = state[2] = 7.0
