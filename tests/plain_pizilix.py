@@ -22,7 +22,7 @@ Feed-forward: ``Wdown (silu(Wgate h) * (Wup h))``.  Output: the norm, the table 
 ``cap * tanh(logits / cap)``.
 
 ``precision="bfloat16"`` rounds activations to bfloat16 where a bfloat16 engine stores them
-(norm outputs, projections, rotated heads, filtered rows, attention output, the recurrence's
+(norm outputs, projections before their biases, rotated heads, filtered rows, attention output, the recurrence's
 gated output, the feed-forward's activation); sums, scores, recurrences and the residual stay
 in double.
 """
@@ -211,8 +211,8 @@ class PlainPizilix:
         return self.linear(f"{prefix}.o", self.round(out.reshape(length, heads * dim)))
 
     def recurrent_mixer(self, prefix: str, sizes: dict, h: np.ndarray) -> np.ndarray:
-        y = self.round(gelu_tanh(self.linear(f"{prefix}.y", h) + self.w[f"{prefix}.y.b"]))
-        x = self.round(self.linear(f"{prefix}.x", h) + self.w[f"{prefix}.x.b"])
+        y = gelu_tanh(self.round(self.linear(f"{prefix}.y", h)) + self.w[f"{prefix}.y.b"])
+        x = self.round(self.linear(f"{prefix}.x", h)) + self.w[f"{prefix}.x.b"]
         u = self.round(causal_filter_bias(x, self.w[f"{prefix}.conv"], self.w[f"{prefix}.conv.b"]))
         r = sigmoid(block_products(u, self.w[f"{prefix}.ra"], self.w[f"{prefix}.ra.b"]))
         i = sigmoid(block_products(u, self.w[f"{prefix}.ri"], self.w[f"{prefix}.ri.b"]))
