@@ -67,7 +67,7 @@ CONFIGS = {
         "architecture": "Pizilix", "vocab": 640, "width": 256, "norm": {"eps": 1e-5},
         "logit_softcap": 20.0, "loop": {"start": 0, "stop": 2, "times": 2},
         "layers": [_rglru(256, 2, 4, 256),
-                   _attention(8, 2, 64, 96, 32, 50000.0, (6.0, 128, 16.0, 2.0), 12.0, 384, sharp=4.0),
+                   _attention(8, 2, 64, 96, 32, 20000.0, (6.0, 128, 16.0, 2.0), 12.0, 384, sharp=4.0),
                    _attention(4, 1, 128, 200, 128, 10000.0, None, 30.0, 256, sharp=4.0)],
     },
     "odd": {

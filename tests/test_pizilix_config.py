@@ -108,7 +108,7 @@ def test_what_the_configuration_refuses(change, complaint):
 
 
 @pytest.mark.parametrize("dims,base,scaling", [
-    (16, 50000.0, (4.0, 2048, 32.0, 1.0)), (12, 10000.0, (4.0, 24, 8.0, 1.0)),
+    (20, 30000.0, (5.0, 640, 16.0, 2.0)), (12, 10000.0, (4.0, 24, 8.0, 1.0)),
     (4, 77.0, (3.0, 10, 2.0, 0.25)), (64, 10000.0, None), (2, 5.0, (8.0, 4, 1.0, 0.5))])
 def test_rotary_table(dims, base, scaling):
     """The table of a position encoding holds the plain frequencies' cosines and sines times the
