@@ -45,10 +45,12 @@ class BlockSpec:
     ``streams`` is the pre-norm order over several residual streams: each sublayer is joined to
     them by a connection part (``mixer_connection``, ``feed_forward_connection``), which reads a
     weighted sum of the streams for the norm and rewrites all streams from the sublayer's output.
+    ``post_norm`` has no norms in front: ``x += c N1(mixer(x)); x += c N2(ff(x))`` with the norms and
+    the constant in ``post_norm`` connections; ``mixer_norm`` and ``feed_forward_norm`` are ``None``.
     """
 
     arrangement: str
-    mixer_norm: PartSpec
+    mixer_norm: Optional[PartSpec]
     mixer: PartSpec
     feed_forward_norm: Optional[PartSpec] = None
     feed_forward: Optional[PartSpec] = None
@@ -62,7 +64,8 @@ class ScheduleEntry:
 
     ``cache_from`` is the index of an earlier schedule entry whose key/value
     cache (or state) this entry reads instead of owning one; ``None`` means the
-    entry owns its cache.  ``add_embedding``: before this entry runs, the embedding's output
+    entry owns its cache.  A mixer that says ``keeps_own_state`` reads the other entry's keys and
+    values but keeps per-request state of its own.  ``add_embedding``: before this entry runs, the embedding's output
     (the residual stream as it stood before the first entry) is added to the residual stream
     once more; models that run a stretch of layers several times feed the input back in at
     the start of every repeat.  ``before``: a part of the family ``entry`` that is run before

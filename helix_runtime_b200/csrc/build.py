@@ -26,6 +26,8 @@ SOURCES = (
     "hx_short_conv.cu",
     "hx_streams.cu",
     "hx_recurrent.cu",
+    "hx_matrix_lstm.cu",
+    "hx_map_attention.cu",
     "hx_gated_recurrence.cu",
     "hx_rotary_norm.cu",
     "hx_gated_connection.cu",
@@ -39,7 +41,7 @@ SOURCES = (
     "hx_attention_tc.cu",
     "hx_sampling.cu",
 )
-HEADERS = ("hx_common.cuh", "hx_mma.cuh", "hx_tcgen05.cuh", "hx_no_alloc.h")
+HEADERS = ("hx_common.cuh", "hx_scan.cuh", "hx_mma.cuh", "hx_tcgen05.cuh", "hx_no_alloc.h")
 NVCC_FLAGS = (
     "-gencode", "arch=compute_100a,code=sm_100a",
     "-O3", "-std=c++17", "-lineinfo",

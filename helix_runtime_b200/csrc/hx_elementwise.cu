@@ -37,7 +37,7 @@ void hx_count_launches(int kernels) { g_hx_launches.fetch_add(kernels, std::memo
 // counts once, when it is captured).
 HX_API long long hx_launch_count() { return g_hx_launches.load(std::memory_order_relaxed); }
 
-HX_API int hx_abi_version() { return 10; }
+HX_API int hx_abi_version() { return 11; }
 
 // Streaming multiprocessors of the current device (asked once per device); 0 with a message
 // when the device cannot be asked.  Launch sizes that should fill the GPU come from here.
@@ -126,6 +126,97 @@ HX_API int hx_embed_scaled(const void* table, int dtype, const int* ids, float* 
 HX_API int hx_embed(const void* table, int dtype, const int* ids, float* out, int tokens,
                     int hidden, int vocab, int* status, cudaStream_t stream) {
   return hx_embed_scaled(table, dtype, ids, out, tokens, hidden, vocab, 1.0f, status, stream);
+}
+
+// out[t, :] = table[id[t], :] * scale + pairs[row, :] with row = (previous id * mul_prev + id * mul_cur)
+// mod buckets, and row `buckets` (the table's last) for a sequence's first token.  The id in front of a
+// portion is the request's state; the CTA of the portion's first token reads it and then leaves the
+// portion's last id there.
+template <typename T>
+__global__ void embed_pairs_kernel(const T* __restrict__ table, const T* __restrict__ pairs,
+                                   const int* __restrict__ ids, const int* __restrict__ positions,
+                                   const int* __restrict__ token_request,
+                                   const int* __restrict__ request_slot,
+                                   const int* __restrict__ request_start, int* __restrict__ previous,
+                                   long long state_stride, float* __restrict__ out, int hidden, int vocab,
+                                   int buckets, long long mul_prev, long long mul_cur, float scale,
+                                   int* status) {
+  __shared__ int shared_row;
+  hx_pdl_prologue();
+  const int token = blockIdx.x;
+  const int id = ids[token];
+  if (threadIdx.x == 0) {
+    const int request = token_request[token];
+    const int start = request_start[request];
+    long long row = buckets;
+    int before = 0;
+    if (token > start) before = ids[token - 1];
+    if (token == start) {
+      int* kept = previous + static_cast<size_t>(request_slot[request]) * state_stride;
+      before = *kept;
+      *kept = ids[request_start[request + 1] - 1];
+    }
+    if (positions[token] > 0) {
+      row = (static_cast<long long>(before) * mul_prev + static_cast<long long>(id) * mul_cur) % buckets;
+      if (row < 0) row += buckets;
+    }
+    shared_row = static_cast<int>(row);
+  }
+  __syncthreads();
+  float* row_out = out + static_cast<size_t>(token) * hidden;
+  if (id < 0 || id >= vocab) {
+    for (int c = threadIdx.x; c < hidden; c += blockDim.x) row_out[c] = __int_as_float(0x7fc00000);
+    if (threadIdx.x == 0 && status != nullptr) atomicOr(status, HX_FLAG_BAD_TOKEN);
+    return;
+  }
+  const T* own = table + static_cast<size_t>(id) * hidden;
+  const T* pair = pairs + static_cast<size_t>(shared_row) * hidden;
+  if constexpr (sizeof(T) == 2) {
+    if (hidden % 4 == 0 && ((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(pairs) |
+                             reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
+#pragma unroll 4
+      for (int q = threadIdx.x; q < hidden / 4; q += blockDim.x) {
+        const uint2 x = reinterpret_cast<const uint2*>(own)[q];
+        const uint2 y = reinterpret_cast<const uint2*>(pair)[q];
+        const float2 x0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.x));
+        const float2 x1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.y));
+        const float2 y0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&y.x));
+        const float2 y1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&y.y));
+        reinterpret_cast<float4*>(row_out)[q] = make_float4(
+            fmaf(x0.x, scale, y0.x), fmaf(x0.y, scale, y0.y), fmaf(x1.x, scale, y1.x), fmaf(x1.y, scale, y1.y));
+      }
+      return;
+    }
+  }
+  for (int c = threadIdx.x; c < hidden; c += blockDim.x)
+    row_out[c] = fmaf(hx_to_float<T>(own[c]), scale, hx_to_float<T>(pair[c]));
+}
+
+// pairs [buckets + 1, hidden] in `dtype` like the table; previous: int32 state, one per slot.
+HX_API int hx_embed_pairs(const void* table, const void* pairs, int dtype, const int* ids,
+                          const int* positions, const int* token_request, const int* request_slot,
+                          const int* request_start, int* previous, long long state_stride, float* out,
+                          int tokens, int hidden, int vocab, int buckets, long long mul_prev,
+                          long long mul_cur, float scale, int* status, cudaStream_t stream) {
+  HX_REQUIRE(tokens >= 0 && hidden > 0 && vocab > 0 && buckets > 0 && state_stride >= 1 && previous != nullptr,
+             "hx_embed_pairs: bad sizes");
+  if (tokens == 0) return HX_OK;
+  const int threads = hidden >= 1024 ? 256 : 128;
+  if (dtype == HX_F32) {
+    hx_launch(embed_pairs_kernel<float>, tokens, threads, 0, stream, static_cast<const float*>(table),
+              static_cast<const float*>(pairs), ids, positions, token_request, request_slot,
+              request_start, previous, state_stride, out, hidden, vocab, buckets, mul_prev, mul_cur,
+              scale, status);
+  } else if (dtype == HX_BF16) {
+    hx_launch(embed_pairs_kernel<__nv_bfloat16>, tokens, threads, 0, stream,
+              static_cast<const __nv_bfloat16*>(table), static_cast<const __nv_bfloat16*>(pairs), ids,
+              positions, token_request, request_slot, request_start, previous, state_stride, out, hidden,
+              vocab, buckets, mul_prev, mul_cur, scale, status);
+  } else {
+    HX_REQUIRE(false, "hx_embed_pairs: unknown dtype %d", dtype);
+  }
+  HX_CHECK_LAUNCH("hx_embed_pairs");
+  return HX_OK;
 }
 
 // x[t, :] += y[t, :] in float32 (a kept copy of the embedding output added back into the

@@ -2,7 +2,8 @@
 //
 //   * hx_norm_residual_add: a sublayer whose output passes an RMS norm BEFORE it joins the
 //     residual, x += mult * y / sqrt(mean(y^2) + eps) * w; optionally the updated row is also
-//     written in the compute type (the input of a product that reads the residual itself);
+//     written in the compute type (the input of a product that reads the residual itself), the
+//     output gets a bias first, and its buffer is left zero for the next sublayer to sum into;
 //   * hx_biased_normed_rows: what an attention layer does to its fused projection
 //     [q | k | v | head gates] before the cache append: biases, ONE RMS norm over all of a
 //     token's query coordinates and one over all of its key coordinates (not per head), a
@@ -17,6 +18,22 @@
 
 namespace {
 
+// four numbers at a time
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 add4(float4 a, float4 b) {
+  return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
+}
+__device__ __forceinline__ float4 scale4(float4 a, float4 w, float f) {
+  return make_float4(a.x * w.x * f, a.y * w.y * f, a.z * w.z * f, a.w * w.w * f);
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+  uint2 packed;
+  *reinterpret_cast<__nv_bfloat162*>(&packed.x) = __floats2bfloat162_rn(v.x, v.y);
+  *reinterpret_cast<__nv_bfloat162*>(&packed.y) = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = packed;
+}
+
 // A thread holds its share of the row in registers between the two passes (up to
 // NORM_ADD_QUADS float4 pieces; wider rows read the rest again), and all of its loads are in
 // flight together: with a few dozen tokens the kernel is a handful of round trips to memory.
@@ -25,15 +42,17 @@ constexpr int NORM_ADD_QUADS = 8;       // 256 threads x 8 x 4 floats: rows up t
 
 template <typename T>
 __global__ __launch_bounds__(NORM_ADD_THREADS) void norm_residual_add_kernel(
-    float* __restrict__ residual, const float* __restrict__ y, const float* __restrict__ weight,
-    float eps, float mult, T* __restrict__ cast_out, int ld_cast, int width) {
+    float* __restrict__ residual, float* __restrict__ y, const float* __restrict__ bias, int clear,
+    const float* __restrict__ weight, float eps, float mult, T* __restrict__ cast_out, int ld_cast,
+    int width) {
   __shared__ float scratch[32];
   hx_pdl_prologue();
   const size_t row = static_cast<size_t>(blockIdx.x) * width;
   T* cast = cast_out == nullptr ? nullptr : cast_out + static_cast<size_t>(blockIdx.x) * ld_cast;
   const bool wide = (width & 3) == 0 &&
                     ((reinterpret_cast<uintptr_t>(residual) | reinterpret_cast<uintptr_t>(y) |
-                      reinterpret_cast<uintptr_t>(weight)) & 15) == 0;
+                      reinterpret_cast<uintptr_t>(weight) | reinterpret_cast<uintptr_t>(bias)) & 15) == 0;
+  const bool wide_cast = (ld_cast & 3) == 0 && (reinterpret_cast<uintptr_t>(cast_out) & 15) == 0;
   if (wide && width <= NORM_ADD_THREADS * NORM_ADD_QUADS * 4) {
     const int quads = width >> 2;
     float4 held[NORM_ADD_QUADS];
@@ -41,8 +60,14 @@ __global__ __launch_bounds__(NORM_ADD_THREADS) void norm_residual_add_kernel(
 #pragma unroll
     for (int i = 0; i < NORM_ADD_QUADS; ++i) {
       const int q = threadIdx.x + i * NORM_ADD_THREADS;
-      held[i] = q < quads ? *reinterpret_cast<const float4*>(y + row + 4 * q)
-                          : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      held[i] = q < quads ? load4(y + row + 4 * q) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    }
+    if (bias != nullptr) {
+#pragma unroll
+      for (int i = 0; i < NORM_ADD_QUADS; ++i) {
+        const int q = threadIdx.x + i * NORM_ADD_THREADS;
+        if (q < quads) held[i] = add4(held[i], load4(bias + 4 * q));
+      }
     }
 #pragma unroll
     for (int i = 0; i < NORM_ADD_QUADS; ++i) {
@@ -56,8 +81,8 @@ __global__ __launch_bounds__(NORM_ADD_THREADS) void norm_residual_add_kernel(
     for (int i = 0; i < NORM_ADD_QUADS; ++i) {
       const int q = threadIdx.x + i * NORM_ADD_THREADS;
       if (q < quads) {
-        w[i] = *reinterpret_cast<const float4*>(weight + 4 * q);
-        x[i] = *reinterpret_cast<const float4*>(residual + row + 4 * q);
+        w[i] = load4(weight + 4 * q);
+        x[i] = load4(residual + row + 4 * q);
       }
     }
 #pragma unroll
@@ -68,27 +93,53 @@ __global__ __launch_bounds__(NORM_ADD_THREADS) void norm_residual_add_kernel(
       x[i].y = fmaf(held[i].y * inverse, w[i].y, x[i].y);
       x[i].z = fmaf(held[i].z * inverse, w[i].z, x[i].z);
       x[i].w = fmaf(held[i].w * inverse, w[i].w, x[i].w);
-      *reinterpret_cast<float4*>(residual + row + 4 * q) = x[i];
+      store4(residual + row + 4 * q, x[i]);
+      if (clear) store4(y + row + 4 * q, make_float4(0.0f, 0.0f, 0.0f, 0.0f));
       if (cast != nullptr) {
-        cast[4 * q] = hx_from_float<T>(x[i].x);
-        cast[4 * q + 1] = hx_from_float<T>(x[i].y);
-        cast[4 * q + 2] = hx_from_float<T>(x[i].z);
-        cast[4 * q + 3] = hx_from_float<T>(x[i].w);
+        if (wide_cast) {
+          store4(cast + 4 * q, x[i]);
+        } else {
+          cast[4 * q] = hx_from_float<T>(x[i].x);
+          cast[4 * q + 1] = hx_from_float<T>(x[i].y);
+          cast[4 * q + 2] = hx_from_float<T>(x[i].z);
+          cast[4 * q + 3] = hx_from_float<T>(x[i].w);
+        }
       }
     }
     return;
   }
+  auto at = [&](int c) { return y[row + c] + (bias != nullptr ? bias[c] : 0.0f); };
   float sum = 0.0f;
 #pragma unroll 4
-  for (int c = threadIdx.x; c < width; c += blockDim.x) sum = fmaf(y[row + c], y[row + c], sum);
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    const float v = at(c);
+    sum = fmaf(v, v, sum);
+  }
   const float inverse =
       mult / sqrtf(hx_block_sum(sum, scratch) / static_cast<float>(width) + eps);
 #pragma unroll 4
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    const float x = fmaf(y[row + c] * inverse, weight[c], residual[row + c]);
+    const float x = fmaf(at(c) * inverse, weight[c], residual[row + c]);
     residual[row + c] = x;
+    if (clear) y[row + c] = 0.0f;
     if (cast != nullptr) cast[c] = hx_from_float<T>(x);
   }
+}
+
+// rows in the compute type, four numbers at a time where width and addresses allow
+template <typename T>
+__global__ __launch_bounds__(256) void cast_rows_kernel(const float* __restrict__ x, T* __restrict__ out,
+                                                        int ld_out, int width) {
+  hx_pdl_prologue();
+  const float* in = x + static_cast<size_t>(blockIdx.x) * width;
+  T* row = out + static_cast<size_t>(blockIdx.x) * ld_out;
+  if (((width | ld_out) & 3) == 0 &&
+      ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
+#pragma unroll 4
+    for (int c = 4 * threadIdx.x; c < width; c += 4 * blockDim.x) store4(row + c, load4(in + c));
+    return;
+  }
+  for (int c = threadIdx.x; c < width; c += blockDim.x) row[c] = hx_from_float<T>(in[c]);
 }
 
 template <typename T>
@@ -307,21 +358,6 @@ __global__ __launch_bounds__(NORMED_ROWS_THREADS) void biased_normed_rows_kernel
 // The same four numbers at a time, for projections whose heads, rows and strides are multiples of
 // four and whose buffers are 16-byte aligned (the host checks): a load, a bias, a weight and a
 // store serve four numbers, and their head is worked out once.
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 add4(float4 a, float4 b) {
-  return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
-}
-__device__ __forceinline__ float4 scale4(float4 a, float4 w, float f) {
-  return make_float4(a.x * w.x * f, a.y * w.y * f, a.z * w.z * f, a.w * w.w * f);
-}
-__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
-  uint2 packed;
-  *reinterpret_cast<__nv_bfloat162*>(&packed.x) = __floats2bfloat162_rn(v.x, v.y);
-  *reinterpret_cast<__nv_bfloat162*>(&packed.y) = __floats2bfloat162_rn(v.z, v.w);
-  *reinterpret_cast<uint2*>(p) = packed;
-}
-
 template <typename T>
 __global__ __launch_bounds__(NORMED_ROWS_THREADS) void biased_normed_rows_quads_kernel(
     const NormedRowsArgs<T> a, const FastDivisor by_dim, const FastDivisor by_value_dim) {
@@ -519,24 +555,50 @@ __global__ __launch_bounds__(128) void token_gate_kernel(
 
 }  // namespace
 
-// residual[:tokens] += mult * y / sqrt(mean(y^2) + eps) * weight, float32 rows [tokens, width]
-// contiguous; cast_out (may be null): the updated rows in `dtype`, row stride ld_cast.
-HX_API int hx_norm_residual_add(float* residual, const float* y, const float* weight, float eps,
-                                float mult, void* cast_out, int ld_cast, int dtype, int tokens,
-                                int width, cudaStream_t stream) {
+// residual[:tokens] += mult * z / sqrt(mean(z^2) + eps) * weight with z = y + bias (bias [width] may be
+// null), float32 rows [tokens, width] contiguous; clear: y is left zero; cast_out (may be null): the
+// updated rows in `dtype`, row stride ld_cast.
+HX_API int hx_norm_residual_add_biased(float* residual, float* y, const float* bias, int clear,
+                                       const float* weight, float eps, float mult, void* cast_out,
+                                       int ld_cast, int dtype, int tokens, int width,
+                                       cudaStream_t stream) {
   HX_REQUIRE(tokens >= 0 && width > 0 && eps > 0.0f, "hx_norm_residual_add: bad sizes");
   HX_REQUIRE(cast_out == nullptr || ld_cast >= width, "hx_norm_residual_add: bad stride");
   if (tokens == 0) return HX_OK;
   if (dtype == HX_F32) {
-    hx_launch(norm_residual_add_kernel<float>, dim3(tokens), NORM_ADD_THREADS, 0, stream, residual, y, weight,
-              eps, mult, static_cast<float*>(cast_out), ld_cast, width);
+    hx_launch(norm_residual_add_kernel<float>, dim3(tokens), NORM_ADD_THREADS, 0, stream, residual, y,
+              bias, clear, weight, eps, mult, static_cast<float*>(cast_out), ld_cast, width);
   } else if (dtype == HX_BF16) {
-    hx_launch(norm_residual_add_kernel<__nv_bfloat16>, dim3(tokens), NORM_ADD_THREADS, 0, stream, residual, y,
-              weight, eps, mult, static_cast<__nv_bfloat16*>(cast_out), ld_cast, width);
+    hx_launch(norm_residual_add_kernel<__nv_bfloat16>, dim3(tokens), NORM_ADD_THREADS, 0, stream, residual,
+              y, bias, clear, weight, eps, mult, static_cast<__nv_bfloat16*>(cast_out), ld_cast, width);
   } else {
     HX_REQUIRE(false, "hx_norm_residual_add: unknown dtype %d", dtype);
   }
   HX_CHECK_LAUNCH("hx_norm_residual_add");
+  return HX_OK;
+}
+
+HX_API int hx_norm_residual_add(float* residual, const float* y, const float* weight, float eps,
+                                float mult, void* cast_out, int ld_cast, int dtype, int tokens,
+                                int width, cudaStream_t stream) {
+  return hx_norm_residual_add_biased(residual, const_cast<float*>(y), nullptr, 0, weight, eps, mult,
+                                     cast_out, ld_cast, dtype, tokens, width, stream);
+}
+
+// out[:tokens] = x[:tokens] in `dtype`; x float32 rows [tokens, width] contiguous, out's stride ld_out.
+HX_API int hx_cast_rows(const float* x, void* out, int ld_out, int dtype, int tokens, int width,
+                        cudaStream_t stream) {
+  HX_REQUIRE(tokens >= 0 && width > 0 && ld_out >= width, "hx_cast_rows: bad sizes");
+  if (tokens == 0) return HX_OK;
+  if (dtype == HX_F32) {
+    hx_launch(cast_rows_kernel<float>, dim3(tokens), 256, 0, stream, x, static_cast<float*>(out), ld_out, width);
+  } else if (dtype == HX_BF16) {
+    hx_launch(cast_rows_kernel<__nv_bfloat16>, dim3(tokens), 256, 0, stream, x,
+              static_cast<__nv_bfloat16*>(out), ld_out, width);
+  } else {
+    HX_REQUIRE(false, "hx_cast_rows: unknown dtype %d", dtype);
+  }
+  HX_CHECK_LAUNCH("hx_cast_rows");
   return HX_OK;
 }
 

@@ -19,7 +19,9 @@ constexpr int ROUTE_MAX_PER_LANE = 32;      // experts a lane can mark as taken:
 
 // What the router's sums become, and what is chosen by and weighted with.
 struct RouteRule {
-  int softmax;                // 0: s = sigmoid(z); 1: s = softmax(z) over all outputs
+  int softmax;                // 0: s = sigmoid(z); 1: s = softmax(z) over all outputs; 2: the choice
+                              // is by z itself and s is the softmax over the CHOSEN outputs alone
+  const float* bias;          // [experts] added to z; may be null
   const float* correction;    // [experts] added to s for the CHOICE only; may be null
   int normalize;              // 1: weights s / (sum of the chosen + 1e-20) * scale; 0: s * scale
 };
@@ -33,24 +35,26 @@ __global__ __launch_bounds__(128) void route_top_kernel(const float* __restrict_
   const int token = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (token >= tokens) return;
   const int lane = threadIdx.x & 31;
-  const float* z = sums + static_cast<size_t>(token) * ld;
+  const float* raw = sums + static_cast<size_t>(token) * ld;
+  auto z = [&](int e) { return rule.bias != nullptr ? raw[e] + rule.bias[e] : raw[e]; };
   // softmax: the row's maximum and the sum of exp(z - max), in ascending order per lane
   float row_max = 0.0f, inverse_sum = 1.0f;
-  if (rule.softmax) {
+  if (rule.softmax == 1) {
     row_max = -INFINITY;
-    for (int e = lane; e < experts; e += 32) row_max = fmaxf(row_max, z[e]);
+    for (int e = lane; e < experts; e += 32) row_max = fmaxf(row_max, z(e));
 #pragma unroll
     for (int offset = 16; offset > 0; offset >>= 1)
       row_max = fmaxf(row_max, __shfl_xor_sync(0xffffffffu, row_max, offset));
     float sum = 0.0f;
-    for (int e = lane; e < experts; e += 32) sum += expf(z[e] - row_max);
+    for (int e = lane; e < experts; e += 32) sum += expf(z(e) - row_max);
 #pragma unroll
     for (int offset = 16; offset > 0; offset >>= 1)
       sum += __shfl_xor_sync(0xffffffffu, sum, offset);
     inverse_sum = 1.0f / sum;
   }
   auto score_of = [&](int e) {
-    return rule.softmax ? expf(z[e] - row_max) * inverse_sum : hx_sigmoid(z[e]);
+    if (rule.softmax == 2) return z(e);
+    return rule.softmax ? expf(z(e) - row_max) * inverse_sum : hx_sigmoid(z(e));
   };
   unsigned taken = 0u;          // bit i: expert lane + 32 i is chosen already
   float total = 0.0f;
@@ -75,6 +79,10 @@ __global__ __launch_bounds__(128) void route_top_kernel(const float* __restrict_
       }
     }
     if ((best_index & 31) == lane && best_index < experts) taken |= 1u << (best_index >> 5);
+    if (rule.softmax == 2) {           // the first choice is the largest: exp(z - z_first)
+      if (k == 0) row_max = best_score;
+      best_score = expf(best_score - row_max);
+    }
     total += best_score;
     if (lane == 0) {
       chosen[static_cast<size_t>(token) * top + k] = best_index;
@@ -346,19 +354,28 @@ __global__ __launch_bounds__(128) void expert_identity_kernel(
 // [tokens, top].  softmax: scores are softmax(z) over all `experts` outputs instead of
 // sigmoid(z); correction [experts] (may be null) is added to the scores for the choice only;
 // normalize 0: the weights are the chosen scores times scale, not divided by their sum.
-HX_API int hx_route_top_ruled(const float* sums, int ld, int tokens, int experts, int top,
-                              float scale, int softmax, const float* correction, int normalize,
-                              int* chosen, float* weights, cudaStream_t stream) {
+HX_API int hx_route_top_biased(const float* sums, int ld, int tokens, int experts, int top,
+                               float scale, int softmax, const float* bias, const float* correction,
+                               int normalize, int* chosen, float* weights, cudaStream_t stream) {
   HX_REQUIRE(tokens >= 0 && experts > 0 && top > 0 && top <= experts && ld >= experts,
              "hx_route_top: bad sizes");
   HX_REQUIRE(experts <= 32 * ROUTE_MAX_PER_LANE && top <= 32,
              "hx_route_top: at most %d experts and 32 choices", 32 * ROUTE_MAX_PER_LANE);
   if (tokens == 0) return HX_OK;
-  const RouteRule rule{softmax, correction, normalize};
+  HX_REQUIRE(softmax >= 0 && softmax <= 2 && (softmax != 2 || correction == nullptr),
+             "hx_route_top: unknown score");
+  const RouteRule rule{softmax, bias, correction, normalize};
   hx_launch(route_top_kernel, dim3((tokens + 3) / 4), 128, 0, stream, sums, ld, tokens, experts,
             top, scale, rule, chosen, weights);
   HX_CHECK_LAUNCH("hx_route_top");
   return HX_OK;
+}
+
+HX_API int hx_route_top_ruled(const float* sums, int ld, int tokens, int experts, int top,
+                              float scale, int softmax, const float* correction, int normalize,
+                              int* chosen, float* weights, cudaStream_t stream) {
+  return hx_route_top_biased(sums, ld, tokens, experts, top, scale, softmax, nullptr, correction,
+                             normalize, chosen, weights, stream);
 }
 
 // s = sigmoid(z), the `top` largest, weights s / (sum of the chosen + 1e-20) * scale.

@@ -26,11 +26,19 @@ from ..weights.loader import TensorRequest
 
 Arrangement = Callable[["Block", StepContext, LayerCache, torch.Tensor, torch.Tensor], None]
 _ARRANGEMENTS: Dict[str, Arrangement] = {}
+# arrangements whose blocks find the residual in the compute dtype in ``normed`` and leave it there
+_READ_ROWS: set = set()
+
+# the key under which the embedding's per-request state lives beside the schedule entries'
+EMBEDDING_STATE = -1
 
 
-def register_arrangement(name: str, run: Arrangement) -> None:
-    """Make ``name`` usable as ``BlockSpec.arrangement``."""
+def register_arrangement(name: str, run: Arrangement, reads_rows: bool = False) -> None:
+    """Make ``name`` usable as ``BlockSpec.arrangement``.  ``reads_rows``: its blocks have no norm in
+    front of a sublayer; when one begins, ``normed`` holds the residual in the compute dtype (the
+    decoder sees to it), and when it ends, the new residual."""
     _ARRANGEMENTS[name] = run
+    (_READ_ROWS.add if reads_rows else _READ_ROWS.discard)(name)
 
 
 def _pre_norm(block: "Block", ctx: StepContext, cache: LayerCache, residual: torch.Tensor,
@@ -85,6 +93,31 @@ def _streams(block: "Block", ctx: StepContext, cache: LayerCache, residual: torc
 register_arrangement("streams", _streams)
 
 
+def _run_joined(part, connection, ctx: StepContext, residual: torch.Tensor, normed: torch.Tensor,
+                output: torch.Tensor, *before) -> None:
+    # the sublayer reads `normed` and sums into `output`, which is zero before and after; a bias of
+    # its output is added where the norm reads it
+    bias = getattr(part, "output_bias", None)
+    if bias is None:
+        part.forward(ctx, *before, normed, output)
+    else:
+        part.forward(ctx, *before, normed, output, bias_in_place=True)
+    connection.join(ctx, residual, output, normed, bias)
+
+
+def _post_norm(block: "Block", ctx: StepContext, cache: LayerCache, residual: torch.Tensor,
+               normed: torch.Tensor) -> None:
+    # x += c N1(mixer(x)); x += c N2(ff(x)): `normed` is x in the compute dtype throughout
+    output = ctx.workspace.accumulator(f"model.sublayer_sums/{block.hidden_size}",
+                                       (ctx.capacity, block.hidden_size))
+    _run_joined(block.mixer, block.mixer_connection, ctx, residual, normed, output, cache)
+    if block.feed_forward is not None:
+        _run_joined(block.feed_forward, block.feed_forward_connection, ctx, residual, normed, output)
+
+
+register_arrangement("post_norm", _post_norm, reads_rows=True)
+
+
 class Block:
     """One decoder layer: its parts, and the arrangement that runs them."""
 
@@ -96,15 +129,25 @@ class Block:
         if (spec.feed_forward is None) != (spec.feed_forward_norm is None) \
                 and spec.arrangement == "pre_norm":
             raise ValueError("a pre_norm block has a feed-forward with its norm, or neither")
-        if spec.arrangement == "streams" and (
+        if spec.arrangement == "streams" and (spec.mixer_norm is None or
                 spec.mixer_connection is None or
                 (spec.feed_forward is not None and (spec.feed_forward_connection is None
                                                     or spec.feed_forward_norm is None))):
             raise ValueError("a streams block joins every sublayer with a connection and a norm")
+        if spec.arrangement == "post_norm" and (
+                spec.mixer_norm is not None or spec.feed_forward_norm is not None
+                or spec.mixer_connection is None
+                or (spec.feed_forward is None) != (spec.feed_forward_connection is None)):
+            raise ValueError("a post_norm block joins every sublayer with a connection and has no "
+                             "norm in front of it")
+        if spec.mixer_norm is None and spec.arrangement not in _READ_ROWS:
+            raise ValueError(f"a {spec.arrangement} block has a norm in front of its mixer")
         self.arrangement = spec.arrangement
         self.hidden_size = hidden_size
         self._run = run
-        self.mixer_norm: Norm = build_part("norm", spec.mixer_norm, hidden_size)
+        self.reads_rows = spec.arrangement in _READ_ROWS
+        self.mixer_norm: Optional[Norm] = None if spec.mixer_norm is None else \
+            build_part("norm", spec.mixer_norm, hidden_size)
         self.mixer: Mixer = build_part("mixer", spec.mixer, hidden_size)
         self.feed_forward_norm: Optional[Norm] = None if spec.feed_forward_norm is None else \
             build_part("norm", spec.feed_forward_norm, hidden_size)
@@ -200,13 +243,17 @@ class DecoderModel:
         """``(kv_needs, state_needs)`` keyed by the schedule entries that own a cache."""
         kv: Dict[int, KvNeed] = {}
         state: Dict[int, StateNeed] = {}
+        embedding_state = getattr(self.embedding, "state_need", None)
+        if embedding_state is not None and embedding_state() is not None:
+            state[EMBEDDING_STATE] = embedding_state()
         for index, entry in enumerate(self.schedule):
-            if entry.cache_from is not None:
-                continue
             mixer = self.blocks[entry.block].mixer
-            need = mixer.kv_need()
-            if need is not None:
-                kv[index] = need
+            if entry.cache_from is None:
+                need = mixer.kv_need()
+                if need is not None:
+                    kv[index] = need
+            elif not mixer.keeps_own_state:
+                continue
             state_need = mixer.state_need()
             if state_need is not None:
                 state[index] = state_need
@@ -232,6 +279,8 @@ class DecoderModel:
             view.num_pages = group.pool.num_pages
             view.window = group.need.window
             view.chunk = group.need.chunk
+        if self.blocks[entry.block].mixer.keeps_own_state:
+            owner = index
         if owner in cache.states:
             view.state = cache.state(owner)
         return view
@@ -248,13 +297,14 @@ class DecoderModel:
                                      torch.float32)
         normed = ctx.workspace.get("model.normed", (ctx.capacity, h), ctx.dtype)
         embedded = None
+        own_state = {"state": cache.state(EMBEDDING_STATE)} if EMBEDDING_STATE in cache.states else {}
         if self.streams > 1:
             # every stream starts as the embedding's output
             first = ctx.workspace.get("model.embedded", (ctx.capacity, h), torch.float32)
-            self.embedding.forward(ctx, first)
+            self.embedding.forward(ctx, first, **own_state)
             ops.streams_spread(first, residual, ctx.n_tokens, self.streams)
         else:
-            self.embedding.forward(ctx, residual)
+            self.embedding.forward(ctx, residual, **own_state)
         # an entry part that does not read the embedding's output says so (needs_embedding)
         if any(entry.add_embedding for entry in self.schedule) or any(
                 getattr(part, "needs_embedding", True)
@@ -263,15 +313,26 @@ class DecoderModel:
                 raise ValueError("adding the embedding back in is defined for one residual stream")
             # the embedding's output is kept for the entries that add it back in
             embedded = ctx.workspace.get("model.embedded", (ctx.capacity, h), torch.float32)
-            self.embedding.forward(ctx, embedded)
+            if own_state:       # an embedding with state runs once a step
+                ops.cast_rows(residual, embedded, ctx.n_tokens)
+            else:
+                self.embedding.forward(ctx, embedded)
+        rows_hold_residual = False      # whether `normed` is the residual in the compute dtype
         for index, entry in enumerate(self.schedule):
+            block = self.blocks[entry.block]
             if entry.add_embedding:
                 ops.add_rows(residual, embedded, ctx.n_tokens)
+                rows_hold_residual = False
             if index in self.entry_parts:
                 self.entry_parts[index].forward(ctx, residual, embedded)
-            self.blocks[entry.block].forward(ctx, self.layer_cache(cache, index), residual, normed)
+                rows_hold_residual = False
+            if block.reads_rows and not rows_hold_residual:
+                ops.cast_rows(residual, normed, ctx.n_tokens)
+            block.forward(ctx, self.layer_cache(cache, index), residual, normed)
+            rows_hold_residual = block.reads_rows
             if index in self.entry_parts_after:
                 self.entry_parts_after[index].forward(ctx, residual, embedded)
+                rows_hold_residual = False
             if self.after_entry is not None:
                 rows = residual[:ctx.n_tokens]
                 self.after_entry(index, rows if self.streams == 1 else

@@ -290,6 +290,35 @@ def _declare(library: ctypes.CDLL) -> None:
                  "hx_token_shift", "hx_outer_product_scan", "hx_gated_group_norm",
                  "hx_norm_rotary_append", "hx_rotate_back"):
         getattr(library, name).restype = _c_int
+    library.hx_embed_pairs.argtypes = [
+        _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_longlong, _c_ptr,
+        _c_int, _c_int, _c_int, _c_int, _c_longlong, _c_longlong, _c_float, _c_ptr, _c_ptr]
+    library.hx_norm_residual_add_biased.argtypes = [
+        _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_float, _c_float, _c_ptr, _c_int, _c_int, _c_int,
+        _c_int, _c_ptr]
+    library.hx_cast_rows.argtypes = [_c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_ptr]
+    library.hx_route_top_biased.argtypes = [_c_ptr, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int,
+                                            _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr]
+    library.hx_filtered_heads.argtypes = [
+        _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_longlong, _c_ptr,
+        _c_ptr, _c_float, _c_ptr, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr,
+        _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+        _c_int, _c_int, _c_int, _c_ptr, _c_ptr]
+    library.hx_map_difference.argtypes = [
+        _c_ptr, _c_int, _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_float, _c_float, _c_float, _c_ptr,
+        _c_int, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]
+    library.hx_matrix_lstm_state_floats.argtypes = [_c_int] * 3
+    library.hx_matrix_lstm_gates.argtypes = [
+        _c_ptr, _c_int, _c_ptr, _c_float, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_longlong, _c_ptr,
+        _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]
+    library.hx_matrix_lstm.argtypes = [
+        _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_float, _c_ptr, _c_ptr,
+        _c_ptr, _c_int, _c_float, _c_float, _c_ptr, _c_float, _c_ptr, _c_longlong, _c_ptr, _c_ptr,
+        _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]
+    for name in ("hx_embed_pairs", "hx_norm_residual_add_biased", "hx_cast_rows",
+                 "hx_route_top_biased", "hx_filtered_heads", "hx_map_difference",
+                 "hx_matrix_lstm_state_floats", "hx_matrix_lstm_gates", "hx_matrix_lstm"):
+        getattr(library, name).restype = _c_int
     for name in ("hx_embed", "hx_rmsnorm", "hx_swiglu", "hx_rope_append", "hx_gemm_simt",
                  "hx_gemm_tc", "hx_gemm_tc_supports", "hx_gemm_tc_token_tile",
                  "hx_paged_attention", "hx_argmax", "hx_sample", "hx_embed_scaled",
@@ -380,6 +409,35 @@ def embed(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, status: tor
     _check(lib().hx_embed_scaled(table.data_ptr(), dtype_code(table.dtype), ids.data_ptr(),
                                  out.data_ptr(), tokens, hidden, vocab, float(scale),
                                  _ptr(status), _stream()))
+
+
+def embed_pairs(table: torch.Tensor, pairs: torch.Tensor, ids: torch.Tensor, positions: torch.Tensor,
+                token_request: torch.Tensor, request_slot: torch.Tensor, request_start: torch.Tensor,
+                previous: torch.Tensor, out: torch.Tensor, tokens: int, buckets: int, mul_prev: int,
+                mul_cur: int, status: torch.Tensor, scale: float = 1.0) -> None:
+    """out[t] (float32) = table[ids[t]] * scale + pairs[(previous id * mul_prev + ids[t] * mul_cur) mod
+    buckets], row ``buckets`` of ``pairs`` for a sequence's first token.  ``previous`` (int32 ``[slots,
+    1]``): the id in front of each request's portion, updated to the portion's last."""
+    _need(ids, torch.int32, "ids")
+    _need(previous, torch.int32, "previous")
+    _need(out, torch.float32, "out")
+    vocab, hidden = table.shape
+    assert table.is_contiguous() and pairs.is_contiguous() and out.is_contiguous()
+    assert pairs.dtype == table.dtype and tuple(pairs.shape) == (buckets + 1, hidden)
+    assert out.shape[1] == hidden
+    _check(lib().hx_embed_pairs(
+        table.data_ptr(), pairs.data_ptr(), dtype_code(table.dtype), ids.data_ptr(),
+        positions.data_ptr(), token_request.data_ptr(), request_slot.data_ptr(),
+        request_start.data_ptr(), previous.data_ptr(), previous.stride(0), out.data_ptr(), tokens,
+        hidden, vocab, buckets, int(mul_prev), int(mul_cur), float(scale), _ptr(status), _stream()))
+
+
+def cast_rows(x: torch.Tensor, out: torch.Tensor, tokens: int) -> None:
+    """out[:tokens] = x[:tokens] (float32, contiguous) in out's dtype."""
+    _need(x, torch.float32, "x")
+    assert x.is_contiguous() and out.stride(-1) == 1 and out.shape[1] == x.shape[1]
+    _check(lib().hx_cast_rows(x.data_ptr(), out.data_ptr(), out.stride(0), dtype_code(out.dtype), tokens,
+                              x.shape[1], _stream()))
 
 
 def add_rows(x: torch.Tensor, y: torch.Tensor, tokens: int) -> None:
@@ -1250,9 +1308,14 @@ def join_rows(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor, tokens: int) 
 # ------------------------------------------------ norms between a product and what follows
 
 def norm_residual_add(residual: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float,
-                      mult: float, tokens: int, cast_out: Optional[torch.Tensor] = None) -> None:
-    """residual[:tokens] += mult * y / sqrt(mean(y^2) + eps) * weight (float32 rows); with
-    ``cast_out`` the updated rows are also written there in its dtype."""
+                      mult: float, tokens: int, cast_out: Optional[torch.Tensor] = None,
+                      bias: Optional[torch.Tensor] = None, clear: bool = False) -> None:
+    """residual[:tokens] += mult * z / sqrt(mean(z^2) + eps) * weight with z = y + bias (float32
+    rows); with ``cast_out`` the updated rows are also written there in its dtype; ``clear``: y is
+    left zero."""
+    if bias is not None:
+        _need(bias, torch.float32, "bias")
+        assert bias.is_contiguous() and bias.numel() == residual.shape[1]
     _need(residual, torch.float32, "residual")
     _need(y, torch.float32, "y")
     _need(weight, torch.float32, "weight")
@@ -1260,10 +1323,10 @@ def norm_residual_add(residual: torch.Tensor, y: torch.Tensor, weight: torch.Ten
     assert residual.is_contiguous() and y.is_contiguous() and y.shape[1] == width
     assert weight.numel() == width
     code = dtype_code(cast_out.dtype) if cast_out is not None else HX_F32
-    _check(lib().hx_norm_residual_add(residual.data_ptr(), y.data_ptr(), weight.data_ptr(),
-                                      float(eps), float(mult), _ptr(cast_out),
-                                      cast_out.stride(0) if cast_out is not None else 0, code,
-                                      tokens, width, _stream()))
+    _check(lib().hx_norm_residual_add_biased(
+        residual.data_ptr(), y.data_ptr(), _ptr(bias), 1 if clear else 0, weight.data_ptr(),
+        float(eps), float(mult), _ptr(cast_out), cast_out.stride(0) if cast_out is not None else 0,
+        code, tokens, width, _stream()))
 
 
 def biased_normed_rows(projected: torch.Tensor, clear: bool, rows: torch.Tensor, tokens: int,
@@ -1333,12 +1396,18 @@ def token_gate(sums: torch.Tensor, clear: bool, table: torch.Tensor, offset: int
 
 def route_top(sums: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor, tokens: int,
               experts: int, top: int, scale: float, softmax: bool = False,
-              correction: Optional[torch.Tensor] = None, normalize: bool = True) -> None:
+              correction: Optional[torch.Tensor] = None, normalize: bool = True,
+              chosen_softmax: bool = False, bias: Optional[torch.Tensor] = None) -> None:
     """Per token the ``top`` largest of ``sigmoid(sums[:, :experts])`` (lowest index among
     equals) into ``chosen`` (int32 ``[tokens, top]``), and their scores over their sum
     (``+ 1e-20``) times ``scale`` into ``weights`` (float32).  ``softmax``: the scores are
     ``softmax(sums[:, :experts])``; ``correction`` (float32 ``[experts]``) is added to the scores
-    for the choice only; ``normalize=False``: the weights are the chosen scores times ``scale``."""
+    for the choice only; ``normalize=False``: the weights are the chosen scores times ``scale``.
+    ``bias`` (float32 ``[experts]``) is added to the sums.  ``chosen_softmax``: the choice is by the
+    (biased) sums themselves and the weights are the softmax over the chosen ones alone."""
+    if bias is not None:
+        _need(bias, torch.float32, "bias")
+        assert bias.numel() == experts
     if correction is not None:
         _need(correction, torch.float32, "correction")
         assert correction.numel() == experts
@@ -1347,10 +1416,127 @@ def route_top(sums: torch.Tensor, chosen: torch.Tensor, weights: torch.Tensor, t
     _need(weights, torch.float32, "weights")
     assert chosen.is_contiguous() and weights.is_contiguous()
     assert chosen.shape[1] == top and weights.shape[1] == top
-    _check(lib().hx_route_top_ruled(sums.data_ptr(), sums.stride(0), tokens, experts, top,
-                                    float(scale), 1 if softmax else 0, _ptr(correction),
-                                    1 if normalize else 0, chosen.data_ptr(), weights.data_ptr(),
-                                    _stream()))
+    _check(lib().hx_route_top_biased(sums.data_ptr(), sums.stride(0), tokens, experts, top,
+                                     float(scale), 2 if chosen_softmax else (1 if softmax else 0),
+                                     _ptr(bias), _ptr(correction), 1 if normalize else 0,
+                                     chosen.data_ptr(), weights.data_ptr(), _stream()))
+
+
+def filtered_heads(projected: torch.Tensor, sums: bool, rows: torch.Tensor, taps: torch.Tensor,
+                   bias: Optional[torch.Tensor], state: Optional[torch.Tensor],
+                   q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], eps: float,
+                   cosine: Optional[torch.Tensor], sine: Optional[torch.Tensor], rotary_dim: int,
+                   positions: torch.Tensor, token_request: torch.Tensor, request_slot: torch.Tensor,
+                   request_start: torch.Tensor, tokens: int, heads: int, kv_heads: int, maps: int,
+                   dim: int, value_dim: int, row_dim: int,
+                   block_tables: Optional[torch.Tensor] = None,
+                   k_cache: Optional[torch.Tensor] = None, v_cache: Optional[torch.Tensor] = None,
+                   page_size: int = 0, num_pages: int = 0,
+                   status: Optional[torch.Tensor] = None) -> None:
+    """From the projection ``[q: heads * maps * dim | k: kv_heads * maps * dim | v: kv_heads *
+    value_dim]`` (further columns ignored; ``sums``: float32 sums, rounded as a store would have)
+    of every token: biases, a causal filter ``taps [channels, n]`` over time with per-request
+    ``state`` (float32, ``(n - 1) * channels`` per slot), an RMS norm per map of a query or key
+    head, rotation of neighbouring pairs by the position; queries into ``rows`` (``row_dim`` per
+    head and map, zero outside the map's ``dim``), keys (all maps of a head in one row) and values
+    to the token's pages.  ``kv_heads=0``: the projection holds queries only."""
+    _need(taps, torch.float32, "taps")
+    channels, count = taps.shape
+    assert channels == (heads + kv_heads) * maps * dim + kv_heads * value_dim and taps.is_contiguous()
+    assert projected.dtype == (torch.float32 if sums else rows.dtype)
+    assert projected.stride(-1) == 1 and rows.stride(-1) == 1
+    for vector, size in ((bias, channels), (q_norm, dim), (k_norm, dim)):
+        if vector is not None:
+            _need(vector, torch.float32, "a float32 argument")
+            assert vector.is_contiguous() and vector.numel() == size
+    if count > 1:
+        _need(state, torch.float32, "state")
+        assert state.shape[1] >= (count - 1) * channels
+    if rotary_dim:
+        assert cosine.is_contiguous() and sine.is_contiguous() and cosine.shape[1] == rotary_dim // 2
+    _check(lib().hx_filtered_heads(
+        None if sums else projected.data_ptr(), 0 if sums else projected.stride(0),
+        projected.data_ptr() if sums else None, projected.stride(0) if sums else 0,
+        dtype_code(rows.dtype), _ptr(bias), taps.data_ptr(), count, _ptr(state),
+        0 if state is None else state.stride(0), _ptr(q_norm), _ptr(k_norm), float(eps), _ptr(cosine),
+        _ptr(sine), int(rotary_dim), cosine.shape[0] if rotary_dim else 0, rows.data_ptr(),
+        rows.stride(0), _ptr(k_cache), _ptr(v_cache), positions.data_ptr(), token_request.data_ptr(),
+        request_slot.data_ptr(), request_start.data_ptr(), _ptr(block_tables),
+        0 if block_tables is None else block_tables.stride(0), tokens, heads, kv_heads, maps, dim,
+        value_dim, row_dim, int(page_size), int(num_pages), _ptr(status), _stream()))
+
+
+def map_difference(context: torch.Tensor, gate: torch.Tensor, gate_sums: bool, lam: float,
+                   scale: float, eps: float, out: torch.Tensor, tokens: int, heads: int,
+                   value_dim: int, row_dim: int, clear: Optional[torch.Tensor] = None) -> None:
+    """Per head ``o = a1 - lam * a2`` of its two rows of ``context``, over ``sqrt(mean(o^2) + eps)``,
+    times ``scale``, times ``sigmoid(gate)``; ``gate_sums``: the gate is a view of float32 sums.
+    ``clear``: float32 rows to zero afterwards, whose last ``heads * value_dim`` columns the gate's sums
+    are when they lie in it."""
+    assert context.dtype == out.dtype and context.stride(-1) == 1 and out.stride(-1) == 1
+    assert gate.dtype == (torch.float32 if gate_sums else out.dtype) and gate.stride(-1) == 1
+    if clear is not None:
+        _need(clear, torch.float32, "clear")
+    _check(lib().hx_map_difference(
+        context.data_ptr(), context.stride(0), None if gate_sums else gate.data_ptr(),
+        0 if gate_sums else gate.stride(0), gate.data_ptr() if gate_sums else None,
+        gate.stride(0) if gate_sums else 0, dtype_code(out.dtype), float(lam), float(scale),
+        float(eps), out.data_ptr(), out.stride(0), _ptr(clear),
+        0 if clear is None else clear.stride(0), 0 if clear is None else clear.shape[1], tokens, heads,
+        value_dim, row_dim, _stream()))
+
+
+def matrix_lstm_state_floats(heads: int, dim: int, value_dim: int) -> int:
+    """Floats of a request's state row (see hx_matrix_lstm.cu); 0: no kernel takes the sizes."""
+    return lib().hx_matrix_lstm_state_floats(heads, dim, value_dim)
+
+
+def matrix_lstm_gates(sums: torch.Tensor, bias: torch.Tensor, cap: float, log_decay: torch.Tensor,
+                      push: torch.Tensor, level: torch.Tensor, state: torch.Tensor,
+                      request_start: torch.Tensor, request_slot: torch.Tensor, requests: int,
+                      tokens: int, heads: int, dim: int, value_dim: int) -> None:
+    """From the float32 sums ``[input gates | forget gates]`` of every token: the decay's logarithm, the
+    input's weight and ``exp(-m)`` (``[heads, >= tokens]`` float32 each); the running maxima in the
+    state rows move on to the portions' ends."""
+    for tensor in (sums, bias, log_decay, push, level, state):
+        _need(tensor, torch.float32, "a float32 argument")
+    assert log_decay.stride(0) == push.stride(0) == level.stride(0) >= tokens
+    _check(lib().hx_matrix_lstm_gates(
+        sums.data_ptr(), sums.stride(0), bias.data_ptr(), float(cap), log_decay.data_ptr(),
+        push.data_ptr(), level.data_ptr(), log_decay.stride(0), state.data_ptr(), state.stride(0),
+        request_start.data_ptr(), request_slot.data_ptr(), requests, tokens, heads, dim, value_dim,
+        _stream()))
+
+
+def matrix_lstm(projected: torch.Tensor, sums: bool, bias: torch.Tensor, cap: float,
+                gates: Optional[Sequence[torch.Tensor]], gate_sums: Optional[torch.Tensor],
+                q_scale: float, floor: float, norm: torch.Tensor, eps: float, state: torch.Tensor,
+                o: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, token_request: torch.Tensor,
+                request_start: torch.Tensor, request_slot: torch.Tensor, requests: int, tokens: int,
+                heads: int, dim: int, value_dim: int) -> None:
+    """The matrix memory over the step's tokens, its division, norm, weight and gate.  ``projected`` is
+    ``[q | k | v | g]`` in the compute dtype, or (``sums``) float32 sums with the gates' columns behind,
+    which are left zero.  ``gate_sums`` (a decode step, one token per request): the gates' columns;
+    otherwise ``gates`` are the three arrays of :func:`matrix_lstm_gates`.  ``o [tokens, heads *
+    value_dim]`` and ``weight [heads, >= tokens]`` are float32 scratch."""
+    _need(o, torch.float32, "o")
+    _need(weight, torch.float32, "weight")
+    _need(state, torch.float32, "state")
+    assert o.is_contiguous() and o.shape[1] == heads * value_dim and norm.numel() == heads * value_dim
+    assert projected.dtype == (torch.float32 if sums else out.dtype) and projected.stride(-1) == 1
+    ld_gates = weight.stride(0)
+    if gate_sums is None:
+        assert all(array.stride(0) == ld_gates for array in gates)
+    log_decay, push, level = (None, None, None) if gates is None else gates
+    _check(lib().hx_matrix_lstm(
+        None if sums else projected.data_ptr(), 0 if sums else projected.stride(0),
+        projected.data_ptr() if sums else None, projected.stride(0) if sums else 0,
+        dtype_code(out.dtype), _ptr(gate_sums), 0 if gate_sums is None else gate_sums.stride(0),
+        bias.data_ptr(), float(cap), _ptr(log_decay), _ptr(push), _ptr(level), ld_gates, float(q_scale),
+        float(floor), norm.data_ptr(), float(eps), state.data_ptr(), state.stride(0), o.data_ptr(),
+        weight.data_ptr(), out.data_ptr(), out.stride(0), token_request.data_ptr(),
+        request_start.data_ptr(), request_slot.data_ptr(), requests, tokens, heads, dim, value_dim,
+        _stream()))
 
 
 def expert_gate_up(x: torch.Tensor, gate_up: torch.Tensor, chosen: torch.Tensor,

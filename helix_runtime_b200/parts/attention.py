@@ -39,7 +39,8 @@ Optional mechanisms, each a parameter (absent: as if it did not exist):
   ``i`` is lowered by ``slope_h * (i - j)``.
 
 :class:`NormedProjectionAttention` adds what sits between the projection and the cache for
-models without a rotation; :class:`LatentAttention` caches one latent for all heads.
+models without a rotation; :class:`LatentAttention` caches one latent for all heads;
+:class:`DifferentialAttention` has two score maps per head over one value.
 
 At load the three projections are fused into one ``[(A + 2 Akv) D, H]`` matrix and,
 when the checkpoint rotates half-split pairs while the encoding rotates adjacent
@@ -69,7 +70,7 @@ from ..config.spec import PartSpec
 from ..ops import library as ops
 from ..weights.loader import TensorRequest
 from .base import LayerCache, Mixer, StepContext, build_part, register_part
-from .position import stretched_frequencies
+from .position import RotaryTable, stretched_frequencies
 from .linear import (STREAMING_MAX_TOKENS, Weight, is_weight_stream, project,
                      project_into_accumulator)
 
@@ -782,6 +783,186 @@ class LatentAttention(PagedAttention):
         project(heads_out, self.w_o, residual, n, ops.EPI_ADD_F32, ctx.status, ctx.ordered_sums)
 
 
+class DifferentialAttention(PagedAttention):
+    """Two score maps per head over the same values; the second is taken off the first.
+
+    Parameters: ``num_heads``, ``num_kv_heads``, ``head_dim`` (of one map of a query or key head),
+    ``value_dim``, ``scale``, ``window``, ``chunk``, ``sinks``, ``softcap`` (as in
+    :class:`PagedAttention`), ``short_conv`` (taps of the causal filter on q, k and v: 1 is a
+    filter of one tap), ``bias`` (True: q, k, v and o have biases), ``qk_norm`` (``{"eps": ...}``: an
+    RMS norm over every map of every query and key head, behind the filter and before the
+    rotation), ``rotary`` (``theta``, ``dims``: leading coordinates of each map that turn,
+    neighbouring pairs; ``scaling``: see :func:`stretched_frequencies`; ``max_positions``), ``diff``
+    (the constant ``d``), ``eps``, ``output_gate`` (``"sigmoid"``), ``shared_cache`` (True: the layer
+    has no keys and values of its own and reads those of the entry its schedule names).  Tensors:
+    ``q`` ``[heads * 2 * head_dim, hidden]`` and ``k`` (per head the first map's rows, then the
+    second's), ``v``, ``g`` ``[heads * value_dim, hidden]``, ``o``, the biases ``q_bias``,
+    ``k_bias``, ``v_bias``, ``o_bias``, the filters ``q_conv``, ``k_conv``, ``v_conv``, the norms
+    ``q_norm``, ``k_norm`` ``[head_dim]`` and ``lq1``, ``lk1``, ``lq2``, ``lk2`` ``[head_dim]``.
+
+    With ``a1``, ``a2`` the two maps' results, ``l = exp(lq1 . lk1) - exp(lq2 . lk2) + d``: ``o = a1 -
+    l a2``, over ``sqrt(mean(o^2) + eps)`` of the head, times ``1 - d``, times ``sigmoid(g x)``, then
+    the output matrix.
+
+    A key/value head caches ONE key row ``[k of map 1 | k of map 2]`` beside its value row, and a
+    map's query row is zero outside its half: the maps are query heads of an ordinary grouped
+    attention (``2 * num_heads`` of them over ``num_kv_heads``), so every attention kernel serves
+    them, a token's key and value are cached once, and a decode step reads them once for both maps.
+    ``[q | k | v | g]`` is one product; one kernel adds biases, filters, norms, rotates, lays out the
+    queries and appends to the pages; attention; one kernel combines the maps, norms and gates.
+    """
+
+    keeps_own_state = True       # the filter's inputs are this layer's, whoever's keys it reads
+
+    def __init__(self, spec: PartSpec, hidden_size: int) -> None:
+        if spec.get("output_gate") != "sigmoid":
+            raise ValueError("differential attention gates its output with 'sigmoid'")
+        maps = 2
+        dim = int(spec["head_dim"])
+        inner = {key: spec.params[key] for key in ("num_kv_heads", "scale", "window", "chunk", "softcap")
+                 if key in spec.params}
+        inner.update(num_heads=maps * int(spec["num_heads"]), head_dim=maps * dim,
+                     value_dim=int(spec.get("value_dim") or dim),
+                     position=PartSpec("none", {"head_dim": maps * dim}))
+        super().__init__(PartSpec(spec.kind, inner, spec.tensors), hidden_size)
+        self.spec = spec
+        self.maps, self.map_dim = maps, dim
+        self.model_heads = int(spec["num_heads"])
+        # single tokens: the query rows of a key/value head attend side by side
+        self.pack_heads, self.pack_always = True, False
+        self.taps = int(spec.get("short_conv") or 1)
+        if self.taps < 1:
+            raise ValueError("short_conv counts the filter's taps: at least 1")
+        self.bias = bool(spec.get("bias", False))
+        norm = spec.get("qk_norm")
+        self.qk_eps = float(norm["eps"]) if norm else 0.0
+        self.qk_norm = norm is not None
+        if self.qk_norm and not self.qk_eps > 0.0:
+            raise ValueError("the query and key norm needs a positive eps")
+        self.eps = float(spec["eps"])
+        if not self.eps > 0.0:
+            raise ValueError("the norm of the maps' difference needs a positive eps")
+        self.diff = float(spec["diff"])
+        self.rotary = spec.get("rotary")
+        self.rotary_dims = int(self.rotary.get("dims", dim)) if self.rotary else 0
+        if self.rotary_dims % 2 or not 0 <= self.rotary_dims <= dim:
+            raise ValueError("rotary dims must be even and at most head_dim")
+        self.shared_cache = bool(spec.get("shared_cache", False))
+        own = 0 if self.shared_cache else self.kv_heads
+        self.own_kv_heads = own
+        self.q_rows = self.model_heads * maps * dim
+        self.k_rows, self.v_rows = own * maps * dim, own * self.value_dim
+        self.o_columns = self.model_heads * self.value_dim
+        self.filtered = self.q_rows + self.k_rows + self.v_rows
+        self.projected_size = self.filtered + self.o_columns
+        self.balance = 0.0
+        self.w_proj: Optional[Weight] = None
+        self.biases = self.taps_weight = self.q_norm = self.k_norm = self.o_bias = None
+        self.table: Optional[RotaryTable] = None
+
+    def state_need(self) -> Optional[StateNeed]:
+        size = (self.taps - 1) * self.filtered
+        return StateNeed((size + size % 2,), torch.float32) if size else None
+
+    def _sources(self):
+        """``(role, rows)`` of what the layer projects and filters."""
+        return [("q", self.q_rows)] + ([] if self.shared_cache else
+                                       [("k", self.k_rows), ("v", self.v_rows)])
+
+    def tensor_requests(self) -> List[TensorRequest]:
+        h = self.hidden_size
+        requests = []
+        for role, rows in self._sources():
+            requests.append(TensorRequest(self.names[role], (rows, h)))
+            requests.append(TensorRequest(self.names[f"{role}_conv"], (rows, self.taps), role="scale"))
+            if self.bias:
+                requests.append(TensorRequest(self.names[f"{role}_bias"], (rows,), role="scale"))
+            if self.qk_norm and role != "v":
+                requests.append(TensorRequest(self.names[f"{role}_norm"], (self.map_dim,), role="scale"))
+        requests += [TensorRequest(self.names[role], (self.map_dim,), role="scale")
+                     for role in ("lq1", "lk1", "lq2", "lk2")]
+        requests += [TensorRequest(self.names["g"], (self.o_columns, h)),
+                     TensorRequest(self.names["o"], (h, self.o_columns))]
+        if self.bias:
+            requests.append(TensorRequest(self.names["o_bias"], (h,), role="scale"))
+        return requests + self._score_term_requests()
+
+    def bind(self, tensors: Mapping[str, torch.Tensor], dtype, device) -> None:
+        def vector(role: str) -> torch.Tensor:
+            return tensors[self.names[role]].to(device=device, dtype=torch.float32).contiguous()
+        sources = [role for role, _ in self._sources()]
+        self.w_proj = Weight(torch.cat([tensors[self.names[role]] for role in (*sources, "g")], dim=0)
+                             .to(device=device, dtype=dtype).contiguous())
+        self.w_o = Weight(tensors[self.names["o"]].to(device=device, dtype=dtype).contiguous())
+        self.taps_weight = torch.cat([vector(f"{role}_conv") for role in sources]).contiguous()
+        if self.bias:
+            self.biases = torch.cat([vector(f"{role}_bias") for role in sources]).contiguous()
+            self.o_bias = vector("o_bias")
+        if self.qk_norm:
+            self.q_norm = vector("q_norm")
+            self.k_norm = None if self.shared_cache else vector("k_norm")
+        l1, l2 = (float(torch.dot(*(tensors[self.names[role]].to(torch.float64).cpu() for role in pair)))
+                  for pair in (("lq1", "lk1"), ("lq2", "lk2")))
+        self.balance = math.exp(l1) - math.exp(l2) + self.diff
+        if self.rotary_dims:
+            frequency, amplitude = stretched_frequencies(self.rotary_dims, float(self.rotary["theta"]),
+                                                         self.rotary.get("scaling"))
+            self.table = RotaryTable.shared(frequency, amplitude, int(self.rotary["max_positions"]), device)
+        self.dtype = dtype
+        self._bind_score_terms(tensors, device)
+
+    @property
+    def graph_safe(self) -> bool:
+        return True
+
+    def weight_bytes(self) -> int:
+        return self.w_proj.nbytes() + self.w_o.nbytes()
+
+    @property
+    def output_bias(self) -> Optional[torch.Tensor]:
+        """The bias of the output matrix (see ``FeedForward.output_bias``)."""
+        return self.o_bias
+
+    def forward(self, ctx: StepContext, cache: LayerCache, x: torch.Tensor,
+                residual: torch.Tensor, bias_in_place: bool = False) -> None:
+        n, get = ctx.n_tokens, ctx.workspace.get
+        rows = get(f"attention.map_rows/{self.q_size}", (ctx.capacity, self.q_size), ctx.dtype)
+        context = get(f"attention.context/{self.q_size}", (ctx.capacity, self.q_size), ctx.dtype)
+        wide = -(-self.o_columns // 8) * 8
+        heads_out = get(f"attention.maps_out/{wide}", (ctx.capacity, wide), ctx.dtype)[:, :self.o_columns]
+        sums = is_weight_stream(x, self.w_proj, n)
+        if sums:
+            size = -(-self.projected_size // 4) * 4
+            projected = ctx.workspace.accumulator(f"attention.projected/{size}",
+                                                  (STREAMING_MAX_TOKENS, size))
+            project_into_accumulator(x, self.w_proj, projected, n, ctx.status, ctx.ordered_sums)
+        else:
+            size = -(-self.projected_size // 8) * 8
+            projected = get(f"attention.projected/{size}", (ctx.capacity, size), ctx.dtype)
+            project(x, self.w_proj, projected, n, ops.EPI_STORE, ctx.status)
+        table = self.table
+        write = not self.shared_cache
+        ops.filtered_heads(projected, sums, rows, self.taps_weight, self.biases,
+                           cache.state if self.taps > 1 else None, self.q_norm, self.k_norm,
+                           self.qk_eps, table.cos if table else None, table.sin if table else None,
+                           self.rotary_dims, ctx.positions, ctx.token_request, ctx.request_slot,
+                           ctx.request_start, n, self.model_heads, self.own_kv_heads, self.maps,
+                           self.map_dim, self.value_dim, self.row_dim,
+                           block_tables=cache.block_tables if write else None,
+                           k_cache=cache.keys if write else None,
+                           v_cache=cache.values if write else None, page_size=cache.page_size,
+                           num_pages=cache.num_pages, status=ctx.status)
+        self.attend(ctx, cache, rows, context)
+        used = projected[:, :self.projected_size]
+        ops.map_difference(context, used[:, self.filtered:], sums, self.balance, 1.0 - self.diff,
+                           self.eps, heads_out, n, self.model_heads, self.value_dim, self.row_dim,
+                           clear=used if sums else None)
+        if self.o_bias is not None and not bias_in_place:
+            ops.add_bias(residual, self.o_bias, n)
+        project(heads_out, self.w_o, residual, n, ops.EPI_ADD_F32, ctx.status, ctx.ordered_sums)
+
+
 register_part("mixer", "paged_attention", PagedAttention)
+register_part("mixer", "differential_attention", DifferentialAttention)
 register_part("mixer", "latent_attention", LatentAttention)
 register_part("mixer", "normed_projection_attention", NormedProjectionAttention)

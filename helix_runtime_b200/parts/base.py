@@ -16,7 +16,9 @@ Interfaces (all tensors live on the device; ``ctx`` is the step's
 * Norm:          ``forward(ctx, x_f32[N,H], out[N,H], rows=None)`` writes the compute dtype.
 * Mixer:         ``forward(ctx, cache, x[N,H], residual_f32[N,H])`` adds its output into
   ``residual``.  ``kv_need()`` / ``state_need()`` say what it wants of the cache manager;
-  ``cache`` is the :class:`LayerCache` of the schedule entry being run.
+  ``cache`` is the :class:`LayerCache` of the schedule entry being run.  A mixer or feed-forward
+  whose output has a bias may offer it (``output_bias``) to whoever owns the buffer it sums into,
+  and is then called with ``bias_in_place=True``.
 * FeedForward:   ``forward(ctx, x[N,H], residual_f32[N,H])`` adds its output into ``residual``.
 * PositionEncoding: owned by a mixer; ``apply(ctx, cache, qkv, ...)`` encodes queries and
   keys in place and stores keys/values into the cache pages.
@@ -192,6 +194,10 @@ class PositionEncoding(Part):
 
 
 class Mixer(Part):
+    # An entry with ``cache_from`` reads the other entry's keys and values, and its state too
+    # unless the mixer keeps its own.
+    keeps_own_state: bool = False
+
     def kv_need(self) -> Optional[KvNeed]:
         return None
 

@@ -216,6 +216,14 @@ class NormedConnection(Part):
         ops.norm_residual_add(streams, output, self.weight, self.eps, self.scale, ctx.n_tokens,
                               cast_out=cast)
 
+    def join(self, ctx: StepContext, residual: torch.Tensor, output: torch.Tensor,
+             rows: torch.Tensor, bias: Optional[torch.Tensor] = None) -> None:
+        """``x += scale * norm(output + bias)``; ``output`` is left zero for the next sublayer and
+        ``rows`` gets the new ``x`` in the compute dtype (what a sublayer without a norm in front
+        reads): one kernel."""
+        ops.norm_residual_add(residual, output, self.weight, self.eps, self.scale, ctx.n_tokens,
+                              cast_out=rows, bias=bias, clear=True)
+
 
 class TokenSideInput(Part):
     needs_embedding = False      # it reads the residual, not the embedding's output

@@ -2,7 +2,8 @@
 
 Parameters: ``intermediate_size``, ``activation`` (``silu``, or ``gelu_tanh``:
 the tanh approximation of GELU, ``z * sigmoid(2 c (z + a z^3))`` with ``c = sqrt(2/pi)``,
-``a = 0.044715``; or ``relu``), ``bias`` (True: all three projections have biases, tensors
+``a = 0.044715``; or ``relu``; or ``clamped_sigmoid`` with ``limit`` ``L``, a function of both: ``g =
+min(gate, L)``, ``u = clamp(up, -L, L)``, ``g sigmoid(1.702 g) (u + 1)``), ``bias`` (True: all three projections have biases, tensors
 ``gate_bias``, ``up_bias``, ``down_bias``).  Tensors: ``gate``, ``up``
 ``[intermediate, hidden]`` and ``down`` ``[hidden, intermediate]``.  gate and up are
 fused into one ``[2I, H]`` matrix at load so that both products read the input once;
@@ -22,7 +23,7 @@ import torch
 from ..config.spec import PartSpec
 from ..ops import library as ops
 from ..weights.loader import TensorRequest
-from .base import FeedForward, StepContext, register_part
+from .base import FeedForward, StepContext, build_part, register_part
 from .linear import Weight, project, project_gated, project_swiglu
 
 
@@ -34,8 +35,9 @@ class GatedMlp(FeedForward):
         if activation not in ops.GATE_ACTIVATIONS:
             raise ValueError(f"activation {activation!r} has no kernel; known: "
                              + ", ".join(sorted(ops.GATE_ACTIVATIONS)))
-        if activation == "clamped_sigmoid":
-            raise ValueError("the clamped gate belongs to routed experts")
+        self.limit = float(spec.get("limit", 0.0))
+        if activation == "clamped_sigmoid" and not self.limit > 0.0:
+            raise ValueError("the clamped gate needs a positive limit")
         self.activation = ops.GATE_ACTIVATIONS[activation]
         self.bias = bool(spec.get("bias", False))
         # the product's own epilogue knows silu and gelu_tanh without biases
@@ -86,7 +88,7 @@ class GatedMlp(FeedForward):
         else:
             project_gated(x, self.w_gate_up, self.intermediate, act, ctx.workspace, ctx.capacity,
                           n, ctx.status, ctx.ordered_sums, self.activation, self.gate_bias,
-                          self.up_bias)
+                          self.up_bias, self.limit)
         if self.down_bias is not None and not bias_in_place:
             ops.add_bias(residual, self.down_bias, n)
         project(act, self.w_down, residual, n, ops.EPI_ADD_F32, ctx.status, ctx.ordered_sums)
@@ -169,7 +171,11 @@ class RoutedExperts(FeedForward):
 
     More rules, each a parameter: ``score`` (``sigmoid``, or ``softmax`` over all router
     outputs), ``correction`` (True: the tensor ``correction`` ``[router outputs]`` is added to the
-    scores for the CHOICE only, the weights use the scores without it), ``normalize`` (False: the
+    scores for the CHOICE only, the weights use the scores without it), ``router_bias`` (True: the
+    tensor ``router_bias`` is added to the router's sums before anything else), ``score``
+    ``chosen_softmax`` (the choice is by the sums themselves, the weights are the softmax over the
+    chosen ones alone), ``shared`` (a feed-forward's part spec: it runs for every token and its output
+    is added), ``normalize`` (False: the
     weights are the chosen scores times ``scale``, not divided by their sum), ``identity`` (so
     many more router outputs behind the experts that have no matrices: chosen, such an output
     contributes ``weight * x``), ``activation`` ``clamped_sigmoid`` with ``limit`` ``L``:
@@ -186,9 +192,16 @@ class RoutedExperts(FeedForward):
         self.intermediate = int(spec["intermediate_size"])
         self.scale = float(spec.get("scale", 1.0))
         score = spec.get("score", "sigmoid")
-        if score not in ("sigmoid", "softmax"):
-            raise ValueError(f"router score {score!r} is neither 'sigmoid' nor 'softmax'")
+        if score not in ("sigmoid", "softmax", "chosen_softmax"):
+            raise ValueError(f"router score {score!r} is none of 'sigmoid', 'softmax' and "
+                             "'chosen_softmax'")
         self.softmax = score == "softmax"
+        self.chosen_softmax = score == "chosen_softmax"
+        self.has_router_bias = bool(spec.get("router_bias", False))
+        self.router_bias: Optional[torch.Tensor] = None
+        shared = spec.get("shared")
+        self.shared: Optional[FeedForward] = None if shared is None else \
+            build_part("feed_forward", shared, hidden_size)
         self.corrected = bool(spec.get("correction", False))
         self.normalize = bool(spec.get("normalize", True))
         self.limit = float(spec.get("limit", 0.0))
@@ -209,6 +222,11 @@ class RoutedExperts(FeedForward):
         if self.corrected:
             requests.append(TensorRequest(self.names["correction"], (self.router_outputs,),
                                           role="scale"))
+        if self.has_router_bias:
+            requests.append(TensorRequest(self.names["router_bias"], (self.router_outputs,),
+                                          role="scale"))
+        if self.shared is not None:
+            requests += self.shared.tensor_requests()
         for e in range(self.experts):
             requests += [TensorRequest(self.names[f"gate.{e}"], (i, h)),
                          TensorRequest(self.names[f"up.{e}"], (i, h)),
@@ -226,10 +244,20 @@ class RoutedExperts(FeedForward):
         if self.corrected:
             self.correction = tensors[self.names["correction"]] \
                 .to(device=device, dtype=torch.float32).contiguous()
+        if self.has_router_bias:
+            self.router_bias = tensors[self.names["router_bias"]] \
+                .to(device=device, dtype=torch.float32).contiguous()
+        if self.shared is not None:
+            self.shared.bind(tensors, dtype, device)
 
     def weight_bytes(self) -> int:
+        shared = 0 if self.shared is None else self.shared.weight_bytes()
         return self.w_router.nbytes() + (self.w_gate_up.numel() + self.w_down.numel()) \
-            * self.w_down.element_size()
+            * self.w_down.element_size() + shared
+
+    @property
+    def graph_safe(self) -> bool:
+        return self.shared is None or self.shared.graph_safe
 
     def forward(self, ctx: StepContext, x: torch.Tensor, residual: torch.Tensor) -> None:
         n = ctx.n_tokens
@@ -242,7 +270,10 @@ class RoutedExperts(FeedForward):
                   (ctx.capacity * self.top, self.intermediate), ctx.dtype)
         project(x, self.w_router, sums, n, ops.EPI_STORE_F32, ctx.status)
         ops.route_top(sums, chosen, weights, n, self.router_outputs, self.top, self.scale,
-                      softmax=self.softmax, correction=self.correction, normalize=self.normalize)
+                      softmax=self.softmax, correction=self.correction, normalize=self.normalize,
+                      chosen_softmax=self.chosen_softmax, bias=self.router_bias)
+        if self.shared is not None:
+            self.shared.forward(ctx, x, residual)
         if self.identity:
             # router outputs behind the experts return the input; the experts' kernels leave
             # such choices out

@@ -75,11 +75,13 @@ def _gemm_tc(x, w: Weight, out, tokens, features, epilogue, status, **options) -
         ops.gemm_tc(x, w.matrix, out, tokens, features, epilogue, status, **options)
 
 
-def _gemm_simt(x, w: Weight, out, tokens, epilogue, softcap: float = 0.0) -> None:
+def _gemm_simt(x, w: Weight, out, tokens, epilogue, softcap: float = 0.0,
+               features: Optional[int] = None) -> None:
     if w.matrix is None:
         raise RuntimeError("this product needs the CUDA-core kernel, but the weight is held as "
                            "tiles for the tensor cores")
-    ops.gemm_simt(x, w.matrix, out, tokens, epilogue, softcap)
+    ops.gemm_simt(x, w.matrix if features is None else w.matrix[:features], out, tokens, epilogue,
+                  softcap)
 
 
 def is_weight_stream(x: torch.Tensor, w: Weight, tokens: int) -> bool:
@@ -108,18 +110,20 @@ def split_k_for(tokens: int, features: int, depth: int, ordered: bool = False) -
 
 
 def project(x: torch.Tensor, w: Weight, out: torch.Tensor, tokens: int, epilogue: int,
-            status: torch.Tensor, ordered: bool = False, softcap: float = 0.0) -> None:
+            status: torch.Tensor, ordered: bool = False, softcap: float = 0.0,
+            features: Optional[int] = None) -> None:
     """``out[:tokens] (op)= x[:tokens] @ w.T``; epilogue is one of ops.EPI_STORE,
-    ops.EPI_STORE_F32, ops.EPI_ADD_F32.  ``ordered``: no split-K (see ``split_k_for``).
+    ops.EPI_STORE_F32, ops.EPI_ADD_F32.  ``features``: only the first so many rows of ``w``.  ``ordered``: no split-K (see ``split_k_for``).
     ``softcap`` > 0 (ops.EPI_STORE_F32 only): ``softcap * tanh(product / softcap)``."""
     if tokens == 0:
         return
     if uses_tensor_cores(x, w, tokens):
         splits = split_k_for(tokens, w.rows, w.depth, ordered) \
             if epilogue == ops.EPI_ADD_F32 else 1
-        _gemm_tc(x, w, out, tokens, w.rows, epilogue, status, k_splits=splits, softcap=softcap)
+        _gemm_tc(x, w, out, tokens, features or w.rows, epilogue, status, k_splits=splits,
+                 softcap=softcap)
     else:
-        _gemm_simt(x, w, out, tokens, epilogue, softcap)
+        _gemm_simt(x, w, out, tokens, epilogue, softcap, features)
 
 
 def project_into_accumulator(x: torch.Tensor, w: Weight, accumulator: torch.Tensor,

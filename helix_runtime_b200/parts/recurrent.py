@@ -1,6 +1,6 @@
 """Recurrent mixers: the selective state-space layer, the time-mixing layer with a decayed
-outer-product state, linear attention, the gated linear recurrence, and mixers that wrap or run
-others.
+outer-product state, linear attention, the gated linear recurrence, the matrix memory with
+exponential gates, and mixers that wrap or run others.
 
 All of them keep per-request state in ONE float32 row per schedule entry (``StateNeed`` of a flat
 shape); a mixer cuts its row into the pieces it needs.  A step brings a portion of each
@@ -48,6 +48,15 @@ Tensors ``y``, ``x`` ``[width, hidden]``, ``y_bias``, ``x_bias``, ``filter`` ``[
 last tap on the token itself), ``filter_bias``, ``r``, ``i`` ``[blocks, width / blocks, width /
 blocks]``, ``r_bias``, ``i_bias`` ``[blocks, width / blocks]``, ``decay`` ``[width]``, ``o``.  State:
 the filter's last inputs and the numbers ``S``.
+
+:class:`MatrixLstm` (``matrix_lstm``).  Parameters ``heads``, ``head_dim``, ``value_dim``,
+``gate_cap`` (``c``), ``q_scale``, ``floor``, ``eps``.  Per head ``i = c tanh((W_i x + b_i) / c)`` and
+``f = log sigmoid(c tanh((W_f x + b_f) / c))``; with the running maximum ``m_t = max(f + m_(t-1), i)``
+(zero at admission) ``S_t = e^(f + m_(t-1) - m_t) S_(t-1) + e^(i - m_t) k v'``, ``n_t`` likewise with ``k``
+alone, ``o = S' q / (max(|n . q|, e^-m) + floor)`` with ``q = q_scale W_q x``.  Each head's ``o`` over its
+root mean square, times ``norm``, times ``sigmoid(W_g x)``, then the output projection.  Tensors ``q``,
+``k``, ``v``, ``g``, ``i``, ``f`` ``[heads, hidden]``, ``i_bias``, ``f_bias``, ``norm`` ``[heads *
+value_dim]``, ``o``.  State: the matrices ``S`` with ``n`` as one more column, and ``m``.
 
 :class:`InputFilter` (``input_filter``).  Parameters ``taps``, ``mixer`` (a part spec): the inner
 mixer reads ``x + conv(x)``, ``conv`` a causal per-channel filter over time (tensor ``filter``
@@ -498,6 +507,97 @@ class GatedRecurrence(Mixer):
         project(gated, self.w_o, residual, n, ops.EPI_ADD_F32, ctx.status, ctx.ordered_sums)
 
 
+class MatrixLstm(Mixer):
+    def __init__(self, spec: PartSpec, hidden_size: int) -> None:
+        super().__init__(spec, hidden_size)
+        self.heads = int(spec["heads"])
+        self.head_dim = int(spec["head_dim"])
+        self.value_dim = int(spec.get("value_dim") or self.head_dim)
+        self.gate_cap = float(spec["gate_cap"])
+        self.q_scale = float(spec.get("q_scale", 1.0))
+        self.floor = float(spec.get("floor", 0.0))
+        self.eps = float(spec["eps"])
+        if not (self.gate_cap > 0.0 and self.eps > 0.0 and self.floor >= 0.0):
+            raise ValueError("gate_cap and eps are positive, floor is not negative")
+        self.qk_width = self.heads * self.head_dim
+        self.v_width = self.heads * self.value_dim
+        self.rows_size = 2 * (self.qk_width + self.v_width)       # q | k | v | g
+        self.projected_size = self.rows_size + 2 * self.heads     # ... | i | f
+        self.names = dict(spec.tensors)
+        self.w_in: Optional[Weight] = None
+        self.w_gates: Optional[Weight] = None
+        self.w_o: Optional[Weight] = None
+
+    def state_need(self) -> Optional[StateNeed]:
+        floats = ops.matrix_lstm_state_floats(self.heads, self.head_dim, self.value_dim)
+        if floats == 0:
+            raise ValueError(f"no kernel takes recurrent heads of {self.head_dim}")
+        return StateNeed((floats,), torch.float32)
+
+    def tensor_requests(self) -> List[TensorRequest]:
+        h = self.hidden_size
+        return [TensorRequest(self.names["q"], (self.qk_width, h)),
+                TensorRequest(self.names["k"], (self.qk_width, h)),
+                TensorRequest(self.names["v"], (self.v_width, h)),
+                TensorRequest(self.names["g"], (self.v_width, h)),
+                TensorRequest(self.names["i"], (self.heads, h)),
+                TensorRequest(self.names["i_bias"], (self.heads,), role="scale"),
+                TensorRequest(self.names["f"], (self.heads, h)),
+                TensorRequest(self.names["f_bias"], (self.heads,), role="scale"),
+                TensorRequest(self.names["norm"], (self.v_width,), role="scale"),
+                TensorRequest(self.names["o"], (h, self.v_width))]
+
+    def bind(self, tensors: Mapping[str, torch.Tensor], dtype, device) -> None:
+        def scale(role: str) -> torch.Tensor:
+            return tensors[self.names[role]].to(device=device, dtype=torch.float32).contiguous()
+
+        def matrix(*roles: str) -> Weight:
+            return Weight(torch.cat([tensors[self.names[role]] for role in roles], dim=0)
+                          .to(device=device, dtype=dtype).contiguous())
+        # few tokens: everything is one weight stream with float32 sums.  Prompts: its first rows
+        # are stored in the compute dtype, and the gates, which stay float32, are a product of
+        # their own with a copy of their few rows.
+        self.w_in = matrix("q", "k", "v", "g", "i", "f")
+        self.w_gates = matrix("i", "f")
+        self.w_o = matrix("o")
+        self.gate_bias = torch.cat([scale("i_bias"), scale("f_bias")]).contiguous()
+        self.norm = scale("norm")
+
+    def weight_bytes(self) -> int:
+        return self.w_in.nbytes() + self.w_o.nbytes()
+
+    def forward(self, ctx: StepContext, cache: LayerCache, x: torch.Tensor,
+                residual: torch.Tensor) -> None:
+        n, heads, get = ctx.n_tokens, self.heads, ctx.workspace.get
+        o = get(f"matrix_lstm.o/{self.v_width}", (ctx.capacity, self.v_width), torch.float32)
+        arrays = get(f"matrix_lstm.gates/{heads}", (4, heads, ctx.capacity), torch.float32)
+        wide = -(-self.v_width // 8) * 8
+        out = get(f"matrix_lstm.out/{wide}", (ctx.capacity, wide), ctx.dtype)[:, :self.v_width]
+        sums = is_weight_stream(x, self.w_in, n)
+        if sums:
+            size = -(-self.projected_size // 4) * 4
+            rows = ctx.workspace.accumulator(f"matrix_lstm.rows/{size}", (STREAMING_MAX_TOKENS, size))
+            project_into_accumulator(x, self.w_in, rows, n, ctx.status, ctx.ordered_sums)
+            gate_sums = rows[:, self.rows_size:]
+        else:
+            size = -(-self.rows_size // 8) * 8
+            rows = get(f"matrix_lstm.rows/{size}", (ctx.capacity, size), ctx.dtype)
+            project(x, self.w_in, rows, n, ops.EPI_STORE, ctx.status, features=self.rows_size)
+            width = -(-2 * heads // 4) * 4
+            gate_sums = get(f"matrix_lstm.gate_sums/{width}", (ctx.capacity, width), torch.float32)
+            project(x, self.w_gates, gate_sums, n, ops.EPI_STORE_F32, ctx.status)
+        batch = (ctx.request_start, ctx.request_slot, ctx.n_requests, n, heads, self.head_dim,
+                 self.value_dim)
+        one_token = n == ctx.n_requests
+        if not one_token:
+            ops.matrix_lstm_gates(gate_sums, self.gate_bias, self.gate_cap, arrays[0], arrays[1],
+                                  arrays[2], cache.state, *batch)
+        ops.matrix_lstm(rows, sums, self.gate_bias, self.gate_cap, None if one_token else arrays[:3],
+                        gate_sums if one_token else None, self.q_scale, self.floor, self.norm, self.eps,
+                        cache.state, o, arrays[3], out, ctx.token_request, *batch)
+        project(out, self.w_o, residual, n, ops.EPI_ADD_F32, ctx.status, ctx.ordered_sums)
+
+
 class InputFilter(Mixer):
     def __init__(self, spec: PartSpec, hidden_size: int) -> None:
         super().__init__(spec, hidden_size)
@@ -616,5 +716,6 @@ register_part("mixer", "state_space", StateSpaceMixer)
 register_part("mixer", "time_mix", TimeMix)
 register_part("mixer", "side_by_side", SideBySide)
 register_part("mixer", "linear_state", LinearState)
+register_part("mixer", "matrix_lstm", MatrixLstm)
 register_part("mixer", "input_filter", InputFilter)
 register_part("mixer", "gated_recurrence", GatedRecurrence)
