@@ -500,6 +500,42 @@ def pizilix_config(shape: dict, options):
                          max_positions=shape["max_position_embeddings"])
 
 
+def manatar_config(shape: dict, options):
+    """The Manatar design with the layer sizes of a Llama shape: the same width, vocabulary and
+    active feed-forward size.  Layers in turn: attention with two maps per head (the shape's heads
+    and value size, a map half as wide, a quarter as many key/value heads, filters of four taps,
+    stretched frequencies, causal), the matrix memory (a quarter of the shape's heads, matrices of
+    twice the head size by four times it), attention over the first one's keys and values, the
+    matrix memory again.  The first layer's feed-forward is dense with a clamped gate, the others
+    are 16 routed experts of a quarter of the shape's feed-forward of which a token uses 3, beside a
+    shared one of the same size; a second embedding table of 65,536 rows."""
+    import math
+
+    from helix_runtime_b200.config.manatar import (DifferentialAttentionConfig, FeedForwardConfig,
+                                                   ManatarConfig, ManatarLayerConfig, MatrixLstmConfig,
+                                                   PairTableConfig)
+    from helix_runtime_b200.config.rorovik import RotaryScalingConfig
+    heads, dim, width = shape["num_attention_heads"], shape["head_dim"], shape["hidden_size"]
+    ff = -(-shape["intermediate_size"] // 4 // 128) * 128
+    dense = FeedForwardConfig(kind="dense", ff=shape["intermediate_size"], limit=7.0)
+    routed = FeedForwardConfig(kind="moe", ff=ff, experts=16, top=3, shared_ff=ff)
+    lstm = MatrixLstmConfig(heads=max(1, heads // 4), dim=2 * dim, vdim=4 * dim, gate_cap=15.0)
+
+    def attention(source):
+        return DifferentialAttentionConfig(
+            heads=heads, kv_heads=options.kv_heads or max(1, heads // 4), dim=dim // 2, vdim=dim,
+            scale=1.0 / math.sqrt(dim // 2), conv=4, diff=0.3, rot_base=500000.0,
+            rot_dims=dim // 2 // 2 * 2,
+            scaling=RotaryScalingConfig(factor=8.0, original=1024, fast=32.0, slow=1.0), kv_from=source)
+    layers = tuple(ManatarLayerConfig(
+        *(("mlstm", lstm) if index % 2 else
+          ("attention", attention(index - 2 if index % 4 == 2 else None))),
+        dense if index == 0 else routed) for index in range(shape["num_hidden_layers"]))
+    return ManatarConfig(vocab=shape["vocab_size"], width=width, norm_eps=shape["rms_norm_eps"],
+                         residual_mult=0.5, pairs=PairTableConfig(65536, 31, 17), layers=layers,
+                         max_positions=shape["max_position_embeddings"])
+
+
 def compare_designs(options, peaks, device) -> int:
     """``--compare``: the Rekasun design beside the Llama design at equal layer sizes
     (``--compare zuzadra``: and the Zuzadra design beside both), a few
@@ -591,16 +627,18 @@ def compare_designs(options, peaks, device) -> int:
         row = {"hidden": shape["hidden_size"], "heads": shape["num_attention_heads"],
                "head_dim": shape["head_dim"], "intermediate": shape["intermediate_size"]}
         designs = [("llama", LlamaConfig(**shape))]
-        if options.compare not in ("rorovik", "pizilix"):
+        if options.compare not in ("rorovik", "pizilix", "manatar"):
             designs.append(("rekasun", rekasun_config(shape, options)))
         if options.compare in ("zuzadra", "medolorn", "pizilix"):
             designs.append(("zuzadra", zuzadra_config(shape, options)))
-        if options.compare in ("medolorn", "rorovik"):
+        if options.compare in ("medolorn", "rorovik", "manatar"):
             designs.append(("medolorn", medolorn_config(shape, options)))
-        if options.compare in ("rorovik", "pizilix"):
+        if options.compare in ("rorovik", "pizilix", "manatar"):
             designs.append(("rorovik", rorovik_config(shape, options)))
         if options.compare == "pizilix":
             designs.append(("pizilix", pizilix_config(shape, options)))
+        if options.compare == "manatar":
+            designs.append(("manatar", manatar_config(shape, options)))
         for design, config in designs:
             model = random_model(config, seed=0, dtype="bfloat16", device=device)
             row[design] = measure(model)
@@ -611,7 +649,8 @@ def compare_designs(options, peaks, device) -> int:
         "metric": "prefill and decode throughput, " + {"zuzadra": "Zuzadra and Rekasun",
                                                         "medolorn": "Medolorn, Zuzadra and Rekasun",
                                                         "rorovik": "Rorovik and Medolorn",
-                                                        "pizilix": "Pizilix, Rorovik and Zuzadra"}
+                                                        "pizilix": "Pizilix, Rorovik and Zuzadra",
+                                                        "manatar": "Manatar, Rorovik and Medolorn"}
                   .get(options.compare, "Rekasun") +
                   " design beside Llama design (bf16)",
         "layers": layers, "prefill_tokens": PREFILL_TOKENS, "decode_context": context,
@@ -647,19 +686,20 @@ def main() -> int:
                         help="layer sizes for --serving, --profile and --timeline (the contract "
                              "line is always the Llama-2-7B shape)")
     parser.add_argument("--design", choices=("llama", "rekasun", "zuzadra", "medolorn", "rorovik",
-                                           "pizilix"),
+                                           "pizilix", "manatar"),
                         default="llama",
                         help="which decoder the layers of --shape are built as, for --profile "
                              "and --timeline (the contract line is always the Llama design)")
     parser.add_argument("--compare", nargs="?", const="rekasun", default=None,
-                        choices=("rekasun", "zuzadra", "medolorn", "rorovik", "pizilix"),
+                        choices=("rekasun", "zuzadra", "medolorn", "rorovik", "pizilix", "manatar"),
                         help="prefill and decode throughput of the Rekasun design beside the "
                              "Llama design at equal layer sizes (a few layers of each --shape), "
                              "as one JSON line of its own; '--compare zuzadra' adds the Zuzadra "
                              "design as a third row, '--compare medolorn' the Medolorn design "
                              "as a fourth; '--compare rorovik' runs the Llama, Medolorn and "
                              "Rorovik designs, '--compare pizilix' the Llama, Zuzadra, Rorovik "
-                             "and Pizilix designs")
+                             "and Pizilix designs, '--compare manatar' the Llama, Medolorn, "
+                             "Rorovik and Manatar designs")
     parser.add_argument("--window", type=int, default=1024,
                         help="--design rekasun / --compare: keys a position sees behind itself")
     parser.add_argument("--keep-first", type=int, default=64,
@@ -722,6 +762,8 @@ def main() -> int:
         config = rorovik_config(shape, options)
     elif options.design == "pizilix":
         config = pizilix_config(shape, options)
+    elif options.design == "manatar":
+        config = manatar_config(shape, options)
     model = random_model(config, seed=0, dtype="bfloat16", device=device)
     rng = np.random.default_rng(0)
     out_dir = options.log_dir or tempfile.mkdtemp(prefix="helix_bench_")

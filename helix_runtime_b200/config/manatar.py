@@ -238,7 +238,7 @@ class ManatarConfig:
     @staticmethod
     def random_scale(name: str, shape: Tuple[int, ...]):
         """What a model with random weights holds in its vectors (None: ones): biases are zero, the
-        maps' vectors small, and a filter passes the token itself on."""
+        vectors of the maps' balance small."""
         leaf = name.rsplit(".", 1)[-1]
         if leaf == "b":
             return 0.0

@@ -45,7 +45,7 @@ class BlockSpec:
     ``streams`` is the pre-norm order over several residual streams: each sublayer is joined to
     them by a connection part (``mixer_connection``, ``feed_forward_connection``), which reads a
     weighted sum of the streams for the norm and rewrites all streams from the sublayer's output.
-    ``post_norm`` has no norms in front: ``x += c N1(mixer(x)); x += c N2(ff(x))`` with the norms and
+    ``output_norm`` has no norms in front: ``x += c N1(mixer(x)); x += c N2(ff(x))`` with the norms and
     the constant in ``post_norm`` connections; ``mixer_norm`` and ``feed_forward_norm`` are ``None``.
     """
 

@@ -27,6 +27,7 @@ SOURCES = (
     "hx_streams.cu",
     "hx_recurrent.cu",
     "hx_matrix_lstm.cu",
+    "hx_state_chunks.cu",
     "hx_map_attention.cu",
     "hx_gated_recurrence.cu",
     "hx_rotary_norm.cu",

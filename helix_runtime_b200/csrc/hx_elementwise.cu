@@ -145,49 +145,77 @@ __global__ void embed_pairs_kernel(const T* __restrict__ table, const T* __restr
   hx_pdl_prologue();
   const int token = blockIdx.x;
   const int id = ids[token];
+  const bool known = id >= 0 && id < vocab;
+  // one thread follows the chain to the previous token while the others fetch the token's own row
   if (threadIdx.x == 0) {
     const int request = token_request[token];
-    const int start = request_start[request];
+    const int position = positions[token];
+    const int ahead = token > 0 ? ids[token - 1] : 0;
+    const int start = request_start[request], end = request_start[request + 1];
+    const int slot = request_slot[request];
     long long row = buckets;
-    int before = 0;
-    if (token > start) before = ids[token - 1];
+    int before = ahead;
     if (token == start) {
-      int* kept = previous + static_cast<size_t>(request_slot[request]) * state_stride;
+      int* kept = previous + static_cast<size_t>(slot) * state_stride;
       before = *kept;
-      *kept = ids[request_start[request + 1] - 1];
+      *kept = ids[end - 1];
     }
-    if (positions[token] > 0) {
+    if (position > 0) {
       row = (static_cast<long long>(before) * mul_prev + static_cast<long long>(id) * mul_cur) % buckets;
       if (row < 0) row += buckets;
     }
     shared_row = static_cast<int>(row);
   }
-  __syncthreads();
   float* row_out = out + static_cast<size_t>(token) * hidden;
-  if (id < 0 || id >= vocab) {
+  const T* own = table + static_cast<size_t>(known ? id : 0) * hidden;
+  if constexpr (sizeof(T) == 2) {
+    constexpr int HELD = 4;
+    if (hidden % 8 == 0 && hidden <= 8 * HELD * static_cast<int>(blockDim.x) &&
+        ((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(pairs) |
+          reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
+      const int pieces = hidden / 8;
+      uint4 x[HELD], y[HELD];
+#pragma unroll
+      for (int i = 0; i < HELD; ++i) {
+        const int p = threadIdx.x + i * blockDim.x;
+        if (p < pieces) x[i] = reinterpret_cast<const uint4*>(own)[p];
+      }
+      __syncthreads();
+      const uint4* pair = reinterpret_cast<const uint4*>(pairs + static_cast<size_t>(shared_row) * hidden);
+#pragma unroll
+      for (int i = 0; i < HELD; ++i) {
+        const int p = threadIdx.x + i * blockDim.x;
+        if (p < pieces) y[i] = pair[p];
+      }
+      const float nan = __int_as_float(0x7fc00000);
+#pragma unroll
+      for (int i = 0; i < HELD; ++i) {
+        const int p = threadIdx.x + i * blockDim.x;
+        if (p >= pieces) continue;
+        const __nv_bfloat162* a = reinterpret_cast<const __nv_bfloat162*>(&x[i]);
+        const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&y[i]);
+        float v[8];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const float2 f = __bfloat1622float2(a[k]), g = __bfloat1622float2(b[k]);
+          v[2 * k] = known ? fmaf(f.x, scale, g.x) : nan;
+          v[2 * k + 1] = known ? fmaf(f.y, scale, g.y) : nan;
+        }
+        float4* wide = reinterpret_cast<float4*>(row_out);
+        wide[2 * p] = make_float4(v[0], v[1], v[2], v[3]);
+        wide[2 * p + 1] = make_float4(v[4], v[5], v[6], v[7]);
+      }
+      if (!known && threadIdx.x == 0 && status != nullptr) atomicOr(status, HX_FLAG_BAD_TOKEN);
+      return;
+    }
+  }
+  __syncthreads();
+  if (!known) {
     for (int c = threadIdx.x; c < hidden; c += blockDim.x) row_out[c] = __int_as_float(0x7fc00000);
     if (threadIdx.x == 0 && status != nullptr) atomicOr(status, HX_FLAG_BAD_TOKEN);
     return;
   }
-  const T* own = table + static_cast<size_t>(id) * hidden;
   const T* pair = pairs + static_cast<size_t>(shared_row) * hidden;
-  if constexpr (sizeof(T) == 2) {
-    if (hidden % 4 == 0 && ((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(pairs) |
-                             reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
-#pragma unroll 4
-      for (int q = threadIdx.x; q < hidden / 4; q += blockDim.x) {
-        const uint2 x = reinterpret_cast<const uint2*>(own)[q];
-        const uint2 y = reinterpret_cast<const uint2*>(pair)[q];
-        const float2 x0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.x));
-        const float2 x1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x.y));
-        const float2 y0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&y.x));
-        const float2 y1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&y.y));
-        reinterpret_cast<float4*>(row_out)[q] = make_float4(
-            fmaf(x0.x, scale, y0.x), fmaf(x0.y, scale, y0.y), fmaf(x1.x, scale, y1.x), fmaf(x1.y, scale, y1.y));
-      }
-      return;
-    }
-  }
   for (int c = threadIdx.x; c < hidden; c += blockDim.x)
     row_out[c] = fmaf(hx_to_float<T>(own[c]), scale, hx_to_float<T>(pair[c]));
 }
@@ -201,7 +229,7 @@ HX_API int hx_embed_pairs(const void* table, const void* pairs, int dtype, const
   HX_REQUIRE(tokens >= 0 && hidden > 0 && vocab > 0 && buckets > 0 && state_stride >= 1 && previous != nullptr,
              "hx_embed_pairs: bad sizes");
   if (tokens == 0) return HX_OK;
-  const int threads = hidden >= 1024 ? 256 : 128;
+  const int threads = hidden >= 2048 ? 256 : 128;
   if (dtype == HX_F32) {
     hx_launch(embed_pairs_kernel<float>, tokens, threads, 0, stream, static_cast<const float*>(table),
               static_cast<const float*>(pairs), ids, positions, token_request, request_slot,

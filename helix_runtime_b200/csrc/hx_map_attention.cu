@@ -14,11 +14,12 @@
 // are q_m . k_m, no attention kernel knows of maps, and a key and its value are cached once.
 // Queries leave in rows of row_dim per (head, map), keys and values go to their pages.
 //
-// A warp owns one unit (a map of a query or key head, or a value head) of a run of consecutive
-// tokens; a lane holds pairs of neighbouring channels, so the norm is a warp's sum and a rotation
-// stays inside a lane.  Only the first taps - 1 tokens of a request's portion reach behind it, into
-// the request's state (its last taps - 1 inputs): the warp of the portion's first token works on all
-// of them and then writes the new state, so one warp per (request, unit) touches it.
+// A unit is a map of a query or key head, or a value head.  Heads in whole 16-byte pieces: a lane owns
+// one piece (8 channels) of a run of consecutive tokens, 2^n neighbouring lanes a unit; other even
+// sizes: a warp owns a unit, a lane pairs of channels; any sizes: the same without a run.  Either way
+// the norm is a sum over lanes and a rotation stays inside a lane.  Only the first taps - 1 tokens of a request's portion reach behind it, into
+// the request's state (its last taps - 1 inputs): whoever has the portion's first token works on all
+// of them and then writes the new state, so one owner per (request, unit) touches it.
 //
 // hx_map_difference.  With a1, a2 the attention results of a head's two maps: o = a1 - lambda a2,
 // over sqrt(mean(o^2) + eps), times `scale`, times sigmoid(g); a warp per (token, head).
@@ -382,6 +383,249 @@ __global__ __launch_bounds__(128) void filtered_heads_pairs_kernel(
   }
 }
 
+// bfloat16 rows whose heads are whole pieces of 8 channels, up to four taps.
+__device__ __forceinline__ void unpack_piece(const uint4& packed, float (&x)[8]) {
+  const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&packed);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 v = __bfloat1622float2(pairs[i]);
+    x[2 * i] = v.x;
+    x[2 * i + 1] = v.y;
+  }
+}
+
+constexpr int EARLY_START_TOKENS = 16;
+
+template <int TAPS>
+__global__ __launch_bounds__(128) void filtered_heads_pieces_kernel(
+    const FilteredHeadsArgs<__nv_bfloat16> a, int qk_lanes, int v_lanes) {
+  constexpr int REACH = TAPS - 1;
+  // few tokens: the attention kernel behind may find its keys while this one runs; with more, all of
+  // its warps would leave their wait at once and stay in step, which costs more than the start saves
+  if (a.tokens <= EARLY_START_TOKENS) hx_pdl_trigger();
+  const int first = blockIdx.x * a.run;
+  const int last = min(first + a.run, a.tokens);
+  const int index = blockIdx.y * blockDim.x + threadIdx.x;     // among a token's lanes
+  const int qk_units = (a.heads + a.kv_heads) * a.maps;
+  const bool is_value = index >= qk_units * qk_lanes;
+  const int own_lanes = is_value ? v_lanes : qk_lanes;
+  const int within = is_value ? index - qk_units * qk_lanes : index;
+  const int unit = within / own_lanes, piece = within - unit * own_lanes;
+  // idle lanes (behind the last unit, or behind a unit's pieces) take part in the sums with zeros
+  const bool live = is_value ? unit < a.kv_heads && 8 * piece < a.vdim : 8 * piece < a.dim;
+  Unit u = unit_of(a, is_value ? (unit < a.kv_heads ? qk_units + unit : 0) : unit);
+  const int c0 = u.column + 8 * piece;
+  float w[TAPS][8], bias[8], weight[8];
+  {
+    float flat[8 * TAPS];
+    const float4* source = reinterpret_cast<const float4*>(a.filter + static_cast<size_t>(c0) * TAPS);
+#pragma unroll
+    for (int v = 0; v < 2 * TAPS; ++v) {
+      const float4 x = live ? source[v] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+      flat[4 * v] = x.x; flat[4 * v + 1] = x.y; flat[4 * v + 2] = x.z; flat[4 * v + 3] = x.w;
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int i = 0; i < 8; ++i) w[j][i] = flat[i * TAPS + j];
+  }
+  const float* norm = u.kind == 0 ? a.q_norm : a.k_norm;
+  const bool normed = u.kind != 2 && norm != nullptr;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    bias[i] = live && a.bias != nullptr ? a.bias[c0 + i] : 0.0f;
+    weight[i] = live && normed ? norm[8 * piece + i] : 1.0f;
+  }
+  int request = a.token_request[first];
+  int start = a.request_start[request], end = a.request_start[request + 1];
+  int slot = a.request_slot[request];
+  hx_pdl_wait();
+
+  const int R = a.row_dim, half = a.rot >> 1, own = u.kind == 2 ? 0 : u.map * a.dim;
+  const float over = 1.0f / static_cast<float>(u.width);
+  auto finish = [&](int token, int position, float (&y)[8]) {
+    if (a.q_norm != nullptr || a.k_norm != nullptr) {
+      float sum = 0.0f;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) sum = fmaf(y[i], y[i], sum);
+#pragma unroll
+      for (int offset = 1; offset < 32; offset <<= 1) {
+        const float other = __shfl_xor_sync(0xffffffffu, sum, offset);
+        if (offset < own_lanes) sum += other;
+      }
+      const float unit_scale = normed ? 1.0f / sqrtf(fmaf(sum, over, a.eps)) : 1.0f;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) y[i] *= unit_scale * weight[i];
+    }
+    if (!live) return;
+    if (u.kind != 2 && 8 * piece < a.rot) {
+      if (position >= a.table_rows) {
+        if (a.status != nullptr) atomicOr(a.status, HX_FLAG_BAD_POSITION);
+        return;
+      }
+      const float* cosine = a.cosine + static_cast<size_t>(position) * half + 4 * piece;
+      const float* sine = a.sine + static_cast<size_t>(position) * half + 4 * piece;
+      float c[4], s[4];
+      if ((a.rot & 7) == 0) {
+        const float4 c4 = *reinterpret_cast<const float4*>(cosine), s4 = *reinterpret_cast<const float4*>(sine);
+        c[0] = c4.x; c[1] = c4.y; c[2] = c4.z; c[3] = c4.w;
+        s[0] = s4.x; s[1] = s4.y; s[2] = s4.z; s[3] = s4.w;
+      } else {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const bool turns = 4 * piece + i < half;
+          c[i] = turns ? cosine[i] : 1.0f;
+          s[i] = turns ? sine[i] : 0.0f;
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float x = y[2 * i], z = y[2 * i + 1];
+        y[2 * i] = x * c[i] - z * s[i];
+        y[2 * i + 1] = z * c[i] + x * s[i];
+      }
+    }
+    uint4 packed;
+    __nv_bfloat162* pairs = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) pairs[i] = __floats2bfloat162_rn(y[2 * i], y[2 * i + 1]);
+    const uint4 zeros = make_uint4(0u, 0u, 0u, 0u);
+    if (u.kind == 0) {
+      // the row's other pieces are zeros, dealt to the unit's lanes
+      uint4* row = reinterpret_cast<uint4*>(a.out + static_cast<size_t>(token) * a.ld_out +
+                                            (u.head * a.maps + u.map) * R);
+      row[(own >> 3) + piece] = packed;
+      const int mine = a.dim >> 3, from = own >> 3, others = (R >> 3) - mine;
+      for (int p = piece; p < others; p += mine) row[p < from ? p : p + mine] = zeros;
+      return;
+    }
+    const int page = a.block_tables[static_cast<size_t>(slot) * a.table_stride + position / a.page_size];
+    if (page < 0 || page >= a.num_pages) {
+      if (a.status != nullptr) atomicOr(a.status, HX_FLAG_BAD_PAGE);
+      return;
+    }
+    __nv_bfloat16* cache = u.kind == 1 ? a.k_cache : a.v_cache;
+    const int place = position % a.page_size;
+    auto at = [&](int d) {
+      return reinterpret_cast<uint4*>(cache + hx_cache_offset(page, u.head, place, d, a.kv_heads, a.page_size, R, 8));
+    };
+    *at(own + 8 * piece) = packed;
+    const int used = u.kind == 2 ? a.vdim : a.maps * a.dim;
+    if (u.kind == 2 || u.map == a.maps - 1)
+      for (int d = used + 8 * piece; d < R; d += u.width) *at(d) = zeros;
+  };
+  auto packed_input = [&](int token) {
+    if (!live) return make_uint4(0u, 0u, 0u, 0u);
+    if (a.accum == nullptr)
+      return *reinterpret_cast<const uint4*>(a.raw + static_cast<size_t>(token) * a.ld_raw + c0);
+    const float4* source =
+        reinterpret_cast<const float4*>(a.accum + static_cast<size_t>(token) * a.ld_accum + c0);
+    const float4 lo = source[0], hi = source[1];
+    uint4 packed;
+    __nv_bfloat162* pairs = reinterpret_cast<__nv_bfloat162*>(&packed);
+    pairs[0] = __floats2bfloat162_rn(lo.x, lo.y);
+    pairs[1] = __floats2bfloat162_rn(lo.z, lo.w);
+    pairs[2] = __floats2bfloat162_rn(hi.x, hi.y);
+    pairs[3] = __floats2bfloat162_rn(hi.z, hi.w);
+    return packed;
+  };
+  // inside a portion the bias passes the filter as a constant
+  float inside[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    float sum = 0.0f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) sum += w[j][i];
+    inside[i] = sum * bias[i];
+  }
+  uint4 rows[TAPS];      // inputs of tokens token - REACH .. token, without the bias
+#pragma unroll
+  for (int j = 0; j < REACH; ++j)
+    rows[j] = first - REACH + j >= start ? packed_input(first - REACH + j) : make_uint4(0u, 0u, 0u, 0u);
+  uint4 ahead = packed_input(first);
+#pragma unroll 1
+  for (int token = first; token < last; ++token) {
+    rows[REACH] = ahead;
+    if (token + 1 < last) ahead = packed_input(token + 1);
+    if (token >= end) {
+      request = a.token_request[token];
+      start = a.request_start[request];
+      end = a.request_start[request + 1];
+      slot = a.request_slot[request];
+    }
+    const int place = token - start;
+    if (place >= REACH && place > 0) {
+      float y[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) y[i] = inside[i];
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        float x[8];
+        unpack_piece(rows[j], x);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) y[i] = fmaf(w[j][i], x[i], y[i]);
+      }
+      finish(token, a.positions[token], y);
+    } else if (place == 0) {
+      const int count = end - start, position = a.positions[token];
+      float* state = a.state + static_cast<size_t>(slot) * a.state_stride + c0;
+      // an input with its bias: the portion's own, or in front of it the state's
+      auto load = [&](int at, float (&x)[8]) {
+        if (at >= 0) {
+          unpack_piece(packed_input(start + at), x);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) x[i] += bias[i];
+        } else {
+#pragma unroll
+          for (int i = 0; i < 8; i += 4) {
+            const float4 v = live ? *reinterpret_cast<const float4*>(
+                                        state + static_cast<size_t>(at + REACH) * a.channels + i)
+                                  : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            x[i] = v.x; x[i + 1] = v.y; x[i + 2] = v.z; x[i + 3] = v.w;
+          }
+        }
+      };
+      const int behind = REACH > 0 ? min(REACH, count) : 1;
+#pragma unroll 1
+      for (int t = 0; t < behind; ++t) {
+        float y[8] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+          float x[8];
+          load(t - REACH + j, x);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) y[i] = fmaf(w[j][i], x[i], y[i]);
+        }
+        finish(start + t, position + t, y);
+      }
+      // the new state: the last REACH inputs up to the portion's end (ascending rows read ahead of
+      // where they write)
+#pragma unroll
+      for (int r = 0; r < REACH; ++r) {
+        float x[8];
+        load(count - REACH + r, x);
+        if (live) {
+          float* target = state + static_cast<size_t>(r) * a.channels;
+          *reinterpret_cast<float4*>(target) = make_float4(x[0], x[1], x[2], x[3]);
+          *reinterpret_cast<float4*>(target + 4) = make_float4(x[4], x[5], x[6], x[7]);
+        }
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < REACH; ++j) rows[j] = rows[j + 1];
+  }
+}
+
+bool heads_pieces_apply(const FilteredHeadsArgs<__nv_bfloat16>& a) {
+  auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  return a.taps <= 4 && a.dim % 8 == 0 && a.dim <= 256 && a.row_dim % 8 == 0 && a.ld_out % 8 == 0 &&
+         aligned(a.out) && aligned(a.filter) && (a.taps == 1 || aligned(a.state)) &&
+         a.state_stride % 4 == 0 && (a.rot == 0 || (aligned(a.cosine) && aligned(a.sine))) &&
+         (a.accum != nullptr ? a.ld_accum % 4 == 0 && aligned(a.accum) : a.ld_raw % 8 == 0 && aligned(a.raw)) &&
+         (a.kv_heads == 0 ||
+          (a.vdim % 8 == 0 && a.vdim <= 256 && aligned(a.k_cache) && aligned(a.v_cache)));
+}
+
 bool heads_pairs_apply(const FilteredHeadsArgs<__nv_bfloat16>& a) {
   auto aligned = [](const void* p, uintptr_t to) { return (reinterpret_cast<uintptr_t>(p) & (to - 1)) == 0; };
   return a.taps <= 4 && a.dim % 2 == 0 && a.vdim % 2 == 0 && a.dim <= 256 && a.vdim <= 256 &&
@@ -408,6 +652,23 @@ template <typename T>
 void launch_filtered_heads(FilteredHeadsArgs<T> a, cudaStream_t stream) {
   const int units = (a.heads + a.kv_heads) * a.maps + a.kv_heads;
   if constexpr (sizeof(T) == 2) {
+    if (heads_pieces_apply(a)) {
+      auto lanes = [](int width) {
+        int n = 1;
+        while (8 * n < width) n *= 2;
+        return n;
+      };
+      a.run = a.tokens >= 1024 ? 8 : (a.tokens >= 256 ? 4 : 1);
+      const int qk_lanes = lanes(a.dim), v_lanes = lanes(a.vdim);
+      const int all = (a.heads + a.kv_heads) * a.maps * qk_lanes + a.kv_heads * v_lanes;
+      const dim3 grid((a.tokens + a.run - 1) / a.run, (all + 127) / 128);
+      switch (a.taps) {
+        case 1: hx_launch(filtered_heads_pieces_kernel<1>, grid, 128, 0, stream, a, qk_lanes, v_lanes); return;
+        case 2: hx_launch(filtered_heads_pieces_kernel<2>, grid, 128, 0, stream, a, qk_lanes, v_lanes); return;
+        case 3: hx_launch(filtered_heads_pieces_kernel<3>, grid, 128, 0, stream, a, qk_lanes, v_lanes); return;
+        default: hx_launch(filtered_heads_pieces_kernel<4>, grid, 128, 0, stream, a, qk_lanes, v_lanes); return;
+      }
+    }
     if (heads_pairs_apply(a)) {
       a.run = a.tokens >= 1024 ? 8 : (a.tokens >= 256 ? 4 : 1);
       const dim3 grid((a.tokens + a.run - 1) / a.run, (units + 3) / 4);

@@ -18,7 +18,8 @@
 //     a time.  d is taken from the rounded maxima that S is scaled by: the difference of two
 //     neighbouring maxima is exact, so a rounding of m (which may be larger than f itself when a
 //     gate hardly forgets) is a change of scale that d undoes, not an error of S.
-//   * scan: token by token, any sizes, both engines; a decode step takes its gates here.
+//   * scan: token by token, any sizes, both engines; a decode step takes its gates here.  Prompt
+//     portions in bfloat16 go through hx_state_chunks instead.
 //   * finish: division, norm, weight and gate; in a decode step also the new maximum, and the
 //     projection's sums are cleared.
 #include "hx_scan.cuh"
@@ -349,27 +350,156 @@ __global__ __launch_bounds__(FINISH_WARPS * 32) void matrix_lstm_finish_kernel(c
   }
 }
 
+// The same in pieces of four numbers: GROUP threads take a head of a token.
+__device__ __forceinline__ float4 row_quad(const LstmArgs<float>& a, size_t token, int c) {
+  return *reinterpret_cast<const float4*>((a.accum != nullptr ? a.accum + token * a.ld_accum
+                                                              : a.rows + token * a.ld) + c);
+}
+__device__ __forceinline__ float4 row_quad(const LstmArgs<__nv_bfloat16>& a, size_t token, int c) {
+  uint2 packed;
+  if (a.accum != nullptr) {
+    const float4 v = *reinterpret_cast<const float4*>(a.accum + token * a.ld_accum + c);
+    *reinterpret_cast<__nv_bfloat162*>(&packed.x) = __floats2bfloat162_rn(v.x, v.y);
+    *reinterpret_cast<__nv_bfloat162*>(&packed.y) = __floats2bfloat162_rn(v.z, v.w);
+  } else {
+    packed = *reinterpret_cast<const uint2*>(a.rows + token * a.ld + c);
+  }
+  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&packed.x));
+  const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&packed.y));
+  return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+__device__ __forceinline__ void put_quad(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put_quad(__nv_bfloat16* p, float4 v) {
+  uint2 packed;
+  *reinterpret_cast<__nv_bfloat162*>(&packed.x) = __floats2bfloat162_rn(v.x, v.y);
+  *reinterpret_cast<__nv_bfloat162*>(&packed.y) = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = packed;
+}
+// the gate's sigmoid: results stored in bfloat16 take the hardware exponential
+template <typename T> __device__ __forceinline__ float gate_of(float x) {
+  return sizeof(T) == 4 ? hx_sigmoid(x) : __fdividef(1.0f, 1.0f + __expf(-x));
+}
+
+template <typename T, bool ONE_TOKEN, int GROUP>
+__global__ __launch_bounds__(128) void matrix_lstm_finish_quads_kernel(const LstmArgs<T> a) {
+  __shared__ float scratch[32];
+  hx_pdl_prologue();
+  const size_t token = blockIdx.x;
+  const int head = blockIdx.y * (128 / GROUP) + threadIdx.x / GROUP, lane = threadIdx.x & (GROUP - 1);
+  if (GROUP == 32 && head >= a.heads) return;          // a block of one group has its head
+  const int vdim = a.vdim, quads = vdim >> 2;
+  const float4* o = reinterpret_cast<const float4*>(a.o + token * (static_cast<size_t>(a.heads) * vdim) + head * vdim);
+  const int g_at = a.heads * (2 * a.dim + vdim) + head * vdim;
+  float4 held[2], gate[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int q = lane + GROUP * i;
+    held[i] = q < quads ? o[q] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    gate[i] = q < quads ? row_quad(a, token, g_at + 4 * q) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  }
+  const size_t at = static_cast<size_t>(head) * a.ld_gates + token;
+  float level, m = 0.0f;
+  float* kept = nullptr;
+  if (ONE_TOKEN) {
+    kept = a.state + static_cast<size_t>(a.request_slot[a.token_request[token]]) * a.state_stride +
+           static_cast<size_t>(a.heads) * a.head_stride + head;
+    float log_decay, push;
+    one_gate(a, token, head, *kept, m, log_decay, push);
+    level = expf(-m);
+  } else {
+    level = a.level[at];
+  }
+  const float inverse = 1.0f / (fmaxf(fabsf(a.weight[at]), level) + a.floor);
+  float sum = 0.0f;
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    held[i].x *= inverse; held[i].y *= inverse; held[i].z *= inverse; held[i].w *= inverse;
+    sum = fmaf(held[i].x, held[i].x, sum); sum = fmaf(held[i].y, held[i].y, sum);
+    sum = fmaf(held[i].z, held[i].z, sum); sum = fmaf(held[i].w, held[i].w, sum);
+  }
+  if (GROUP == 32) {
+#pragma unroll
+    for (int offset = 16; offset > 0; offset >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, offset);
+  } else {
+    sum = hx_block_sum(sum, scratch);
+  }
+  const float unit = 1.0f / sqrtf(sum / static_cast<float>(vdim) + a.eps);
+  T* out = a.out + token * a.ld_out + head * vdim;
+  const float4* norm = reinterpret_cast<const float4*>(a.norm + head * vdim);
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int q = lane + GROUP * i;
+    if (q >= quads) continue;
+    const float4 w = norm[q];
+    put_quad(out + 4 * q, make_float4(held[i].x * unit * w.x * gate_of<T>(gate[i].x),
+                                      held[i].y * unit * w.y * gate_of<T>(gate[i].y),
+                                      held[i].z * unit * w.z * gate_of<T>(gate[i].z),
+                                      held[i].w * unit * w.w * gate_of<T>(gate[i].w)));
+  }
+  // everybody has read the old maximum and the gates' sums (the sum above synchronised the group)
+  if (ONE_TOKEN && lane == 0) *kept = m;
+  if (a.clear != nullptr) {
+    float* row = a.clear + token * a.ld_accum;
+    const float4 zeros = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    for (int q = lane; q < a.dim >> 2; q += GROUP) {
+      put_quad(row + head * a.dim + 4 * q, zeros);
+      put_quad(row + (a.heads + head) * a.dim + 4 * q, zeros);
+    }
+    for (int q = lane; q < quads; q += GROUP) {
+      put_quad(row + 2 * a.heads * a.dim + head * vdim + 4 * q, zeros);
+      put_quad(row + g_at + 4 * q, zeros);
+    }
+    if (lane == 0) {
+      const int gates = 2 * a.heads * (a.dim + vdim);
+      row[gates + head] = 0.0f;
+      row[gates + a.heads + head] = 0.0f;
+    }
+  }
+}
+
+template <typename T, bool ONE_TOKEN>
+void launch_finish(const LstmArgs<T>& a, cudaStream_t stream) {
+  auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  if (a.vdim % 4 == 0 && a.dim % 4 == 0 && a.vdim <= 1024 && a.ld_out % 4 == 0 && aligned(a.o) &&
+      aligned(a.norm) && aligned(a.out) && aligned(a.rows) && aligned(a.accum) &&
+      (a.accum != nullptr ? a.ld_accum : a.ld) % 4 == 0) {
+    if (a.vdim <= 256) {
+      hx_launch(matrix_lstm_finish_quads_kernel<T, ONE_TOKEN, 32>, dim3(a.tokens, (a.heads + 3) / 4), 128, 0,
+                stream, a);
+    } else {
+      hx_launch(matrix_lstm_finish_quads_kernel<T, ONE_TOKEN, 128>, dim3(a.tokens, a.heads), 128, 0, stream, a);
+    }
+    return;
+  }
+  hx_launch(matrix_lstm_finish_kernel<T, ONE_TOKEN>,
+            dim3(a.tokens, (a.heads + FINISH_WARPS - 1) / FINISH_WARPS), FINISH_WARPS * 32, 0, stream, a);
+}
+
 template <typename T>
-int run_matrix_lstm(LstmArgs<T> a, int requests, cudaStream_t stream) {
+int run_matrix_lstm(LstmArgs<T> a, int requests, bool scan, cudaStream_t stream) {
   const int columns = a.vdim + 1;
   a.parts = parts_for(a.dim);
   a.block_lanes = min(columns, SCAN_THREADS / a.parts) * a.parts;
   a.per_token = staged_floats(2, a.dim, a.block_lanes / a.parts + 2);
   a.tile = tile_for(a.per_token);
   HX_REQUIRE(a.tile >= 1, "hx_matrix_lstm: a token's vectors do not fit shared memory");
-  const int threads = (a.block_lanes + 31) / 32 * 32;
-  const int column_blocks = (columns * a.parts + a.block_lanes - 1) / a.block_lanes;
-  const dim3 grid(requests, a.heads, column_blocks);
-  const size_t one_bytes = static_cast<size_t>(a.per_token) * sizeof(float);
-  const dim3 finish_grid(a.tokens, (a.heads + FINISH_WARPS - 1) / FINISH_WARPS);
-  if (a.gate_sums != nullptr) {
-    hx_launch(matrix_lstm_scan_kernel<T, true>, grid, threads, one_bytes, stream, a);
-    hx_launch(matrix_lstm_finish_kernel<T, true>, finish_grid, FINISH_WARPS * 32, 0, stream, a);
-  } else {
-    hx_launch(matrix_lstm_scan_kernel<T, false>, grid, threads, a.tile * one_bytes, stream, a);
-    hx_launch(matrix_lstm_finish_kernel<T, false>, finish_grid, FINISH_WARPS * 32, 0, stream, a);
+  if (scan) {
+    const int threads = (a.block_lanes + 31) / 32 * 32;
+    const int column_blocks = (columns * a.parts + a.block_lanes - 1) / a.block_lanes;
+    const dim3 grid(requests, a.heads, column_blocks);
+    const size_t one_bytes = static_cast<size_t>(a.per_token) * sizeof(float);
+    if (a.gate_sums != nullptr) {
+      hx_launch(matrix_lstm_scan_kernel<T, true>, grid, threads, one_bytes, stream, a);
+    } else {
+      hx_launch(matrix_lstm_scan_kernel<T, false>, grid, threads, a.tile * one_bytes, stream, a);
+    }
+    hx_count_launches(1);
   }
-  hx_count_launches(1);
+  if (a.gate_sums != nullptr) {
+    launch_finish<T, true>(a, stream);
+  } else {
+    launch_finish<T, false>(a, stream);
+  }
   return HX_OK;
 }
 
@@ -408,12 +538,12 @@ HX_API int hx_matrix_lstm_gates(const float* sums, int ld, const float* bias, fl
 // ld_accum] (rounded into `dtype` when read, and cleared): q [heads * dim] | k | v [heads * vdim] | g,
 // accum with the 2 * heads gate columns behind.  gate_sums not null: a decode step (one token per
 // request), gates from these columns; null: gates from hx_matrix_lstm_gates' arrays [heads,
-// ld_gates].  o float32 [tokens, heads * vdim] and weight [heads, ld_gates] are scratch; out [tokens,
-// ld_out] in `dtype`.
+// ld_gates].  scan 0: o float32 [tokens, heads * vdim] and weight [heads, ld_gates] hold the recurrence's
+// results already (hx_state_chunks); else they are scratch.  out [tokens, ld_out] in `dtype`.
 HX_API int hx_matrix_lstm(const void* rows, int ld, float* accum, int ld_accum, int dtype,
                           const float* gate_sums, int ld_gate_sums, const float* bias, float cap,
                           const float* log_decay, const float* push, const float* level, int ld_gates,
-                          float q_scale, float floor, const float* norm, float eps, float* state,
+                          int scan, float q_scale, float floor, const float* norm, float eps, float* state,
                           long long state_stride, float* o, float* weight, void* out, int ld_out,
                           const int* token_request, const int* request_start, const int* request_slot,
                           int requests, int tokens, int heads, int dim, int vdim, cudaStream_t stream) {
@@ -422,6 +552,7 @@ HX_API int hx_matrix_lstm(const void* rows, int ld, float* accum, int ld_accum, 
              "hx_matrix_lstm: bad sizes");
   HX_REQUIRE(parts_for(dim) > 0, "hx_matrix_lstm: heads of %d are more than %d", dim, 32 * 16);
   const int columns = 2 * heads * (dim + vdim);
+  HX_REQUIRE(scan || gate_sums == nullptr, "hx_matrix_lstm: a decode step scans");
   HX_REQUIRE((rows != nullptr) != (accum != nullptr),
              "hx_matrix_lstm: give the projected rows or their sums");
   HX_REQUIRE(rows == nullptr || ld >= columns, "hx_matrix_lstm: row stride too small");
@@ -442,7 +573,7 @@ HX_API int hx_matrix_lstm(const void* rows, int ld, float* accum, int ld_accum, 
                                          weight, norm, static_cast<float*>(out), ld_out, accum,
                                          columns + 2 * heads, request_start, request_slot,
                                          token_request, tokens, heads, dim, vdim, 0, 0, 0, 0},
-                         requests, stream);
+                         requests, scan != 0, stream);
   } else if (dtype == HX_BF16) {
     rc = run_matrix_lstm(LstmArgs<__nv_bfloat16>{
                              static_cast<const __nv_bfloat16*>(rows), ld, accum, ld_accum, q_scale, floor,
@@ -451,7 +582,7 @@ HX_API int hx_matrix_lstm(const void* rows, int ld, float* accum, int ld_accum, 
                              static_cast<__nv_bfloat16*>(out), ld_out, accum, columns + 2 * heads,
                              request_start, request_slot, token_request, tokens, heads, dim, vdim, 0, 0,
                              0, 0},
-                         requests, stream);
+                         requests, scan != 0, stream);
   } else {
     HX_REQUIRE(false, "hx_matrix_lstm: unknown dtype %d", dtype);
   }

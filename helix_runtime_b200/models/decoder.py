@@ -105,7 +105,7 @@ def _run_joined(part, connection, ctx: StepContext, residual: torch.Tensor, norm
     connection.join(ctx, residual, output, normed, bias)
 
 
-def _post_norm(block: "Block", ctx: StepContext, cache: LayerCache, residual: torch.Tensor,
+def _output_norm(block: "Block", ctx: StepContext, cache: LayerCache, residual: torch.Tensor,
                normed: torch.Tensor) -> None:
     # x += c N1(mixer(x)); x += c N2(ff(x)): `normed` is x in the compute dtype throughout
     output = ctx.workspace.accumulator(f"model.sublayer_sums/{block.hidden_size}",
@@ -115,7 +115,7 @@ def _post_norm(block: "Block", ctx: StepContext, cache: LayerCache, residual: to
         _run_joined(block.feed_forward, block.feed_forward_connection, ctx, residual, normed, output)
 
 
-register_arrangement("post_norm", _post_norm, reads_rows=True)
+register_arrangement("output_norm", _output_norm, reads_rows=True)
 
 
 class Block:
@@ -134,11 +134,11 @@ class Block:
                 (spec.feed_forward is not None and (spec.feed_forward_connection is None
                                                     or spec.feed_forward_norm is None))):
             raise ValueError("a streams block joins every sublayer with a connection and a norm")
-        if spec.arrangement == "post_norm" and (
+        if spec.arrangement == "output_norm" and (
                 spec.mixer_norm is not None or spec.feed_forward_norm is not None
                 or spec.mixer_connection is None
                 or (spec.feed_forward is None) != (spec.feed_forward_connection is None)):
-            raise ValueError("a post_norm block joins every sublayer with a connection and has no "
+            raise ValueError("an output_norm block joins every sublayer with a connection and has no "
                              "norm in front of it")
         if spec.mixer_norm is None and spec.arrangement not in _READ_ROWS:
             raise ValueError(f"a {spec.arrangement} block has a norm in front of its mixer")

@@ -92,7 +92,7 @@ def build_manatar_spec(config: ManatarConfig) -> ModelSpec:
         prefix = f"l{index}"
         has_mlp = layer.mlp is not None
         blocks.append(BlockSpec(
-            arrangement="post_norm",
+            arrangement="output_norm",
             mixer_norm=None,
             mixer=MIXER_SPECS[layer.type](prefix, layer.mixer, config),
             feed_forward=_feed_forward(f"{prefix}.mlp", layer.mlp) if has_mlp else None,

@@ -313,11 +313,19 @@ def _declare(library: ctypes.CDLL) -> None:
         _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]
     library.hx_matrix_lstm.argtypes = [
         _c_ptr, _c_int, _c_ptr, _c_int, _c_int, _c_ptr, _c_int, _c_ptr, _c_float, _c_ptr, _c_ptr,
-        _c_ptr, _c_int, _c_float, _c_float, _c_ptr, _c_float, _c_ptr, _c_longlong, _c_ptr, _c_ptr,
-        _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]
+        _c_ptr, _c_int, _c_int, _c_float, _c_float, _c_ptr, _c_float, _c_ptr, _c_longlong, _c_ptr,
+        _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int, _c_ptr]
+    library.hx_state_chunks_supports.argtypes = [_c_int, _c_int]
+    library.hx_state_chunks_scratch.argtypes = [_c_int, _c_int]
+    library.hx_state_chunks_scratch.restype = _c_longlong
+    library.hx_state_chunks.argtypes = [
+        _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_ptr, _c_float, _c_ptr,
+        _c_longlong, _c_int, _c_ptr, _c_ptr, _c_ptr, _c_ptr, _c_int, _c_int, _c_int, _c_int, _c_int,
+        _c_ptr]
     for name in ("hx_embed_pairs", "hx_norm_residual_add_biased", "hx_cast_rows",
                  "hx_route_top_biased", "hx_filtered_heads", "hx_map_difference",
-                 "hx_matrix_lstm_state_floats", "hx_matrix_lstm_gates", "hx_matrix_lstm"):
+                 "hx_matrix_lstm_state_floats", "hx_matrix_lstm_gates", "hx_matrix_lstm",
+                 "hx_state_chunks_supports", "hx_state_chunks"):
         getattr(library, name).restype = _c_int
     for name in ("hx_embed", "hx_rmsnorm", "hx_swiglu", "hx_rope_append", "hx_gemm_simt",
                  "hx_gemm_tc", "hx_gemm_tc_supports", "hx_gemm_tc_token_tile",
@@ -1513,12 +1521,13 @@ def matrix_lstm(projected: torch.Tensor, sums: bool, bias: torch.Tensor, cap: fl
                 q_scale: float, floor: float, norm: torch.Tensor, eps: float, state: torch.Tensor,
                 o: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, token_request: torch.Tensor,
                 request_start: torch.Tensor, request_slot: torch.Tensor, requests: int, tokens: int,
-                heads: int, dim: int, value_dim: int) -> None:
+                heads: int, dim: int, value_dim: int, scan: bool = True) -> None:
     """The matrix memory over the step's tokens, its division, norm, weight and gate.  ``projected`` is
     ``[q | k | v | g]`` in the compute dtype, or (``sums``) float32 sums with the gates' columns behind,
     which are left zero.  ``gate_sums`` (a decode step, one token per request): the gates' columns;
     otherwise ``gates`` are the three arrays of :func:`matrix_lstm_gates`.  ``o [tokens, heads *
-    value_dim]`` and ``weight [heads, >= tokens]`` are float32 scratch."""
+    value_dim]`` and ``weight [heads, >= tokens]`` are float32 scratch, or (``scan=False``) hold the
+    recurrence's results already (:func:`state_chunks`)."""
     _need(o, torch.float32, "o")
     _need(weight, torch.float32, "weight")
     _need(state, torch.float32, "state")
@@ -1532,11 +1541,47 @@ def matrix_lstm(projected: torch.Tensor, sums: bool, bias: torch.Tensor, cap: fl
         None if sums else projected.data_ptr(), 0 if sums else projected.stride(0),
         projected.data_ptr() if sums else None, projected.stride(0) if sums else 0,
         dtype_code(out.dtype), _ptr(gate_sums), 0 if gate_sums is None else gate_sums.stride(0),
-        bias.data_ptr(), float(cap), _ptr(log_decay), _ptr(push), _ptr(level), ld_gates, float(q_scale),
-        float(floor), norm.data_ptr(), float(eps), state.data_ptr(), state.stride(0), o.data_ptr(),
+        bias.data_ptr(), float(cap), _ptr(log_decay), _ptr(push), _ptr(level), ld_gates,
+        1 if scan else 0, float(q_scale), float(floor), norm.data_ptr(), float(eps), state.data_ptr(), state.stride(0), o.data_ptr(),
         weight.data_ptr(), out.data_ptr(), out.stride(0), token_request.data_ptr(),
         request_start.data_ptr(), request_slot.data_ptr(), requests, tokens, heads, dim, value_dim,
         _stream()))
+
+
+def state_chunks_supports(dim: int, value_dim: int) -> bool:
+    """Whether :func:`state_chunks` takes heads of these sizes."""
+    return bool(lib().hx_state_chunks_supports(dim, value_dim))
+
+
+def state_chunks_scratch(heads: int, tokens: int) -> int:
+    """bfloat16 elements of the ``weights`` scratch of :func:`state_chunks`."""
+    return lib().hx_state_chunks_scratch(heads, tokens)
+
+
+def state_chunks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor,
+                 push: torch.Tensor, total: torch.Tensor, weights: torch.Tensor, q_scale: float,
+                 state: torch.Tensor, o: torch.Tensor, extra: torch.Tensor,
+                 request_start: torch.Tensor, request_slot: torch.Tensor, requests: int, tiles: int,
+                 heads: int, dim: int, value_dim: int) -> None:
+    """``S <- e^d S + p k [v, 1]'``, ``o = q_scale S' q`` over every request's portion, 64 tokens at a time
+    on the tensor cores (bfloat16 rows).  ``q``, ``k``, ``v`` are views of the same rows; ``decay`` and
+    ``push`` ``[heads, >= tokens]`` hold ``d`` and ``p`` and are overwritten; ``total`` (like them) and
+    ``weights`` (:func:`state_chunks_scratch`) are scratch; ``extra [heads, >= tokens]`` gets the last
+    column's output.  ``state``: rows of :func:`matrix_lstm_state_floats`.  ``tiles``:
+    :func:`recurrence_tiles` of the step."""
+    for tensor in (decay, push, total, state, o, extra):
+        _need(tensor, torch.float32, "a float32 argument")
+    for tensor in (q, k, v, weights):
+        _need(tensor, torch.bfloat16, "a bfloat16 argument")
+    ld = decay.stride(0)
+    assert q.stride(0) == k.stride(0) == v.stride(0) and o.is_contiguous()
+    assert push.stride(0) == total.stride(0) == extra.stride(0) == ld
+    assert weights.numel() >= state_chunks_scratch(heads, ld)
+    _check(lib().hx_state_chunks(
+        q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), decay.data_ptr(), push.data_ptr(),
+        total.data_ptr(), ld, weights.data_ptr(), float(q_scale), state.data_ptr(), state.stride(0),
+        scan_state_floats(value_dim + 1, dim), o.data_ptr(), extra.data_ptr(), request_start.data_ptr(),
+        request_slot.data_ptr(), requests, tiles, heads, dim, value_dim, _stream()))
 
 
 def expert_gate_up(x: torch.Tensor, gate_up: torch.Tensor, chosen: torch.Tensor,

@@ -287,7 +287,7 @@ class RoutedExperts(FeedForward):
 
     # Fewer pairs than this and an expert's matrices are read about once anyway: a product
     # per pair streams them; from here on the pairs are sorted by expert.
-    GROUPED_FROM_PAIRS = 32
+    GROUPED_FROM_PAIRS = 16
 
     def grouped(self, ctx: StepContext, tokens: int) -> bool:
         return (ctx.dtype == torch.bfloat16 and tokens * self.top >= self.GROUPED_FROM_PAIRS

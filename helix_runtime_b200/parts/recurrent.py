@@ -560,6 +560,8 @@ class MatrixLstm(Mixer):
         self.w_in = matrix("q", "k", "v", "g", "i", "f")
         self.w_gates = matrix("i", "f")
         self.w_o = matrix("o")
+        self.chunked = dtype == torch.bfloat16 and \
+            ops.state_chunks_supports(self.head_dim, self.value_dim)
         self.gate_bias = torch.cat([scale("i_bias"), scale("f_bias")]).contiguous()
         self.norm = scale("norm")
 
@@ -570,10 +572,11 @@ class MatrixLstm(Mixer):
                 residual: torch.Tensor) -> None:
         n, heads, get = ctx.n_tokens, self.heads, ctx.workspace.get
         o = get(f"matrix_lstm.o/{self.v_width}", (ctx.capacity, self.v_width), torch.float32)
-        arrays = get(f"matrix_lstm.gates/{heads}", (4, heads, ctx.capacity), torch.float32)
+        arrays = get(f"matrix_lstm.gates/{heads}", (5, heads, ctx.capacity), torch.float32)
         wide = -(-self.v_width // 8) * 8
         out = get(f"matrix_lstm.out/{wide}", (ctx.capacity, wide), ctx.dtype)[:, :self.v_width]
-        sums = is_weight_stream(x, self.w_in, n)
+        one_token = n == ctx.n_requests
+        sums = one_token and is_weight_stream(x, self.w_in, n)
         if sums:
             size = -(-self.projected_size // 4) * 4
             rows = ctx.workspace.accumulator(f"matrix_lstm.rows/{size}", (STREAMING_MAX_TOKENS, size))
@@ -588,13 +591,24 @@ class MatrixLstm(Mixer):
             project(x, self.w_gates, gate_sums, n, ops.EPI_STORE_F32, ctx.status)
         batch = (ctx.request_start, ctx.request_slot, ctx.n_requests, n, heads, self.head_dim,
                  self.value_dim)
-        one_token = n == ctx.n_requests
+        decay, push, level, weight, total = arrays
+        chunked = not one_token and self.chunked
         if not one_token:
-            ops.matrix_lstm_gates(gate_sums, self.gate_bias, self.gate_cap, arrays[0], arrays[1],
-                                  arrays[2], cache.state, *batch)
-        ops.matrix_lstm(rows, sums, self.gate_bias, self.gate_cap, None if one_token else arrays[:3],
+            ops.matrix_lstm_gates(gate_sums, self.gate_bias, self.gate_cap, decay, push, level,
+                                  cache.state, *batch)
+        if chunked:
+            a, b = self.qk_width, 2 * self.qk_width
+            scratch = ctx.workspace.at_least("matrix_lstm.weights",
+                                             ops.state_chunks_scratch(heads, ctx.capacity), ctx.dtype)
+            ops.state_chunks(rows[:, :a], rows[:, a:b], rows[:, b:b + self.v_width], decay, push, total,
+                             scratch, self.q_scale, cache.state, o, weight, ctx.request_start,
+                             ctx.request_slot, ctx.n_requests,
+                             ops.recurrence_tiles(ctx.host_query_lengths), heads, self.head_dim,
+                             self.value_dim)
+        ops.matrix_lstm(rows, sums, self.gate_bias, self.gate_cap,
+                        None if one_token else (decay, push, level),
                         gate_sums if one_token else None, self.q_scale, self.floor, self.norm, self.eps,
-                        cache.state, o, arrays[3], out, ctx.token_request, *batch)
+                        cache.state, o, weight, out, ctx.token_request, *batch, scan=not chunked)
         project(out, self.w_o, residual, n, ops.EPI_ADD_F32, ctx.status, ctx.ordered_sums)
 
 

@@ -304,7 +304,7 @@ class PlainManatar:
         positions = np.arange(len(tokens), dtype=np.float64)
         self.margins = np.full(len(tokens), np.inf)
         x = self.w["embed"][tokens]
-        pairs = self.config["embedding"].get("bigram")
+        pairs = (self.config.get("embedding") or {}).get("bigram")
         if pairs:
             x = x + self.w["bigram"][pair_rows(tokens, pairs["buckets"], pairs["mul_prev"],
                                                pairs["mul_cur"])]
