@@ -443,8 +443,10 @@ def test_matrix_memory_of_sizes_without_chunks(dtype):
     from helix_runtime_b200.ops import library as ops
     assert not ops.state_chunks_supports(18, 7) and not ops.state_chunks_supports(520, 8)
     rng = np.random.default_rng(71)
-    case = LstmCase(rng, dtype, 3, 18, 7, 4.0, [50, 3])
-    case.check(rounds_of(case.totals, rng), [1, 0], "portions", chunks=False)
+    for heads, dim, vdim in ((3, 18, 7), (1, 5, 1), (40, 3, 2)):
+        case = LstmCase(rng, dtype, heads, dim, vdim, 4.0, [50, 3])
+        case.eps = 0.3      # heads of one or two values: not only their signs
+        case.check(rounds_of(case.totals, rng), [1, 0], f"{heads} {dim} {vdim}", chunks=False)
 
 
 @pytest.mark.parametrize("dtype,chunks", LSTM_FORMS)

@@ -1,9 +1,9 @@
 """Randomly drawn Manatar configurations through the engine against the plain implementation: the
 order and number of layers, layers that use an earlier layer's keys and values, every size of the
-two mixers (heads, grouped key/value heads, maps of 2 to 136 coordinates, values of 6 to 264,
+two mixers (heads, grouped key/value heads, maps of 4 to 136 coordinates, values of 6 to 264,
 filters of 1 to 6 taps, rotation of some or all coordinates with and without stretched
-frequencies; matrices of 1 to 320 by 7 to 264), dense and routed feed-forwards or none, with and
-without a shared expert and a table of pairs (a head of one or two values is normed to little more
+frequencies; matrices of 4 to 320 by 7 to 264), dense and routed feed-forwards or none, with and
+without a shared expert and a table of pairs (a head of one or two numbers is normed to little more
 than their signs, which anything that rounds differently turns where they are near zero: no model
 has such heads); every model is replayed as mixed batches over a pool
 made for its live requests only."""
@@ -43,7 +43,7 @@ def draw_config(seed: int):
                              diff=pick([0.1, 0.5, 0.8]))
                 mixer["scale"] = pick([1.0, 2.0, 4.0]) / math.sqrt(mixer["dim"])
             else:
-                dim, kv_heads = pick([2, 4, 9, 16, 20, 32, 48, 64, 72, 136]), pick([1, 1, 2, 3])
+                dim, kv_heads = pick([4, 6, 9, 16, 20, 32, 48, 64, 72, 136]), pick([1, 1, 2, 3])
                 vdim = pick([6, 7, 16, max(2 * dim, 6), 2 * dim + 6, max(dim, 6), 40, 128]) if rng.random() < 0.9 else 264
                 rot = {"base": float(pick([100.0, 10000.0, 500000.0])),
                        "dims": pick([d for d in (2, dim // 4 * 2, dim) if d % 2 == 0 and d > 0])}
@@ -57,7 +57,7 @@ def draw_config(seed: int):
                          "conv": pick([1, 2, 3, 4, 4, 6]), "diff": pick([0.1, 0.3, 0.6]), "rot": rot}
         else:
             kind = "mlstm"
-            mixer = {"heads": pick([1, 2, 3, 5]), "dim": pick([1, 8, 16, 18, 40, 64, 104, 128, 200, 320]),
+            mixer = {"heads": pick([1, 2, 3, 5]), "dim": pick([4, 8, 16, 18, 40, 64, 104, 128, 200, 320]),
                      "vdim": pick([7, 8, 17, 32, 64, 136, 264]), "gate_cap": float(pick([1.0, 5.0, 15.0]))}
         draw = rng.random()
         mlp = None
