@@ -704,7 +704,8 @@ struct MapDifferenceArgs {
 
 constexpr int DIFFERENCE_WARPS = 4;
 
-// grid (tokens, ceil(heads / DIFFERENCE_WARPS)).  HELD numbers a lane are kept between the passes.
+// grid (tokens, ceil(heads / DIFFERENCE_WARPS)).  HELD numbers a lane are kept between the passes.  Any
+// sizes.
 template <typename T, int HELD>
 __global__ __launch_bounds__(DIFFERENCE_WARPS * 32) void map_difference_kernel(const MapDifferenceArgs<T> a) {
   hx_pdl_prologue();
@@ -756,10 +757,87 @@ __global__ __launch_bounds__(DIFFERENCE_WARPS * 32) void map_difference_kernel(c
   }
 }
 
+// Four numbers at a time, for heads of up to 256 values in whole pieces of four.
+__device__ __forceinline__ float4 load_quad(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load_quad(const __nv_bfloat16* p) {
+  const uint2 packed = *reinterpret_cast<const uint2*>(p);
+  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&packed.x));
+  const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&packed.y));
+  return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+__device__ __forceinline__ void store_quad(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store_quad(__nv_bfloat16* p, float4 v) {
+  uint2 packed;
+  *reinterpret_cast<__nv_bfloat162*>(&packed.x) = __floats2bfloat162_rn(v.x, v.y);
+  *reinterpret_cast<__nv_bfloat162*>(&packed.y) = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = packed;
+}
+// results stored in bfloat16 take the hardware exponential
+template <typename T> __device__ __forceinline__ float gate_factor(float x) {
+  if constexpr (sizeof(T) == 4) return hx_sigmoid(x);
+  return __fdividef(1.0f, 1.0f + __expf(-hx_to_float<T>(hx_from_float<T>(x))));
+}
+
+template <typename T>
+__global__ __launch_bounds__(DIFFERENCE_WARPS * 32) void map_difference_quads_kernel(const MapDifferenceArgs<T> a) {
+  constexpr int HELD = 2;
+  hx_pdl_prologue();
+  const size_t token = blockIdx.x;
+  const int head = blockIdx.y * DIFFERENCE_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (head >= a.heads) return;
+  const T* first = a.context + token * a.ld_context + static_cast<size_t>(2 * head) * a.row_dim;
+  const int quads = a.vdim >> 2, column = head * a.vdim;
+  const float4 zeros = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  float4 x[HELD], y[HELD], g[HELD];
+#pragma unroll
+  for (int i = 0; i < HELD; ++i) {
+    const int q = lane + 32 * i;
+    x[i] = y[i] = g[i] = zeros;
+    if (q < quads) {
+      x[i] = load_quad(first + 4 * q);
+      y[i] = load_quad(first + a.row_dim + 4 * q);
+      g[i] = a.gate_sums != nullptr ? load_quad(a.gate_sums + token * a.ld_sums + column + 4 * q)
+                                    : load_quad(a.gate + token * a.ld_gate + column + 4 * q);
+    }
+  }
+  float sum = 0.0f;
+#pragma unroll
+  for (int i = 0; i < HELD; ++i) {
+    x[i].x -= a.lambda * y[i].x; x[i].y -= a.lambda * y[i].y;
+    x[i].z -= a.lambda * y[i].z; x[i].w -= a.lambda * y[i].w;
+    sum = fmaf(x[i].x, x[i].x, sum); sum = fmaf(x[i].y, x[i].y, sum);
+    sum = fmaf(x[i].z, x[i].z, sum); sum = fmaf(x[i].w, x[i].w, sum);
+  }
+  const float unit = a.scale / sqrtf(warp_sum(sum) / static_cast<float>(a.vdim) + a.eps);
+#pragma unroll
+  for (int i = 0; i < HELD; ++i) {
+    const int q = lane + 32 * i;
+    if (q < quads)
+      store_quad(a.out + token * a.ld_out + column + 4 * q,
+                 make_float4(x[i].x * unit * gate_factor<T>(g[i].x), x[i].y * unit * gate_factor<T>(g[i].y),
+                             x[i].z * unit * gate_factor<T>(g[i].z), x[i].w * unit * gate_factor<T>(g[i].w)));
+  }
+  if (a.clear != nullptr) {
+    // see map_difference_kernel: the head's own gate columns, and its share of the rest
+    float* row = a.clear + token * a.ld_clear;
+    const int rest = (a.clear_width - a.heads * a.vdim) >> 2;
+    const int from = static_cast<int>(static_cast<long long>(rest) * head / a.heads);
+    const int to = static_cast<int>(static_cast<long long>(rest) * (head + 1) / a.heads);
+    for (int q = from + lane; q < to; q += 32) store_quad(row + 4 * q, zeros);
+    for (int q = lane; q < quads; q += 32) store_quad(row + 4 * rest + column + 4 * q, zeros);
+  }
+}
+
 template <typename T>
 void launch_map_difference(const MapDifferenceArgs<T>& a, int tokens, cudaStream_t stream) {
   const dim3 grid(tokens, (a.heads + DIFFERENCE_WARPS - 1) / DIFFERENCE_WARPS);
-  if (a.vdim <= 128) {
+  auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  if (a.vdim % 4 == 0 && a.vdim <= 256 && a.row_dim % 4 == 0 && a.ld_context % 4 == 0 && a.ld_out % 4 == 0 &&
+      (a.gate_sums != nullptr ? a.ld_sums : a.ld_gate) % 4 == 0 && aligned(a.context) && aligned(a.out) &&
+      aligned(a.gate_sums) && (reinterpret_cast<uintptr_t>(a.gate) & 7) == 0 && (sizeof(T) == 2 || aligned(a.gate)) &&
+      (a.clear == nullptr || (a.ld_clear % 4 == 0 && a.clear_width % 4 == 0 && aligned(a.clear)))) {
+    hx_launch(map_difference_quads_kernel<T>, grid, DIFFERENCE_WARPS * 32, 0, stream, a);
+  } else if (a.vdim <= 128) {
     hx_launch(map_difference_kernel<T, 4>, grid, DIFFERENCE_WARPS * 32, 0, stream, a);
   } else {
     hx_launch(map_difference_kernel<T, 8>, grid, DIFFERENCE_WARPS * 32, 0, stream, a);

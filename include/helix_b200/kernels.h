@@ -69,6 +69,14 @@ int hx_embed(const void* table, int dtype, const int* ids, float* out, int token
 /* the same times a constant: out[t, :] = table[ids[t], :] * scale, the product in float32 */
 int hx_embed_scaled(const void* table, int dtype, const int* ids, float* out, int tokens,
                     int hidden, int vocab, float scale, int* status, cudaStream_t stream);
+/* out[t] = table[ids[t]] * scale + pairs[row], row = (previous id * mul_prev + ids[t] * mul_cur) mod
+ * buckets, row `buckets` for a sequence's first token (position 0); previous[slot * state_stride]:
+ * the id in front of a request's portion, updated to its last */
+int hx_embed_pairs(const void* table, const void* pairs, int dtype, const int* ids,
+                   const int* positions, const int* token_request, const int* request_slot,
+                   const int* request_start, int* previous, long long state_stride, float* out,
+                   int tokens, int hidden, int vocab, int buckets, long long mul_prev,
+                   long long mul_cur, float scale, int* status, cudaStream_t stream);
 /* x[t, :] += y[t, :], float32 rows of `hidden` */
 int hx_add_rows(float* x, const float* y, int tokens, int hidden, cudaStream_t stream);
 /* y[r, :] = (x[r', :] - mean) / sqrt(var + eps) * weight + bias, r' = rows ? rows[r] : r, var the
@@ -256,6 +264,13 @@ int hx_join_rows(const float* a, const float* b, void* out, int ld_out, int dtyp
 int hx_norm_residual_add(float* residual, const float* y, const float* weight, float eps,
                          float mult, void* cast_out, int ld_cast, int dtype, int tokens, int width,
                          cudaStream_t stream);
+/* the same with y[t] + bias in place of y[t] (bias may be null); clear: y is left zero */
+int hx_norm_residual_add_biased(float* residual, float* y, const float* bias, int clear,
+                                const float* weight, float eps, float mult, void* cast_out,
+                                int ld_cast, int dtype, int tokens, int width, cudaStream_t stream);
+/* out[t] = x[t] in `dtype` (x float32 [tokens][width]) */
+int hx_cast_rows(const float* x, void* out, int ld_out, int dtype, int tokens, int width,
+                 cudaStream_t stream);
 /* projected float32 = [heads * head_dim q | kv_heads * head_dim k | kv_heads * value_dim v |
  * heads gate sums (with gates)]: biases (may be null), one RMS norm over ALL of a token's q
  * and one over all of its k (weights null: none), q times 1 + temp_coef * ln(floor((p + 1) /
@@ -291,6 +306,11 @@ int hx_route_top(const float* sums, int ld, int tokens, int experts, int top, fl
 int hx_route_top_ruled(const float* sums, int ld, int tokens, int experts, int top, float scale,
                        int softmax, const float* correction, int normalize, int* chosen,
                        float* weights, cudaStream_t stream);
+/* the same with a bias [experts] (may be null) on the sums; softmax 2: the choice is by the sums
+ * themselves, the weights are the softmax over the chosen ones alone */
+int hx_route_top_biased(const float* sums, int ld, int tokens, int experts, int top, float scale,
+                        int softmax, const float* bias, const float* correction, int normalize,
+                        int* chosen, float* weights, cudaStream_t stream);
 /* act[t * top + k] = f(Wg[e] x[t]) * (Wu[e] x[t]), e = chosen[t][k]; gate_up [experts][2 ff]
  * [width] (gate rows first) */
 int hx_expert_gate_up(const void* x, int ld_x, const void* gate_up, const int* chosen, void* act,
@@ -323,6 +343,64 @@ int hx_expert_combine(const float* y, int ld_y, const int* pair_row, const float
 int hx_expert_identity_add(const void* x, int ld_x, const int* chosen, const float* weights,
                            float* out, int ld_out, int dtype, int tokens, int top, int width,
                            int experts, cudaStream_t stream);
+
+/* ---- heads with several score maps ------------------------------------------------------ */
+/* rows [q: heads * maps * dim | k: kv_heads * maps * dim | v: kv_heads * vdim | ...] in `dtype` (raw) or
+ * as float32 sums (accum): + bias, a causal filter over time [channels][taps] (state: the last
+ * taps - 1 inputs, [taps - 1][channels] float32 per slot), RMS norm per map of a query or key head
+ * (weights [dim], may be null), rotation of neighbouring pairs over the first `rot` coordinates by
+ * table rows [position][rot / 2]; queries to rows of row_dim per (head, map), zero outside the
+ * map's part; keys (all maps of a head in one row) and values to the token's pages.  kv_heads 0:
+ * queries only */
+int hx_filtered_heads(const void* raw, int ld_raw, const float* accum, int ld_accum, int dtype,
+                      const float* bias, const float* filter, int taps, float* state,
+                      long long state_stride, const float* q_norm, const float* k_norm, float eps,
+                      const float* cosine, const float* sine, int rot, int table_rows, void* out,
+                      int ld_out, void* k_cache, void* v_cache, const int* positions,
+                      const int* token_request, const int* request_slot, const int* request_start,
+                      const int* block_tables, int table_stride, int tokens, int heads, int kv_heads,
+                      int maps, int dim, int vdim, int row_dim, int page_size, int num_pages,
+                      int* status, cudaStream_t stream);
+/* o = a1 - lambda a2 of a head's two rows of `context`, over sqrt(mean(o^2) + eps), times scale,
+ * times sigmoid(gate) (gate in `dtype` or gate_sums float32); clear (may be null): accumulator rows
+ * to zero, whose last heads * vdim columns gate_sums are */
+int hx_map_difference(const void* context, int ld_context, const void* gate, int ld_gate,
+                      const float* gate_sums, int ld_sums, int dtype, float lambda, float scale,
+                      float eps, void* out, int ld_out, float* clear, int ld_clear, int clear_width,
+                      int tokens, int heads, int vdim, int row_dim, cudaStream_t stream);
+
+/* ---- matrix memory with exponential gates ------------------------------------------------ */
+/* floats of a request's state row: per head the matrix [dim][vdim + 1] (hx_scan_state_floats), then the
+ * running maxima [heads]; 0: no kernel takes the sizes */
+int hx_matrix_lstm_state_floats(int heads, int dim, int vdim);
+/* sums float32 [input gates | forget gates] + bias -> per head and token the decay's logarithm, the
+ * input's weight and exp(-m), [heads][ld_out] each; the maxima move on */
+int hx_matrix_lstm_gates(const float* sums, int ld, const float* bias, float cap, float* log_decay,
+                         float* push, float* level, int ld_out, float* state,
+                         long long state_stride, const int* request_start, const int* request_slot,
+                         int requests, int tokens, int heads, int dim, int vdim,
+                         cudaStream_t stream);
+/* S <- e^log_decay S + push k [v, 1]', o = q_scale S' q / (max(|n . q|, e^-m) + floor), each head over its
+ * root mean square, times norm, times sigmoid(g).  rows [q | k | v | g] in `dtype` or accum (float32
+ * sums with the gates' columns behind, left zero); gate_sums not null: one token per request, gates
+ * from these columns; scan 0: o and weight hold the recurrence's results already */
+int hx_matrix_lstm(const void* rows, int ld, float* accum, int ld_accum, int dtype,
+                   const float* gate_sums, int ld_gate_sums, const float* bias, float cap,
+                   const float* log_decay, const float* push, const float* level, int ld_gates,
+                   int scan, float q_scale, float floor, const float* norm, float eps, float* state,
+                   long long state_stride, float* o, float* weight, void* out, int ld_out,
+                   const int* token_request, const int* request_start, const int* request_slot,
+                   int requests, int tokens, int heads, int dim, int vdim, cudaStream_t stream);
+/* the same recurrence 64 tokens at a time on the tensor cores (bfloat16): decay and push hold the
+ * logarithms of the decays and the inputs' weights and are overwritten; total and weights are
+ * scratch; o gets q_scale S' q, extra the last column's */
+int hx_state_chunks_supports(int dim, int vdim);
+long long hx_state_chunks_scratch(int heads, int ld_gates);
+int hx_state_chunks(const void* q, const void* k, const void* v, int ld, float* decay, float* push,
+                    float* total, int ld_gates, void* weights, float q_scale, float* state,
+                    long long state_stride, int head_stride, float* o, float* extra,
+                    const int* request_start, const int* request_slot, int requests, int tiles,
+                    int heads, int dim, int vdim, cudaStream_t stream);
 
 /* ---- attention over a cached latent ----------------------------------------------------- */
 /* down [tokens][q_rank + kv_rank + rot] float32: both latents RMS-normed with a weight; the
