@@ -18,7 +18,7 @@ import traces
 from conftest import ROOT, random_tokens
 from engine_harness import Harness, assert_close
 from manatar_configs import CONFIGS, PAGE_SIZE, make_folder
-from plain_manatar import PlainManatar
+from plain_manatar import PlainManatar, to_bfloat16
 
 pytestmark = pytest.mark.gpu
 
@@ -83,8 +83,17 @@ class Expected:
             exact = PlainManatar(folder, "float32")
             self.moved = {name: relative_error(self.logits[name], exact.forward(tokens))
                           for name, tokens in requests.items()}
-            # what rounding does to one row is one draw of its noise: the rows of the model that
-            # it moves most say how large the draws are
+            # what rounding does to a row is one draw; a row where the maps or the recurrence's terms
+            # nearly cancel shows in others (every rounded value moved by half a unit or so first)
+            for seed in range(3):
+                rng = np.random.default_rng(seed)
+                other = PlainManatar(folder, "bfloat16")
+                other.round = lambda values: to_bfloat16(
+                    values * (1.0 + 2.0 ** -9 * rng.normal(size=np.shape(values))))
+                for name, tokens in requests.items():
+                    self.moved[name] = np.maximum(
+                        self.moved[name], 0.7 * relative_error(other.forward(tokens), self.logits[name]))
+            # and the rows of the model that it moves most say how large the draws are
             self.floor = float(np.quantile(np.concatenate(list(self.moved.values())), 0.9))
 
 
@@ -147,7 +156,7 @@ def test_most_bfloat16_rows_are_held_to_the_tolerance(expectations):
     for name in NAMES:
         expected = expectations(name, "bfloat16", 30)
         moved = np.concatenate([rows[:expected.held[request]] for request, rows in expected.moved.items()])
-        assert (4.0 * moved > 0.05).mean() <= 0.6, name
+        assert (4.0 * moved > 0.1).mean() <= 0.5, name
         lengths = [len(rows) for rows in expected.moved.values()]
         assert sum(min(expected.held[request], length) for request, length
                    in zip(expected.moved, lengths)) >= 0.5 * sum(lengths), name
