@@ -532,7 +532,7 @@ def manatar_config(shape: dict, options):
           ("attention", attention(index - 2 if index % 4 == 2 else None))),
         dense if index == 0 else routed) for index in range(shape["num_hidden_layers"]))
     return ManatarConfig(vocab=shape["vocab_size"], width=width, norm_eps=shape["rms_norm_eps"],
-                         residual_mult=0.5, pairs=PairTableConfig(65536, 31, 17), layers=layers,
+                         residual_mult=0.5, pairs=PairTableConfig(65536, 1009, 613), layers=layers,
                          max_positions=shape["max_position_embeddings"])
 
 

@@ -79,7 +79,7 @@ CONFIGS = {
     },
     "fast": {
         "architecture": "Manatar", "vocab": 640, "width": 256, "norm": {"eps": 1e-5},
-        "residual_mult": 0.5, "embedding": {"bigram": {"buckets": 500, "mul_prev": 31, "mul_cur": 7}},
+        "residual_mult": 0.5, "embedding": {"bigram": {"buckets": 500, "mul_prev": 29, "mul_cur": 7}},
         "layers": [_attention(4, 2, 64, 128, 4, 0.3, 64, 20000.0, (6.0, 128, 16.0, 2.0),
                               mlp=_dense(384, 1.5), sharp=1.5),
                    _mlstm(2, 64, 128, 12.0, _moe(8, 2, 128, 128)),
